@@ -12,7 +12,9 @@ groups of layers with different needs, and slots for per-request state of fixed 
   position in them has fallen out of the window of the request's next query; the
   group of full layers keeps them until the request ends.  A window that also keeps
   the first F positions of a request readable forms a group of its own (key
-  ``(W, F)``) that never gives back the pages holding those positions.
+  ``(W, F)``) that never gives back the pages holding those positions.  Layers whose
+  queries read only their own chunk of C positions form a group (key
+  ``("chunk", C)``) that gives a chunk's pages back when the request leaves it.
 * A request holds a **slot**: the row of its block tables and the index of its
   state in every :class:`StateSpec` tensor ([max_slots, *shape], zeroed at
   admission).  Freed pages and slots are used again, most recently freed first.
@@ -57,6 +59,7 @@ class LayerCache:
     writes: bool = True
     window: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
     states: Optional[Dict[str, torch.Tensor]] = None  # a state made of named tensors, each [max_slots, *shape]
     table_host: Optional[np.ndarray] = None  # the host's view of the block table (int32 [max_slots, table_width]), for
     #                                          mixers that plan a prompt step's work from the pages it reads
@@ -92,8 +95,9 @@ class _PoolView:
 
 
 class _Group:
-    def __init__(self, mgr, index, window, n_pages, max_slots, width, device, keep_first=0):
+    def __init__(self, mgr, index, window, n_pages, max_slots, width, device, keep_first=0, chunk=None):
         self.index = index
+        self.chunk = chunk
         self.window = window
         self.keep_first = keep_first
         self.caches: List[int] = []
@@ -146,11 +150,14 @@ class CacheManager:
             if cs is not None and cs.paged is not None:
                 window = cs.paged.window
                 keep = int(getattr(cs.paged, "keep_first", 0) or 0) if window is not None else 0
-                key = window if keep == 0 else (window, keep)
+                chunk = cs.paged.chunk
+                if chunk is not None and (window is not None or chunk < 1):
+                    raise CacheError(f"cache {idx}: a chunk is a positive number of positions and goes without a window")
+                key = ("chunk", chunk) if chunk is not None else window if keep == 0 else (window, keep)
                 if key not in self.groups:
                     n = n_pages[key] if isinstance(n_pages, dict) else int(n_pages)
                     self.groups[key] = _Group(self, len(self.groups), window, n, self.max_slots, self.table_width,
-                                              self.device, keep_first=keep)
+                                              self.device, keep_first=keep, chunk=chunk)
                 g = self.groups[key]
                 g.caches.append(idx)
                 for ts in cs.paged.tensors:
@@ -181,6 +188,8 @@ class CacheManager:
         for g in order:
             if g.keep_first:
                 self._lib.fxh_set_keep_first(self._h, g.index, g.keep_first)
+            if g.chunk is not None:
+                self._lib.fxh_set_chunk(self._h, g.index, g.chunk)
         for g in order:
             g.table = np.ctypeslib.as_array(self._lib.fxh_table(self._h, g.index), shape=(self.max_slots, self.table_width))
         self._order = order
@@ -245,9 +254,9 @@ class CacheManager:
         return self._ok(self._lib.fxh_reserve(self._h, int(slot), int(new_len)), slot) == 0
 
     def commit(self, slot: int, new_len: int) -> None:
-        """The request now holds ``new_len`` positions.  Windowed groups give back the
+        """The request now holds ``new_len`` positions.  Windowed and chunked groups give back the
         pages that no later query can read: the next query, at position new_len,
-        reads from new_len - W + 1 on."""
+        reads from new_len - W + 1 (from its chunk's start) on."""
         self._ok(self._lib.fxh_commit(self._h, int(slot), int(new_len)), slot)
 
     def reserve_step(self, slots: Sequence[int], counts: Sequence[int]) -> Optional[List[int]]:
@@ -274,6 +283,8 @@ class CacheManager:
 
     @staticmethod
     def _key(g):
+        if g.chunk is not None:
+            return ("chunk", g.chunk)
         return g.window if not g.keep_first else (g.window, g.keep_first)
 
     def held_pages(self, slot: int) -> Dict[object, List[int]]:
@@ -313,6 +324,7 @@ class CacheManager:
             writes=writes,
             window=g.window if g is not None else None,
             keep_first=g.keep_first if g is not None else 0,
+            chunk=g.chunk if g is not None else None,
             states=self._named_state[cache_index],
             table_host=g.table if g is not None else None,
         )

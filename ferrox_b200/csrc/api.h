@@ -22,13 +22,15 @@ int fx_embed(const void* table, int dtype, const int* ids, float* out, int n_tok
 // h[r] += scale * y[r] and, with a weight w, x_out[r] = rmsnorm(h[r]) * w on the new rows (elementwise.cu)
 int fx_scaled_add_norm(float* h, const float* y, float scale, const void* w, int w_dtype, float eps, void* x_out,
                        int x_dtype, int n_rows, int hidden, void* stream);
+int fx_embed_norm(const void* table, int dtype, const int* ids, const void* w, int w_dtype, float eps, float* out,
+                  int n_tokens, int hidden, int vocab, int* status, void* stream);   // the embedding's rows, RMS-normed
 int fx_rmsnorm(const float* x, const int* rows, const void* w, int w_dtype, float eps, void* out, int out_dtype,
                int n_rows, int hidden, void* stream);
 int fx_silu_mul(const void* gu, long ld_in, void* out, long ld_out, int dtype, const int* n_rows_dev, int rows, int n,
                 void* stream);
 int fx_glu_mul(const void* gu, long ld_in, void* out, long ld_out, int dtype, const int* n_rows_dev, int rows, int n,
                int act, float act_limit, float act_alpha, void* stream);   // act 0: SiLU(gate) * up, 1: ReLU(gate) * up,
-                                                                          // 2: the clamped unit (fx_clamped_glu)
+                                                                          // 2: the clamped unit, 3: GELU (fx_gate)
 int fx_rope_kv_write(void* qkv, int dtype, long ld, const int* positions, const int* token_seq, const int* seq_slot,
                      const float* inv_freq, const float* cos_sin, int rotary_dim, int pairing, void* k_pages, void* v_pages, const int* block_table,
                      int table_width, int page_size, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
@@ -49,7 +51,10 @@ int fx_paged_attention_ex(const void* q, long ldq, long ldqh, const void* k_page
                           int dtype, const int* block_table, int table_width, int page_size, const int* positions,
                           const int* token_seq, const int* seq_slot, void* out, long ldo, long ldoh, int n_tokens,
                           int n_heads, int n_kv_heads, int key_dim, int value_dim, int window, float scale, float softcap,
-                          const float* slopes, int keep_first, const float* sinks, int value_share, void* stream);
+                          const float* slopes, int keep_first, const float* sinks, int value_share, int chunk,
+                          const void* gate, long ldg, void* stream);
+// chunk > 0: a query sees the keys of its own chunk of that many positions only.  gate (optional, token rows of n_heads *
+// value_dim): the result is multiplied by sigmoid(gate).
 // sinks (optional, one per head): exp(sinks[h]) joins the softmax's denominator once.  value_share >= 1: that many
 // consecutive key heads read one value head (the value pages hold n_kv_heads / value_share heads).
 
@@ -61,7 +66,7 @@ int fx_general_attention(const void* q, long ldq, long ldqh, const void* k_pages
                          const int* token_seq, const int* seq_slot, const int* items, int n_items, void* out, long ldo,
                          long ldoh, int n_heads, int n_kv_heads, int key_dim, int value_dim, int window, float scale,
                          const float* slopes, int n_splits, float* part_o, float* part_ml, int keep_first, float softcap,
-                         const float* sinks, int value_share, void* stream);
+                         const float* sinks, int value_share, int chunk, const void* gate, long ldg, void* stream);
 
 int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                             const int* block_table, int table_width, int page_size, const int* items, int n_items,
@@ -112,6 +117,21 @@ int fx_route_fused(const void* X, long ldx, const void* W, long ldw, int n_token
                    int top_k, int renorm, float* logits, long ldl, int* ids, float* weights, int* offsets, int* src_token,
                    int* inv_perm, int* active, int n_slots, void* xp_out, long ldxp, const float* choice_bias,
                    float weight_scale, float renorm_eps, void* stream);
+// Routing by a table of token ids, for n_tables layers at once (tables: device array of n_tables pointers to int32
+// [vocab, top_k]); outputs per table side by side, weights (1 / top_k) once (moe_routing.cu)
+int fx_route_table(const int* token_ids, const int* const* tables, int n_tables, int vocab, int n_tokens, int n_experts,
+                   int top_k, float* weights, int* offsets, int* src_token, int* inv_perm, int* active, int n_slots,
+                   void* stream);
+// h += rms(z) * w_post, x_out = rms(h) * w_next; z = y, or a token's expert rows added up (layernorm.cu)
+int fx_rmsnorm_residual(float* h, const void* y, int y_dtype, const int* place, const float* weight, int top_k,
+                        const void* shared, const float* shared_gate, long gate_ld, const void* w_post, int wp_dtype, float eps,
+                        const void* w_next, int wn_dtype, float eps_next, void* x_out, int x_dtype, int n_rows, int hidden,
+                        void* stream);
+// rotation of q and k, mixing of v with another layer's values, cache write (attention_prep.cu)
+int fx_rotary_mix_store(void* qkv, int dtype, long ld, const int* positions, const int* token_seq, const int* seq_slot,
+                        const float* cos_sin, int rot, int pairing, const void* v_first, long ld_first, float lambda,
+                        void* k_pages, void* v_pages, const int* block_table, int table_width, int page_size, int n_tokens,
+                        int n_heads, int n_kv_heads, int key_dim, int value_dim, int write_cache, int* status, void* stream);
 int fx_rope_table(const int* positions, const float* inv_freq, int n_tokens, int half, float* cos_sin, float magnitude,
                   void* stream);   // cos and sin times `magnitude`
 // A few tokens against a plain matrix that fits the shared memory of all SMs together (gemm_slab.cu): every block asks

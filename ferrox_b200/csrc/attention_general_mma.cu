@@ -76,7 +76,11 @@ struct GArgs {
     float cap_log2e, scale_over_cap;
     const float* sinks;   // (optional, one per head) exp(sinks[h]) joins the softmax's denominator once
     int value_share;      // consecutive key heads that read one value head
+    int chunk;            // > 0: a query sees the keys of its own chunk of that many positions only
+    const bf16* gate; long ldg;   // (optional) token rows of n_heads * value_dim: the result times sigmoid(gate)
 };
+
+__device__ __forceinline__ float sigmoid_of(float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); }
 
 // DVMAX: most value columns one warp accumulates.  NSPLIT: sets of 4 warps that share out the value columns.
 // BKEY: keys a block of the loop holds.
@@ -115,7 +119,7 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
     const int* table = a.block_table + (long)a.seq_slot[entry] * a.table_width;
     const int kchunks = a.key_dim / 8, vchunks = a.value_dim / 8;   // 16-byte chunks per row
     int last_pos = pos0 + n_tok - 1;
-    int key_lo = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;   // first key any row may see
+    int key_lo = fx_first_key(pos0, a.window, a.chunk);   // first key any row may see
     int keep = a.keep_first;   // kept first positions this block takes
     if (a.n_splits > 1) {      // (one token a tile) this block's run of the token's keys
         int k_begin, k_end;
@@ -175,7 +179,7 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
     const int r0 = qrow0 + g, r1 = r0 + 8;
     // each row's own position, first visible key and slope (in units of log2 e)
     const int p_row0 = pos0 + min(r0, rows - 1) / n_h, p_row1 = pos0 + min(r1, rows - 1) / n_h;
-    const int lo0 = max(a.window > 0 ? p_row0 - a.window + 1 : 0, key_lo), lo1 = max(a.window > 0 ? p_row1 - a.window + 1 : 0, key_lo);
+    const int lo0 = max(fx_first_key(p_row0, a.window, a.chunk), key_lo), lo1 = max(fx_first_key(p_row1, a.window, a.chunk), key_lo);
     const int hi0 = min(p_row0, last_pos), hi1 = min(p_row1, last_pos);      // each row's last visible key here
     float sl0 = 0.f, sl1 = 0.f;
     if (a.slopes) {
@@ -184,7 +188,7 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
     }
     // the warp's rows cover the tokens of rows qrow0 .. qrow0 + 15
     const int w_first = pos0 + min(qrow0, rows - 1) / n_h, w_last = min(last_pos, pos0 + min(qrow0 + 15, rows - 1) / n_h);
-    const int w_lo = max(key_lo, (a.window > 0 && w_first - a.window + 1 > 0) ? w_first - a.window + 1 : 0);
+    const int w_lo = max(key_lo, fx_first_key(w_first, a.window, a.chunk));
 
     for (int blk = 0; blk < n_blocks; ++blk) {
         const int buf = blk & 1;
@@ -307,14 +311,22 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
         if (l0 > 0.f) { const float mm = fmaxf(m0, k0), f = exp2f(m0 - mm); inv0 = f / (l0 * f + exp2f(k0 - mm)); }
         if (l1 > 0.f) { const float mm = fmaxf(m1, k1), f = exp2f(m1 - mm); inv1 = f / (l1 * f + exp2f(k1 - mm)); }
     }
+    const bf16* g0 = a.gate ? a.gate + (long)(tok0 + min(r0, rows - 1) / n_h) * a.ldg + (long)(head0 + min(r0, rows - 1) % n_h) * a.value_dim + col0 : nullptr;
+    const bf16* g1 = a.gate ? a.gate + (long)(tok0 + min(r1, rows - 1) / n_h) * a.ldg + (long)(head0 + min(r1, rows - 1) % n_h) * a.value_dim + col0 : nullptr;
     bf16* o0 = a.out + (long)(tok0 + min(r0, rows - 1) / n_h) * a.ldo + (long)(head0 + min(r0, rows - 1) % n_h) * a.ldoh + col0;
     bf16* o1 = a.out + (long)(tok0 + min(r1, rows - 1) / n_h) * a.ldo + (long)(head0 + min(r1, rows - 1) % n_h) * a.ldoh + col0;
 #pragma unroll
     for (int i = 0; i < ON; ++i) {
         const int col = i * 8 + 2 * t4;
         if (col < my_cols) {
-            if (r0 < rows) *reinterpret_cast<uint32_t*>(o0 + col) = pack_bf16(o[i][0] * inv0, o[i][1] * inv0);
-            if (r1 < rows) *reinterpret_cast<uint32_t*>(o1 + col) = pack_bf16(o[i][2] * inv1, o[i][3] * inv1);
+            float x0 = o[i][0] * inv0, x1 = o[i][1] * inv0, x2 = o[i][2] * inv1, x3 = o[i][3] * inv1;
+            if (a.gate) {      // the output gate, on the 32-bit result
+                const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g0 + col));
+                const float2 gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g1 + col));
+                x0 *= sigmoid_of(ga.x); x1 *= sigmoid_of(ga.y); x2 *= sigmoid_of(gb.x); x3 *= sigmoid_of(gb.y);
+            }
+            if (r0 < rows) *reinterpret_cast<uint32_t*>(o0 + col) = pack_bf16(x0, x1);
+            if (r1 < rows) *reinterpret_cast<uint32_t*>(o1 + col) = pack_bf16(x2, x3);
         }
     }
 }
@@ -322,13 +334,14 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
 // One block a (token, head): the runs of a token's keys added up, each weighted by 2^(its maximum - the largest).
 __global__ void general_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                      const int* __restrict__ positions, bf16* __restrict__ out, long ldo, long ldoh,
-                                     int n_heads, int value_dim, int n_splits, int window, const float* __restrict__ sinks)
+                                     int n_heads, int value_dim, int n_splits, int window, const float* __restrict__ sinks,
+                                     int chunk, const bf16* __restrict__ gate, long ldg)
 {
     fx_pdl_wait();
     const int tkn = blockIdx.x, h = blockIdx.y;
     const long base = ((long)tkn * n_heads + h) * n_splits;
     const int pos = positions[tkn];
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = fx_first_key(pos, window, chunk);
     auto has_keys = [&](int s) { int b, e; fx_split_range(pos, lo, s, n_splits, 0, b, e); return b < e; };
     float mm = -INFINITY;
     for (int s = 0; s < n_splits; ++s)
@@ -349,7 +362,9 @@ __global__ void general_merge_kernel(const float* __restrict__ part_o, const flo
             ll += part_ml[(base + s) * 2 + 1] * w;
             acc += part_o[(base + s) * value_dim + e] * w;
         }
-        out[(long)tkn * ldo + (long)h * ldoh + e] = __float2bfloat16_rn(ll > 0.f ? acc / ll : 0.f);
+        float x = ll > 0.f ? acc / ll : 0.f;
+        if (gate) x *= sigmoid_of(__bfloat162float(gate[(long)tkn * ldg + (long)h * value_dim + e]));
+        out[(long)tkn * ldo + (long)h * ldoh + e] = __float2bfloat16_rn(x);
     }
 }
 
@@ -365,7 +380,7 @@ int launch(dim3 grid, size_t smem, cudaStream_t s, const GArgs& a)
     if (a.n_splits > 1)
         fx_launch_pdl(general_merge_kernel, dim3(grid.x, a.n_heads), dim3(64), 0, s, (const float*)a.part_o,
                       (const float*)a.part_ml, a.positions, a.out, a.ldo, a.ldoh, a.n_heads, a.value_dim, a.n_splits,
-                      a.window, a.sinks);
+                      a.window, a.sinks, a.chunk, a.gate, a.ldg);
     return fx_launch_status();
 }
 
@@ -396,6 +411,8 @@ extern "C" int fx_general_attention_ok(int key_dim, int value_dim, int alias)
 
 // items: int32 [n_items, 5] = (first flat token, tokens, entry, first query head, heads), heads of one kv head,
 // tokens x heads <= 64; or nullptr: one token a tile, n_items = tokens.  bfloat16 only.
+// chunk > 0: a query sees the keys of its own chunk of that many positions (counted from the request's start) only.
+// gate (optional): token rows of n_heads * value_dim, ldg elements apart; the result is multiplied by sigmoid(gate).
 // softcap c > 0: the scaled scores pass through c tanh(s / c) before bias and softmax.  sinks (optional, one per
 // head): exp(sinks[h]) joins the denominator once (with runs: in the merge).  value_share >= 1: that many consecutive
 // key heads read one value head (value head = key head / value_share).
@@ -407,7 +424,8 @@ extern "C" int fx_general_attention(const void* q, long ldq, long ldqh, const vo
                                     int n_items, void* out, long ldo, long ldoh, int n_heads, int n_kv_heads,
                                     int key_dim, int value_dim, int window, float scale, const float* slopes,
                                     int n_splits, float* part_o, float* part_ml, int keep_first, float softcap,
-                                    const float* sinks, int value_share, void* stream)
+                                    const float* sinks, int value_share, int chunk, const void* gate, long ldg,
+                                    void* stream)
 {
     if (n_items <= 0) return FX_OK;
     if (value_share < 1) value_share = 1;
@@ -433,6 +451,9 @@ extern "C" int fx_general_attention(const void* q, long ldq, long ldqh, const vo
     a.softcap = softcap > 0.f ? softcap : 0.f;
     a.cap_log2e = a.softcap * 1.4426950408889634f; a.scale_over_cap = a.softcap > 0.f ? scale / a.softcap : 0.f;
     a.sinks = sinks; a.value_share = value_share;
+    if (chunk < 0 || (chunk > 0 && a.keep_first > 0)) return FX_ERR_SIZE;
+    if (gate && (ldg % 2 || (uintptr_t)gate % 4)) return FX_ERR_ALIGN;
+    a.chunk = chunk; a.gate = (const bf16*)gate; a.ldg = ldg;
     a.n_splits = n_splits > 1 ? n_splits : 1; a.part_o = part_o; a.part_ml = part_ml;
     if (a.n_splits > 1 && (items || !part_o || !part_ml || a.n_splits > 65535)) return FX_ERR_SIZE;
     const int bkey = general_bkey(key_dim, value_dim, alias);

@@ -32,6 +32,8 @@
 // `sinks` (optional, one per head): exp(sinks[h]) is added to the softmax's denominator, once, unscaled.
 // `value_share` (>= 1): that many consecutive key heads read one value head (value head = key head / value_share;
 // the value pages hold n_kv_heads / value_share heads), for attention maps of their own keys over shared values.
+// `chunk` (> 0): a query sees only the keys of its own chunk of that many positions, counted from the request's start.
+// `gate` (optional, token rows of n_heads * value_dim): the result is multiplied element by element by sigmoid(gate).
 #include "common.cuh"
 #include "api.h"
 
@@ -48,7 +50,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
     const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
     T* __restrict__ out, long ldo, long ldoh, int n_heads, int n_kv_heads, int key_dim, int value_dim, int window,
     float scale, float softcap, const float* __restrict__ slopes, int keep_first, const float* __restrict__ sinks,
-    int value_share)
+    int value_share, int chunk, const T* __restrict__ gate, long ldg)
 {
     __shared__ float q_s[WARPS][MAX_DK];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -64,7 +66,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
     __syncwarp();
     const float slope = slopes ? slopes[h] : 0.f;
 
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = fx_first_key(pos, window, chunk);
     float m = -INFINITY, l = 0.f;
     float acc[NV];
 #pragma unroll
@@ -127,7 +129,11 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int d = lane + 32 * i;
-        if (d < value_dim) o[d] = from_f32<T>(acc[i] * inv);
+        if (d < value_dim) {
+            float v = acc[i] * inv;
+            if (gate) v *= 1.0f / (1.0f + expf(-to_f32(gate[(long)t * ldg + (long)h * value_dim + d])));
+            o[d] = from_f32<T>(v);
+        }
     }
 }
 
@@ -136,14 +142,14 @@ int launch_paged(const void* q, long ldq, long ldqh, const void* k_pages, const 
                  const int* block_table, int table_width, int page_size, const int* positions, const int* token_seq,
                  const int* seq_slot, void* out, long ldo, long ldoh, int n_tokens, int n_heads, int n_kv_heads,
                  int key_dim, int value_dim, int window, float scale, float softcap, const float* slopes, int keep_first,
-                 const float* sinks, int value_share, cudaStream_t s)
+                 const float* sinks, int value_share, int chunk, const void* gate, long ldg, cudaStream_t s)
 {
     dim3 grid(n_tokens, (unsigned)fx_cdiv(n_heads, WARPS));
 #define FX_GO(NV)                                                                                                     \
     paged_attention_kernel<T, NV><<<grid, WARPS * 32, 0, s>>>((const T*)q, ldq, ldqh, (const T*)k_pages,              \
         (const T*)v_pages, ldk, ldv, block_table, table_width, page_size, positions, token_seq, seq_slot, (T*)out,    \
         ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks,        \
-        value_share)
+        value_share, chunk, (const T*)gate, ldg)
     if (value_dim <= 64) FX_GO(2);
     else if (value_dim <= 128) FX_GO(4);
     else if (value_dim <= 256) FX_GO(8);
@@ -162,12 +168,13 @@ extern "C" int fx_paged_attention_ex(const void* q, long ldq, long ldqh, const v
                                      void* out, long ldo, long ldoh, int n_tokens, int n_heads, int n_kv_heads,
                                      int key_dim, int value_dim, int window, float scale, float softcap,
                                      const float* slopes, int keep_first, const float* sinks, int value_share,
-                                     void* stream)
+                                     int chunk, const void* gate, long ldg, void* stream)
 {
     if (n_tokens <= 0) return FX_OK;
     if (value_share < 1) value_share = 1;
     if (n_kv_heads % value_share) return FX_ERR_SIZE;
     if (keep_first < 0 || window <= 0) keep_first = 0;
+    if (chunk < 0 || (chunk > 0 && keep_first > 0)) return FX_ERR_SIZE;
     if (key_dim > MAX_DK || value_dim > MAX_DV || key_dim <= 0 || value_dim <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || ldk < key_dim || ldv < value_dim)
         return FX_ERR_SIZE;
@@ -175,11 +182,11 @@ extern "C" int fx_paged_attention_ex(const void* q, long ldq, long ldqh, const v
     if (dtype == FX_F32)
         return launch_paged<float>(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, table_width, page_size,
                                    positions, token_seq, seq_slot, out, ldo, ldoh, n_tokens, n_heads, n_kv_heads,
-                                   key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, s);
+                                   key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, chunk, gate, ldg, s);
     if (dtype == FX_BF16)
         return launch_paged<bf16>(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, table_width, page_size,
                                   positions, token_seq, seq_slot, out, ldo, ldoh, n_tokens, n_heads, n_kv_heads,
-                                  key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, s);
+                                  key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, chunk, gate, ldg, s);
     return FX_ERR_DTYPE;
 }
 
@@ -192,5 +199,5 @@ extern "C" int fx_paged_attention(const void* q, long ldq, const void* k_pages, 
 {
     return fx_paged_attention_ex(q, ldq, head_dim, k_pages, v_pages, head_dim, head_dim, dtype, block_table, table_width,
                                  page_size, positions, token_seq, seq_slot, out, ldo, head_dim, n_tokens, n_heads,
-                                 n_kv_heads, head_dim, head_dim, window, scale, softcap, nullptr, 0, nullptr, 1, stream);
+                                 n_kv_heads, head_dim, head_dim, window, scale, softcap, nullptr, 0, nullptr, 1, 0, nullptr, 0, stream);
 }

@@ -78,6 +78,93 @@ __global__ void qk_norm_store_kernel(T* __restrict__ qkv, long ld, const int* __
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Rows of [q heads | k heads | v heads] (head widths D, D, V) of an attention that rotates part of its heads and mixes
+// its values with another layer's:
+//   the first rot elements of every q and k head turned by the token's angles (cos_sin [tokens][rot / 2][2]; pairing 0:
+//   pairs (i, i + rot / 2), 1: neighbours; cos_sin == nullptr: none), q in place, k straight into its page;
+//   v <- (1 - lambda) v + lambda v_first (v_first: row views of the same token's values in the other layer; nullptr:
+//   v as it is), into its page.  The rows' own v stays as projected, for the layers that read it as v_first.
+// One block a token; items of N elements (of both partners of a pair): N = 1, or 16 bytes where widths and rows allow.
+template <typename T, int N> struct Items {      // N elements as 32-bit values
+    static __device__ __forceinline__ void load(const T* p, float* o) { o[0] = to_f32(*p); }
+    static __device__ __forceinline__ void store(T* p, const float* o) { *p = from_f32<T>(o[0]); }
+};
+template <> struct Items<float, 4> : Pack<float> {};
+template <> struct Items<bf16, 8> : Pack<bf16> {};
+
+template <typename T, int N>
+__global__ void rotary_mix_store_kernel(T* __restrict__ qkv, long ld, const int* __restrict__ positions,
+                                        const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
+                                        const float* __restrict__ cos_sin, int rot, int pairing,
+                                        const T* __restrict__ v_first, long ld_first, float lambda,
+                                        T* __restrict__ k_pages, T* __restrict__ v_pages,
+                                        const int* __restrict__ block_table, int table_width, int page_size, int H, int G,
+                                        int D, int V, int write_cache, int* __restrict__ status)
+{
+    fx_pdl_wait();
+    const int t = blockIdx.x;
+    const int pos = positions[t];
+    T* row = qkv + (long)t * ld;
+    long place = -1;      // (page, kv head 0, position in the page) as one index
+    if (write_cache) {
+        const int page = block_table[(long)seq_slot[token_seq[t]] * table_width + pos / page_size];
+        if (page < 0) { if (threadIdx.x == 0 && status) atomicExch(status, 2); }
+        else place = (long)page * G * page_size + (pos % page_size);
+    }
+    const int half = cos_sin ? rot >> 1 : 0;
+    const float* cs = cos_sin + (long)t * half * 2;
+    const int per_head = half / N;                  // rotated items of a head
+    const int rest = (D - 2 * half) / N;            // and those that pass unchanged (k heads only: they are copied)
+    const int n_q = H * per_head, n_k = G * (per_head + rest), n_v = G * (V / N);
+    for (int idx = threadIdx.x; idx < n_q + n_k + n_v; idx += blockDim.x) {
+        if (idx < n_q + n_k) {
+            const bool is_q = idx < n_q;
+            const int j = is_q ? idx : idx - n_q, per = is_q ? per_head : per_head + rest;
+            const int h = j / per, c = j - h * per;
+            T* x = row + (long)(is_q ? h : H + h) * D;
+            T* dst = is_q ? x : place >= 0 ? k_pages + (place + (long)h * page_size) * D : nullptr;
+            if (!dst) continue;
+            if (c >= per_head) {      // beyond the rotated part
+                const int i = 2 * half + (c - per_head) * N;
+                float a[N];
+                Items<T, N>::load(x + i, a);
+                Items<T, N>::store(dst + i, a);
+            } else if (pairing == 0) {
+                const int i = c * N;
+                float a[N], b[N], ra[N], rb[N];
+                Items<T, N>::load(x + i, a);
+                Items<T, N>::load(x + i + half, b);
+#pragma unroll
+                for (int e = 0; e < N; ++e) {
+                    const float2 f = *reinterpret_cast<const float2*>(cs + (i + e) * 2);
+                    ra[e] = a[e] * f.x - b[e] * f.y;
+                    rb[e] = b[e] * f.x + a[e] * f.y;
+                }
+                Items<T, N>::store(dst + i, ra);
+                Items<T, N>::store(dst + i + half, rb);
+            } else {                  // (neighbours: N is 1)
+                const float2 f = *reinterpret_cast<const float2*>(cs + c * 2);
+                const float a = to_f32(x[2 * c]), b = to_f32(x[2 * c + 1]);
+                dst[2 * c] = from_f32<T>(a * f.x - b * f.y);
+                dst[2 * c + 1] = from_f32<T>(b * f.x + a * f.y);
+            }
+        } else if (place >= 0) {
+            const int j = idx - n_q - n_k, per = V / N;
+            const int g = j / per, i = (j - g * per) * N;
+            float a[N];
+            Items<T, N>::load(row + (long)(H + G) * D + (long)g * V + i, a);
+            if (v_first) {
+                float b[N];
+                Items<T, N>::load(v_first + (long)t * ld_first + (long)g * V + i, b);
+#pragma unroll
+                for (int e = 0; e < N; ++e) a[e] = (1.0f - lambda) * a[e] + lambda * b[e];
+            }
+            Items<T, N>::store(v_pages + (place + (long)g * page_size) * V + i, a);
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // The latent form.  Per token: `dkv` = [C latent | R rotated key part] as projected, `q` = H heads of [D | R].
 //   c <- dkv[:C] / sqrt(mean(dkv[:C]^2) + eps) * wc            -> pages[position][0:C]
 //   k_rot <- pairs (2i, 2i+1) of the first rot_dims of dkv[C:] turned by the position's angles, the rest as it is
@@ -214,6 +301,37 @@ extern "C" int fx_qk_norm_store(void* qkv, int dtype, long ld, const int* positi
                   n_heads, n_kv_heads, key_dim, value_dim, write_cache, status, v_eps)
     if (dtype == FX_F32) FX_GO(float);
     else if (dtype == FX_BF16) FX_GO(bf16);
+    else return FX_ERR_DTYPE;
+#undef FX_GO
+    return fx_launch_status();
+}
+
+extern "C" int fx_rotary_mix_store(void* qkv, int dtype, long ld, const int* positions, const int* token_seq,
+                                   const int* seq_slot, const float* cos_sin, int rot, int pairing, const void* v_first,
+                                   long ld_first, float lambda, void* k_pages, void* v_pages, const int* block_table,
+                                   int table_width, int page_size, int n_tokens, int n_heads, int n_kv_heads, int key_dim,
+                                   int value_dim, int write_cache, int* status, void* stream)
+{
+    if (n_tokens <= 0) return FX_OK;
+    if (key_dim <= 0 || value_dim <= 0 || page_size <= 0 || n_heads <= 0 || n_kv_heads <= 0 || pairing < 0 || pairing > 1)
+        return FX_ERR_SIZE;
+    if (!cos_sin) rot = 0;
+    if (rot < 0 || rot % 2 || rot > key_dim) return FX_ERR_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int vw = dtype == FX_F32 ? 4 : 8;
+    const int es = dtype == FX_F32 ? 4 : 2;
+    const bool vec = pairing == 0 && (rot / 2) % vw == 0 && key_dim % vw == 0 && value_dim % vw == 0 && (ld * es) % 16 == 0 &&
+                     (ld_first * es) % 16 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)v_first % 16 == 0 &&
+                     (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0;
+    const int n = vec ? vw : 1;
+    const int items = (n_heads * (rot / 2) + n_kv_heads * (key_dim - rot / 2 + value_dim)) / n;
+    const int nt = threads_for_width(items);
+#define FX_GO(T, N)                                                                                                   \
+    fx_launch_pdl(rotary_mix_store_kernel<T, N>, n_tokens, nt, 0, s, (T*)qkv, ld, positions, token_seq, seq_slot,    \
+                  cos_sin, rot, pairing, (const T*)v_first, ld_first, lambda, (T*)k_pages, (T*)v_pages, block_table, \
+                  table_width, page_size, n_heads, n_kv_heads, key_dim, value_dim, write_cache, status)
+    if (dtype == FX_F32) { if (vec) FX_GO(float, 4); else FX_GO(float, 1); }
+    else if (dtype == FX_BF16) { if (vec) FX_GO(bf16, 8); else FX_GO(bf16, 1); }
     else return FX_ERR_DTYPE;
 #undef FX_GO
     return fx_launch_status();

@@ -36,6 +36,39 @@ __device__ __forceinline__ float load_any(const void* p, int dtype, long i) {
                            : __bfloat162float(reinterpret_cast<const bf16*>(p)[i]);
 }
 
+// 16 bytes of a row as 32-bit values.
+template <typename T> struct Pack;
+template <> struct Pack<float> {
+    static constexpr int N = 4;
+    static __device__ __forceinline__ void load(const float* p, float* o) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+    }
+    static __device__ __forceinline__ void store(float* p, const float* o) {
+        *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]);
+    }
+};
+template <> struct Pack<bf16> {
+    static constexpr int N = 8;
+    static __device__ __forceinline__ void load(const bf16* p, float* o) {
+        const uint4 v = *reinterpret_cast<const uint4*>(p);
+        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            o[2 * i] = __uint_as_float(w[i] << 16);
+            o[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+        }
+    }
+    static __device__ __forceinline__ void store(bf16* p, const float* o) {
+        uint4 v;
+        __nv_bfloat162 a = __floats2bfloat162_rn(o[0], o[1]), b = __floats2bfloat162_rn(o[2], o[3]);
+        __nv_bfloat162 c = __floats2bfloat162_rn(o[4], o[5]), d = __floats2bfloat162_rn(o[6], o[7]);
+        v.x = *reinterpret_cast<uint32_t*>(&a); v.y = *reinterpret_cast<uint32_t*>(&b);
+        v.z = *reinterpret_cast<uint32_t*>(&c); v.w = *reinterpret_cast<uint32_t*>(&d);
+        *reinterpret_cast<uint4*>(p) = v;
+    }
+};
+
 // What a plain product's result may pass through before it is stored (the kernels' `gated` argument below zero:
 // -code): 1 the square of ReLU.
 __device__ __forceinline__ float fx_unary(float x, int code) {
@@ -80,6 +113,31 @@ __device__ __forceinline__ float fx_clamped_glu(float g, float u, float limit, f
     u = fminf(fmaxf(u, -limit), limit);
     const float e = FAST ? __expf(-alpha * g) : expf(-alpha * g);
     return g / (1.0f + e) * (u + 1.0f);
+}
+
+// z * (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) / 2, the tanh form of GELU, written with 1 + tanh(y) = 2 / (1 + e^(-2y)).
+template <bool FAST>
+__device__ __forceinline__ float fx_gelu_tanh(float z) {
+    const float y2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);      // 2 sqrt(2/pi) (z + 0.044715 z^3)
+    return FAST ? __fdividef(z, 1.0f + __expf(-y2)) : z / (1.0f + expf(-y2));
+}
+
+// A gated feed-forward's unit act(g) * u; act 0: SiLU, 1: ReLU, 2: the clamped unit, 3: GELU in its tanh form.  FAST:
+// the hardware's exponential and quotient.
+template <bool FAST>
+__device__ __forceinline__ float fx_gate(float g, float u, int act, float limit, float alpha) {
+    if (act == 2) return fx_clamped_glu<FAST>(g, u, limit, alpha);
+    if (act == 1) return fmaxf(g, 0.f) * u;
+    if (act == 3) return fx_gelu_tanh<FAST>(g) * u;
+    return (FAST ? __fdividef(g, 1.0f + __expf(-g)) : g / (1.0f + expf(-g))) * u;
+}
+
+// The first key the query at position pos may see: of a window of the last `window` positions (0: no window) and of
+// chunks of `chunk` positions counted from the request's start (0: no chunks), in which a query sees its own chunk only.
+__host__ __device__ __forceinline__ int fx_first_key(int pos, int window, int chunk) {
+    int lo = window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
+    if (chunk > 0) { const int c = pos - pos % chunk; lo = c > lo ? c : lo; }
+    return lo;
 }
 
 // Key range [k_begin, k_end) of run `split` of a decoding token at position pos whose first visible key is lo.

@@ -45,6 +45,27 @@ __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict_
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = ok ? to_f32(row[i]) * scale : 0.f;
 }
 
+// out[t, :] = z / sqrt(mean(z^2) + eps) * w with z = table[ids[t], :], for models that norm their embedding.
+template <typename T>
+__global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ ids, const void* __restrict__ w,
+                                  int w_dtype, float eps, float* __restrict__ out, int hidden, int vocab,
+                                  int* __restrict__ status)
+{
+    __shared__ float scratch[33];
+    fx_pdl_wait();
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && threadIdx.x == 0 && status) atomicExch(status, 1);
+    const T* row = table + (long)(ok ? id : 0) * hidden;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) { const float v = to_f32(row[i]); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss / (float)hidden + eps);
+    float* o = out + (long)t * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = ok ? to_f32(row[i]) * scale * load_any(w, w_dtype, i) : 0.f;
+}
+
 // ---------------------------------------------------------------------------
 // RMSNorm: out = x * (1/sqrt(mean(x^2) + eps)) * w, multiplied in that order
 // (reference: crates/ferrox-core/src/matmul.rs:62-69,121-123).  x is the 32-bit
@@ -81,8 +102,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ gu, long ld_in, T* __restr
         const long r = i / n; const int c = (int)(i - r * n);
         const float g = to_f32(gu[r * ld_in + c]);
         const float u = to_f32(gu[r * ld_in + n + c]);
-        out[r * ld_out + c] = from_f32<T>(act == 2 ? fx_clamped_glu<false>(g, u, act_limit, act_alpha)
-                                                   : (act ? fmaxf(g, 0.f) : g / (1.0f + expf(-g))) * u);   // act 1: ReLU
+        out[r * ld_out + c] = from_f32<T>(fx_gate<false>(g, u, act, act_limit, act_alpha));
     }
 }
 
@@ -221,38 +241,7 @@ __global__ void residual_add_kernel(float* __restrict__ h, const T* __restrict__
 }
 
 // ---------------------------------------------------------------------------
-// 16-byte vector forms of the kernels above, used when widths and addresses allow.
-template <typename T> struct Pack;
-template <> struct Pack<float> {
-    static constexpr int N = 4;
-    static __device__ __forceinline__ void load(const float* p, float* o) {
-        const float4 v = *reinterpret_cast<const float4*>(p);
-        o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
-    }
-    static __device__ __forceinline__ void store(float* p, const float* o) {
-        *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]);
-    }
-};
-template <> struct Pack<bf16> {
-    static constexpr int N = 8;
-    static __device__ __forceinline__ void load(const bf16* p, float* o) {
-        const uint4 v = *reinterpret_cast<const uint4*>(p);
-        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            o[2 * i] = __uint_as_float(w[i] << 16);
-            o[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-        }
-    }
-    static __device__ __forceinline__ void store(bf16* p, const float* o) {
-        uint4 v;
-        __nv_bfloat162 a = __floats2bfloat162_rn(o[0], o[1]), b = __floats2bfloat162_rn(o[2], o[3]);
-        __nv_bfloat162 c = __floats2bfloat162_rn(o[4], o[5]), d = __floats2bfloat162_rn(o[6], o[7]);
-        v.x = *reinterpret_cast<uint32_t*>(&a); v.y = *reinterpret_cast<uint32_t*>(&b);
-        v.z = *reinterpret_cast<uint32_t*>(&c); v.w = *reinterpret_cast<uint32_t*>(&d);
-        *reinterpret_cast<uint4*>(p) = v;
-    }
-};
+// 16-byte vector forms of the kernels above (Pack, common.cuh), used when widths and addresses allow.
 
 // RMSNorm, 4 elements per thread and pass (hidden % 4 == 0, rows 16-byte aligned).
 template <typename OT>
@@ -504,6 +493,19 @@ extern "C" int fx_embed(const void* table, int dtype, const int* ids, float* out
     return fx_launch_status();
 }
 
+extern "C" int fx_embed_norm(const void* table, int dtype, const int* ids, const void* w, int w_dtype, float eps, float* out,
+                             int n_tokens, int hidden, int vocab, int* status, void* stream)
+{
+    if (n_tokens <= 0) return FX_OK;
+    if (hidden <= 0 || vocab <= 0 || !w) return FX_ERR_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int nt = threads_for(hidden > 512 ? 512 : hidden);
+    if (dtype == FX_F32) fx_launch_pdl(embed_norm_kernel<float>, n_tokens, nt, 0, s, (const float*)table, ids, w, w_dtype, eps, out, hidden, vocab, status);
+    else if (dtype == FX_BF16) fx_launch_pdl(embed_norm_kernel<bf16>, n_tokens, nt, 0, s, (const bf16*)table, ids, w, w_dtype, eps, out, hidden, vocab, status);
+    else return FX_ERR_DTYPE;
+    return fx_launch_status();
+}
+
 extern "C" int fx_rmsnorm(const float* x, const int* rows, const void* w, int w_dtype, float eps, void* out,
                           int out_dtype, int n_rows, int hidden, void* stream)
 {
@@ -533,7 +535,7 @@ extern "C" int fx_silu_mul(const void* gu, long ld_in, void* out, long ld_out, i
     return fx_glu_mul(gu, ld_in, out, ld_out, dtype, n_rows_dev, rows, n, 0, 0.f, 0.f, stream);
 }
 
-// act(gate) * up over rows of [gate | up]; act 0: SiLU, 1: ReLU; 2: the clamped unit (fx_clamped_glu).
+// act(gate) * up over rows of [gate | up]; act as in fx_gate (common.cuh).
 extern "C" int fx_glu_mul(const void* gu, long ld_in, void* out, long ld_out, int dtype, const int* n_rows_dev,
                           int rows, int n, int act, float act_limit, float act_alpha, void* stream)
 {

@@ -50,7 +50,7 @@ struct SkinnyArgs {
     int c_transposed;              // store C[n][r] instead of C[r][n] (ldc is then the pitch of a feature's row)
     int n_tokens; int N; int K;
     int gate_up_offset;            // gated form: row of `up` matching gate row i is i + gate_up_offset
-    int act;                       // gated form: 0 SiLU, 1 ReLU on the gate, 2 the clamped unit (fx_clamped_glu)
+    int act;                       // gated form: 0 SiLU, 1 ReLU on the gate, 2 the clamped unit, 3 GELU (fx_gate)
     float act_limit, act_alpha;
     const int* group_offsets;      // grouped form: rows [off[e], off[e+1]) belong to expert e
     const int* active_groups;      // grouped form: the experts that got rows, then -1
@@ -203,8 +203,7 @@ __global__ void __launch_bounds__(NTHREADS) skinny_kernel(SkinnyArgs a)
                 if (a.bias) v += load_any(a.bias, a.bias_dtype, n);
                 // (a gated product's bias holds the gate rows' values, then at gate_up_offset the up rows')
                 if (MODE == 1 && a.bias) up += load_any(a.bias, a.bias_dtype, a.gate_up_offset + n);
-                if (MODE == 1) v = a.act == 2 ? fx_clamped_glu<false>(v, up, a.act_limit, a.act_alpha)
-                                               : (a.act ? fmaxf(v, 0.f) : v / (1.0f + expf(-v))) * up;
+                if (MODE == 1) v = fx_gate<false>(v, up, a.act, a.act_limit, a.act_alpha);
                 else if (a.act) v = fx_unary(v, a.act);     // a plain product with an activation on its result
                 auto store = [&](int col, float val) {
                     const long at = a.c_transposed ? (long)col * a.ldc + r : (long)r * a.ldc + col;

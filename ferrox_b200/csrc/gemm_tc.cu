@@ -52,7 +52,7 @@ struct TcArgs {
     int M, N, K;
     int gate_up_offset;             // gated: W row of `up` feature j is gate_up_offset + j
     int act;                        // gated: what the gate passes through before it multiplies `up`: 0 SiLU, 1 ReLU,
-                                    // 2 the clamped unit (fx_clamped_glu) with act_limit and act_alpha
+                                    // 2 the clamped unit with act_limit and act_alpha, 3 GELU (fx_gate)
     float act_limit, act_alpha;
     const int* group_offsets;       // grouped: rows [off[e], off[e+1]) use matrix e
     int n_groups;
@@ -281,8 +281,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_tc_kernel(const __grid_const
                     float x = __uint_as_float(r[j]);
                     if (a.bias) x += bias_s[quad][c * 32 + j];
                     if (GATED && a.bias) u[j] = __float_as_uint(__uint_as_float(u[j]) + bias_up_s[quad][c * 32 + j]);
-                    if (GATED) x = a.act == 2 ? fx_clamped_glu<true>(x, __uint_as_float(u[j]), a.act_limit, a.act_alpha)
-                                           : (a.act ? fmaxf(x, 0.f) : __fdividef(x, 1.0f + __expf(-x))) * __uint_as_float(u[j]);
+                    if (GATED) x = fx_gate<true>(x, __uint_as_float(u[j]), a.act, a.act_limit, a.act_alpha);
                     else if (a.act) x = fx_unary(x, a.act);     // a plain product with an activation on its result
                     v[j] = x;
                 }

@@ -54,7 +54,7 @@ struct SwArgs {
     const void* bias; int bias_dtype;
     int M, N, K;
     int gate_up_offset;
-    int act;                        // gated: 0 SiLU, 1 ReLU on the gate, 2 the clamped unit (fx_clamped_glu)
+    int act;                        // gated: 0 SiLU, 1 ReLU on the gate, 2 the clamped unit, 3 GELU (fx_gate)
     float act_limit, act_alpha;
     const int* group_offsets;
     int n_groups;
@@ -279,8 +279,7 @@ __global__ void __launch_bounds__(NTHREADS, (TNB <= 32 ? 2 : 1)) gemm_tc_swap_ke
                     if (row0 + j >= t.row_end) break;
                     float x = __uint_as_float(r[j]) + bias;
                     if (GATED) u[j] = __float_as_uint(__uint_as_float(u[j]) + bias_up);
-                    if (GATED) x = a.act == 2 ? fx_clamped_glu<true>(x, __uint_as_float(u[j]), a.act_limit, a.act_alpha)
-                                           : (a.act ? fmaxf(x, 0.f) : x / (1.0f + __expf(-x))) * __uint_as_float(u[j]);
+                    if (GATED) x = fx_gate<true>(x, __uint_as_float(u[j]), a.act, a.act_limit, a.act_alpha);
                     else if (a.act) x = fx_unary(x, a.act);     // a plain product with an activation on its result
                     if (a.k_splits > 1) {   // a run of K: the plain partial sum
                         a.partials[((long)t.split * a.M + row0 + j) * a.N + f] = __uint_as_float(r[j]);

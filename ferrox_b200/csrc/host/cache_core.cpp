@@ -9,7 +9,8 @@
 // commit, the pages whose every position is older than new_len - window + 1; a group
 // whose window also keeps the first `keep_first` positions of a request readable
 // never gives back the pages that hold them (logical pages below keep_pages stay
-// mapped beside the held range).
+// mapped beside the held range).  A group with a chunk gives back, at commit, the pages
+// that lie wholly before the chunk of the next position.
 // reserve() is all-or-nothing over all groups.
 //
 // Reference: crates/ferrox-core/src/cache.rs:331-405 (shared pages, LIFO free list),
@@ -23,6 +24,7 @@ namespace {
 
 struct Group {
     int window;  // -1: every earlier position stays readable
+    int chunk = 0;  // > 0: a query reads its own chunk of that many positions only (counted from position 0)
     int keep_pages = 0;  // logical pages at the start of a request that a windowed group never gives back
     int n_pages;
     std::vector<int> free_list;      // back() is handed out next
@@ -84,6 +86,15 @@ int fxh_set_keep_first(void* h, int group, int keep_first)
     Cache* c = static_cast<Cache*>(h);
     if (group < 0 || group >= (int)c->groups.size() || keep_first < 0) return FXH_BAD_SLOT;
     c->groups[group].keep_pages = pages_for(*c, keep_first);
+    return FXH_OK;
+}
+
+// Queries of this (windowless) group read their own chunk of `chunk` positions only.  Set before any request is opened.
+int fxh_set_chunk(void* h, int group, int chunk)
+{
+    Cache* c = static_cast<Cache*>(h);
+    if (group < 0 || group >= (int)c->groups.size() || chunk < 0) return FXH_BAD_SLOT;
+    c->groups[group].chunk = chunk;
     return FXH_OK;
 }
 
@@ -174,9 +185,10 @@ int fxh_commit(void* h, int slot, int new_len)
     if (new_len < c->seq_len[slot]) return FXH_SHRINK;
     c->seq_len[slot] = new_len;
     for (Group& G : c->groups) {
-        if (G.window < 0) continue;
-        // the next query, at position new_len, reads from new_len - window + 1 on
-        int first_needed = new_len - G.window + 1;
+        if (G.window < 0 && G.chunk <= 0) continue;
+        // the next query, at position new_len, reads from new_len - window + 1 on, or from its chunk's start on
+        int first_needed = G.window < 0 ? 0 : new_len - G.window + 1;
+        if (G.chunk > 0 && new_len / G.chunk * G.chunk > first_needed) first_needed = new_len / G.chunk * G.chunk;
         if (first_needed < 0) first_needed = 0;
         int upto = first_needed / c->page_size;
         if (upto > G.n_logical[slot]) upto = G.n_logical[slot];

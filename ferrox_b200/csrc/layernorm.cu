@@ -73,6 +73,114 @@ __global__ void __launch_bounds__(LN_THREADS) layernorm_residual_kernel(
         o[i] = from_f32<OT>((hr[i] - sn.mean) * sn.rstd * load_any(w_next, wn_dtype, i));
 }
 
+// The RMS form: z = y, or z = sum_k weight[t, k] y[place[t, k]] (the rows of a token's experts, added up here) plus a
+// shared expert's row;  h += z / sqrt(mean(z^2) + eps) * w_post;  x_out = h / sqrt(mean(h^2) + eps_next) * w_next (if
+// asked for).  One block a row, which stays in registers from the first pass to the last: a thread holds up to CH items
+// of N elements, N = 1 or 16 bytes of y.
+template <typename T, int N> struct Row {
+    static __device__ __forceinline__ void load(const T* p, float* o) { o[0] = to_f32(*p); }
+};
+template <> struct Row<float, 4> : Pack<float> {};
+template <> struct Row<bf16, 8> : Pack<bf16> {};
+
+constexpr int RMS_THREADS = 512;   // at most
+
+struct RmsArgs {
+    float* h; const void* y;
+    const int* place; const float* weight; int top_k;         // place == nullptr: z is the token's own row of y
+    const void* shared; const float* shared_gate; long gate_ld;
+    const void* w_post; int wp_dtype; float eps;
+    const void* w_next; int wn_dtype; float eps_next;         // w_next == nullptr: no second norm
+    void* x_out; int hidden;
+};
+
+template <typename T, typename OT, int N, int CH>
+__global__ void __launch_bounds__(RMS_THREADS) rms_residual_kernel(RmsArgs a)
+{
+    __shared__ float scratch[33];
+    fx_pdl_wait();
+    const int t = blockIdx.x;
+    const T* y = reinterpret_cast<const T*>(a.y);
+    const T* shared = reinterpret_cast<const T*>(a.shared);
+    float* hr = a.h + (long)t * a.hidden;
+    float sg = 1.f;
+    if (shared && a.shared_gate) sg = 1.0f / (1.0f + expf(-a.shared_gate[(long)t * a.gate_ld]));
+    float z[CH][N], hv[CH][N];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * N;
+        if (i >= a.hidden) continue;
+        // the stream's row is asked for together with y's
+        if (N == 1) hv[c][0] = hr[i];
+        else {
+#pragma unroll
+            for (int e = 0; e + 3 < N; e += 4) Pack<float>::load(hr + i + e, &hv[c][e]);
+        }
+        if (a.place) {
+#pragma unroll
+            for (int e = 0; e < N; ++e) z[c][e] = 0.f;
+            for (int k = 0; k < a.top_k; ++k) {
+                const long r = a.place[(long)t * a.top_k + k];
+                const float w = a.weight ? a.weight[(long)t * a.top_k + k] : 1.f;
+                float v[N];
+                Row<T, N>::load(y + r * a.hidden + i, v);
+#pragma unroll
+                for (int e = 0; e < N; ++e) z[c][e] = fmaf(w, v[e], z[c][e]);
+            }
+            if (shared) {
+                float v[N];
+                Row<T, N>::load(shared + (long)t * a.hidden + i, v);
+#pragma unroll
+                for (int e = 0; e < N; ++e) z[c][e] = fmaf(sg, v[e], z[c][e]);
+            }
+        } else {
+            Row<T, N>::load(y + (long)t * a.hidden + i, z[c]);
+        }
+#pragma unroll
+        for (int e = 0; e < N; ++e) ss = fmaf(z[c][e], z[c][e], ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float r = 1.0f / sqrtf(ss / (float)a.hidden + a.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * N;
+        if (i >= a.hidden) continue;
+#pragma unroll
+        for (int e = 0; e < N; ++e) {
+            hv[c][e] += z[c][e] * r * load_any(a.w_post, a.wp_dtype, i + e);
+            ss = fmaf(hv[c][e], hv[c][e], ss);
+        }
+        if (N == 1) hr[i] = hv[c][0];
+        else {
+#pragma unroll
+            for (int e = 0; e + 3 < N; e += 4) Pack<float>::store(hr + i + e, &hv[c][e]);
+        }
+    }
+    if (!a.w_next) return;      // (uniform)
+    ss = block_sum(ss, scratch);
+    const float rn = 1.0f / sqrtf(ss / (float)a.hidden + a.eps_next);
+    OT* o = reinterpret_cast<OT*>(a.x_out) + (long)t * a.hidden;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * N;
+        if (i >= a.hidden) continue;
+        float v[N];
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[e] = hv[c][e] * rn * load_any(a.w_next, a.wn_dtype, i + e);
+        if (N == 1) o[i] = from_f32<OT>(v[0]);
+        else if (sizeof(OT) == 4) {
+#pragma unroll
+            for (int e = 0; e + 3 < N; e += 4) Pack<float>::store(reinterpret_cast<float*>(o) + i + e, v + e);
+        } else {
+#pragma unroll
+            for (int e = 0; e + 1 < N; e += 2)
+                *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf16*>(o) + i + e) = __floats2bfloat162_rn(v[e], v[e + 1]);
+        }
+    }
+}
+
 __global__ void scale_kernel(float* __restrict__ x, long n, float s)
 {
     fx_pdl_wait();
@@ -116,6 +224,49 @@ extern "C" int fx_layernorm_residual(float* h, const void* y1, int y1_dtype, flo
         fx_launch_pdl(layernorm_residual_kernel<bf16>, n_rows, ln_threads(hidden, n_rows), 0, s, h, y1, y1_dtype, s1, y2, y2_dtype, s2,
                       w_post, wp_dtype, eps, w_next, wn_dtype, eps_next, (bf16*)x_out, hidden);
     else return FX_ERR_DTYPE;
+    return fx_launch_status();
+}
+
+// h += rms(z) * w_post and, with w_next, x_out = rms(h) * w_next on the new rows; z as rms_residual_kernel says.  Refuses
+// (FX_ERR_SIZE) rows of more than 16,384 elements (8,192 where rows are not 16-byte aligned).
+extern "C" int fx_rmsnorm_residual(float* h, const void* y, int y_dtype, const int* place, const float* weight, int top_k,
+                                   const void* shared, const float* shared_gate, long gate_ld, const void* w_post,
+                                   int wp_dtype, float eps, const void* w_next, int wn_dtype, float eps_next, void* x_out,
+                                   int x_dtype, int n_rows, int hidden, void* stream)
+{
+    if (n_rows <= 0) return FX_OK;
+    if (hidden <= 0 || !y || !w_post || (w_next && !x_out) || (place && top_k <= 0) || (shared && !place)) return FX_ERR_SIZE;
+    if ((y_dtype != FX_F32 && y_dtype != FX_BF16) || (w_next && x_dtype != FX_F32 && x_dtype != FX_BF16)) return FX_ERR_DTYPE;
+    RmsArgs a;
+    a.h = h; a.y = y; a.place = place; a.weight = weight; a.top_k = top_k; a.shared = shared; a.shared_gate = shared_gate;
+    a.gate_ld = gate_ld; a.w_post = w_post; a.wp_dtype = wp_dtype; a.eps = eps; a.w_next = w_next; a.wn_dtype = wn_dtype;
+    a.eps_next = eps_next; a.x_out = x_out; a.hidden = hidden;
+    const int vw = y_dtype == FX_F32 ? 4 : 8;
+    const bool vec = hidden % vw == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)shared % 16 == 0 &&
+                     (uintptr_t)x_out % 16 == 0;
+    const int items = vec ? hidden / vw : hidden;
+    // few rows (a decode step): a block's trips through its row are the kernel's time, so an item a thread
+    int nt = 64;
+    const int most = n_rows >= 256 ? 256 : RMS_THREADS, max_ch = vec ? 32 / vw : 16;
+    while (nt < items && nt < most) nt <<= 1;
+    while (fx_cdiv(items, nt) > max_ch && nt < RMS_THREADS) nt <<= 1;
+    const int ch = (int)fx_cdiv(items, nt);
+    if (ch > max_ch) return FX_ERR_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool out32 = !w_next || x_dtype == FX_F32;
+#define FX_GO(T, OT, N, CH) fx_launch_pdl(rms_residual_kernel<T, OT, N, CH>, n_rows, nt, 0, s, a)
+#define FX_CH(T, OT, N)                                                                                              \
+    do { if (ch <= 1) FX_GO(T, OT, N, 1); else if (ch <= 2) FX_GO(T, OT, N, 2); else if (ch <= 4) FX_GO(T, OT, N, 4); \
+         else if (ch <= 8) FX_GO(T, OT, N, (N == 8 ? 4 : 8)); else FX_GO(T, OT, N, (N == 1 ? 16 : 4)); } while (0)
+    if (y_dtype == FX_F32) {
+        if (vec) { if (out32) FX_CH(float, float, 4); else FX_CH(float, bf16, 4); }
+        else { if (out32) FX_CH(float, float, 1); else FX_CH(float, bf16, 1); }
+    } else {
+        if (vec) { if (out32) FX_CH(bf16, float, 8); else FX_CH(bf16, bf16, 8); }
+        else { if (out32) FX_CH(bf16, float, 1); else FX_CH(bf16, bf16, 1); }
+    }
+#undef FX_CH
+#undef FX_GO
     return fx_launch_status();
 }
 

@@ -386,7 +386,87 @@ __global__ void scan_place_kernel(const int* __restrict__ ids, int n, int n_expe
     }
 }
 
+// Routing without a router: token id t's experts are the entries of row t of a table [vocab, top_k] (distinct, below
+// n_experts), each with weight 1 / top_k.  Nothing of it depends on the activations, so ONE launch at the first such
+// layer of a step serves every layer whose table has these sizes: block l counts, sums and places the (token, rank)
+// pairs of table l, all in shared memory.  Outputs per table, `n_tables` of each side by side: offsets [n_experts + 1],
+// src_token [n_tokens * top_k], inv_perm [n_tokens * top_k], active [n_slots]; weights [n_tokens * top_k] once.
+__global__ void __launch_bounds__(1024) route_table_kernel(
+    const int* __restrict__ token_ids, const int* const* __restrict__ tables, int vocab, int n_tokens, int n_experts,
+    int top_k, float* __restrict__ weights, int* __restrict__ offsets, int* __restrict__ src_token,
+    int* __restrict__ inv_perm, int* __restrict__ active, int n_slots)
+{
+    extern __shared__ int table_s[];      // counts [n_experts], then offsets [n_experts]
+    int* counts = table_s;
+    int* offs = table_s + n_experts;
+    fx_pdl_wait();
+    const int* table = tables[blockIdx.x];
+    const long n = (long)n_tokens * top_k;
+    offsets += (long)blockIdx.x * (n_experts + 1);
+    src_token += blockIdx.x * n;
+    inv_perm += blockIdx.x * n;
+    if (active) active += (long)blockIdx.x * n_slots;
+    // (an id outside the vocabulary has raised the step's status in the embedding; here it only must stay in bounds,
+    // and the loader has refused tables with entries outside the experts)
+    auto expert_of = [&](long i) {
+        const int t = (int)(i / top_k), k = (int)(i - (long)t * top_k);
+        const int id = token_ids[t];
+        const int e = id >= 0 && id < vocab ? table[(long)id * top_k + k] : k;
+        return e >= 0 && e < n_experts ? e : 0;
+    };
+    for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
+    __syncthreads();
+    for (long i = threadIdx.x; i < n; i += blockDim.x) {
+        atomicAdd(&counts[expert_of(i)], 1);
+        if (blockIdx.x == 0) weights[i] = 1.0f / (float)top_k;
+    }
+    __syncthreads();
+    if (threadIdx.x < 32) {
+        // offsets = running sum of the counts, 32 experts a pass; the experts with rows, in ascending order
+        const int lane = threadIdx.x;
+        int run = 0, n_active = 0;
+        for (int e0 = 0; e0 < n_experts; e0 += 32) {
+            const int e = e0 + lane;
+            const int c = e < n_experts ? counts[e] : 0;
+            int incl = c;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xffffffffu, incl, o); if (lane >= o) incl += v; }
+            const int off = run + incl - c;
+            if (e < n_experts) { offs[e] = off; offsets[e] = off; counts[e] = 0; }      // the count becomes the cursor
+            const unsigned has = __ballot_sync(0xffffffffu, c > 0);
+            if (active && c > 0) {
+                const int slot = n_active + __popc(has & ((1u << lane) - 1u));
+                if (slot < n_slots) active[slot] = e;
+            }
+            n_active += __popc(has);
+            run += __shfl_sync(0xffffffffu, incl, 31);
+        }
+        if (lane == 0) offsets[n_experts] = run;
+        if (active) for (int i = min(n_active, n_slots) + lane; i < n_slots; i += 32) active[i] = -1;
+    }
+    __syncthreads();
+    for (long i = threadIdx.x; i < n; i += blockDim.x) {
+        const int e = expert_of(i);
+        const int r = offs[e] + atomicAdd(&counts[e], 1);
+        src_token[r] = (int)(i / top_k);
+        inv_perm[i] = r;
+    }
+}
+
 }  // namespace
+
+extern "C" int fx_route_table(const int* token_ids, const int* const* tables, int n_tables, int vocab, int n_tokens,
+                              int n_experts, int top_k, float* weights, int* offsets, int* src_token, int* inv_perm,
+                              int* active, int n_slots, void* stream)
+{
+    if (n_tokens <= 0 || n_tables <= 0) return FX_OK;
+    if (top_k <= 0 || top_k > n_experts || n_experts > SCAN_MAX_EXPERTS || vocab <= 0 || n_tables > 65535) return FX_ERR_SIZE;
+    int nt = 64;
+    while (nt < n_tokens * (long)top_k && nt < 1024) nt <<= 1;
+    fx_launch_pdl(route_table_kernel, n_tables, nt, 2 * (size_t)n_experts * sizeof(int), (cudaStream_t)stream, token_ids, tables,
+                  vocab, n_tokens, n_experts, top_k, weights, offsets, src_token, inv_perm, active, n_slots);
+    return fx_launch_status();
+}
 
 static RouteExtra route_extra(const float* choice_bias, float weight_scale, float renorm_eps)
 {

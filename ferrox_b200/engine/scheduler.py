@@ -125,10 +125,10 @@ class Scheduler:
         worst = len(prompt) + max(0, max_new - 1)
         need = (worst + self.cache.page_size - 1) // self.cache.page_size
         for key, g in self.cache.groups.items():
-            # a windowed group holds at most the window plus the pages of one portion
+            # a windowed group holds at most the window plus the pages of one portion (a chunked group: its chunk)
             ps = self.cache.page_size
-            floor = need if g.window is None else min(
-                need, (g.window + ps - 1) // ps + 2 + (g.keep_first + ps - 1) // ps)
+            reach = g.window if g.window is not None else g.chunk
+            floor = need if reach is None else min(need, (reach + ps - 1) // ps + 2 + (g.keep_first + ps - 1) // ps)
             if floor > g.pool.n_pages:
                 raise AdmissionError(
                     f"request of up to {worst} positions needs {floor} pages, the pool has {g.pool.n_pages}")

@@ -37,6 +37,7 @@ _SIGNATURES = {
     "fx_set_scan_lanes": [_I],
     "fx_gemm": [_P, _I, _L, _P, _P, _I, _L, _P, _I, _P, _I, _L, _I, _I, _I, _I, _P, _I, _L, _P],
     "fx_embed": [_P, _I, _P, _P, _I, _I, _I, _P, _F, _P],
+    "fx_embed_norm": [_P, _I, _P, _P, _I, _F, _P, _I, _I, _I, _P, _P],
     "fx_scaled_add_norm": [_P, _P, _F, _P, _I, _F, _P, _I, _I, _I, _P],
     "fx_rmsnorm": [_P, _P, _P, _I, _F, _P, _I, _I, _I, _P],
     "fx_silu_mul": [_P, _L, _P, _L, _I, _P, _I, _I, _P],
@@ -49,10 +50,13 @@ _SIGNATURES = {
     "fx_gather_rows": [_P, _L, _P, _P, _L, _I, _I, _I, _P],
     "fx_gather_rows_scaled": [_P, _L, _P, _P, _P, _I, _P, _L, _I, _I, _I, _P],
     "fx_paged_attention_ex": [_P, _L, _L, _P, _P, _L, _L, _I, _P, _I, _I, _P, _P, _P, _P, _L, _L, _I, _I, _I, _I, _I, _I, _F,
-                              _F, _P, _I, _P, _I, _P],
+                              _F, _P, _I, _P, _I, _I, _P, _L, _P],
     "fx_general_attention_ok": [_I, _I, _I],
     "fx_general_attention": [_P, _L, _L, _P, _P, _L, _L, _P, _P, _I, _I, _P, _P, _P, _P, _I, _P, _L, _L, _I, _I, _I, _I, _I,
-                             _F, _P, _I, _P, _P, _I, _F, _P, _I, _P],
+                             _F, _P, _I, _P, _P, _I, _F, _P, _I, _I, _P, _L, _P],
+    "fx_rotary_mix_store": [_P, _I, _L, _P, _P, _P, _P, _I, _I, _P, _L, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "fx_route_table": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _I, _P],
+    "fx_rmsnorm_residual": [_P, _P, _I, _P, _P, _I, _P, _P, _L, _P, _I, _F, _P, _I, _F, _P, _I, _I, _I, _P],
     "fx_qk_norm_store": [_P, _I, _L, _P, _P, _P, _P, _P, _I, _F, _F, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _F,
                          _P],
     "fx_latent_prep": [_P, _L, _P, _L, _I, _P, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P,
@@ -303,6 +307,14 @@ def embed(table, ids, out, status=None, stream=None, scale=1.0):
     return out
 
 
+def embed_norm(table, ids, weight, eps, out, status=None, stream=None):
+    """out[t] = z / sqrt(mean(z^2) + eps) * weight with z = table[ids[t]], in 32 bits."""
+    T = ids.numel()
+    call("fx_embed_norm", _ptr(table), code(table), _ptr(ids), _ptr(weight), code(weight), float(eps), _ptr(out), T,
+         table.shape[1], table.shape[0], _ptr(status), stream if stream is not None else stream_ptr())
+    return out
+
+
 def scaled_add_norm(h, y, scale, norm=None, stream=None):
     """h += scale * y over the 32-bit rows of the residual stream; ``norm`` = (weight, eps, out): also out = h /
     sqrt(mean(h^2) + eps) * weight on the new rows, in the same kernel.  Returns ``out`` (None without a norm)."""
@@ -324,7 +336,7 @@ def rmsnorm(x, weight, eps, out, rows=None, stream=None):
     return out
 
 
-GATE_ACTIVATIONS = {"silu": 0, "relu": 1, "clamped_swish": 2}   # what a gated feed-forward passes its gate through
+GATE_ACTIVATIONS = {"silu": 0, "relu": 1, "clamped_swish": 2, "gelu_tanh": 3}   # what a gated feed-forward passes its gate through
 
 
 UNARY_ACTIVATIONS = {"relu_square": 1}     # what a plain product's result may pass through in the kernel's epilogue
@@ -362,8 +374,8 @@ def gate_code(activation) -> int:
 
 
 def _gate_args(gated):
-    """The kernels' (gated, act_limit, act_alpha): ``gated`` is 0 / False (plain), 1 / True (SiLU gate), 2 (ReLU gate)
-    or (3, limit, alpha) (the clamped unit)."""
+    """The kernels' (gated, act_limit, act_alpha): ``gated`` is 0 / False (plain), 1 / True (SiLU gate), 2 (ReLU gate),
+    4 (the tanh form of GELU) or (3, limit, alpha) (the clamped unit)."""
     if isinstance(gated, tuple):
         return int(gated[0]), float(gated[1]), float(gated[2])
     return int(gated), 0.0, 0.0
@@ -409,6 +421,37 @@ def layernorm_residual(h, y, weight, eps, *, scale=1.0, y2=None, scale2=1.0, the
     call("fx_layernorm_residual", _ptr(h), _ptr(y), code(y), float(scale), _ptr(y2), code(y2) if y2 is not None else 0,
          float(scale2), _ptr(weight), code(weight), float(eps), _ptr(wn), code(wn) if wn is not None else 0, float(en),
          _ptr(out), code(out) if out is not None else 0, T, H, stream if stream is not None else stream_ptr())
+    return out
+
+
+def rmsnorm_residual_ok(h) -> bool:
+    """Whether :func:`rmsnorm_residual` holds rows of this width in registers."""
+    H = h.shape[1]
+    return H <= (16384 if H % 8 == 0 else 8192)
+
+
+def rmsnorm_residual(h, y, weight, eps, *, then=None, expert_rows=None, stream=None):
+    """h += z / sqrt(mean(z^2) + eps) * weight over whole rows, z = ``y`` [T, hidden].  ``then`` = (weight, eps, out):
+    also out = h / sqrt(mean(h^2) + eps) * weight on the new rows, in the same kernel; returned.  ``expert_rows`` =
+    (inv_perm [T, top_k], weights [T, top_k] or None, shared [T, hidden] or None, its gate's logits or None): ``y``
+    holds the rows of the tokens' experts in expert order and z is what :func:`moe_combine` would add to the stream."""
+    T, H = h.shape
+    if h.dtype != torch.float32 or not h.is_contiguous() or not y.is_contiguous() or y.shape[-1] != H:
+        raise KernelError("rmsnorm_residual: a contiguous 32-bit stream and contiguous rows of its width")
+    place = wts = shared = gate = None
+    top_k = 0
+    if expert_rows is not None:
+        place, wts, shared, gate = expert_rows
+        top_k = place.numel() // T
+        if shared is not None and shared.dtype != y.dtype:
+            raise KernelError("rmsnorm_residual: the shared expert's rows have the experts' element type")
+    elif y.shape != h.shape:
+        raise KernelError("rmsnorm_residual: the sublayer's output has the stream's shape")
+    wn, en, out = then if then is not None else (None, 0.0, None)
+    call("fx_rmsnorm_residual", _ptr(h), _ptr(y), code(y), _ptr(place), _ptr(wts), top_k, _ptr(shared), _ptr(gate),
+         gate.stride(0) if gate is not None else 0, _ptr(weight), code(weight), float(eps), _ptr(wn),
+         code(wn) if wn is not None else 0, float(en), _ptr(out), code(out) if out is not None else 0, T, H,
+         stream if stream is not None else stream_ptr())
     return out
 
 
@@ -668,6 +711,21 @@ def route(logits, top_k, renorm, ids, weights, scratch, offsets, src_token, inv_
          *_route_extra(extra), stream if stream is not None else stream_ptr())
 
 
+ROUTE_TABLE_MAX_EXPERTS = 4096
+
+
+def route_table(token_ids, tables, n_tables, vocab, n_experts, top_k, weights, offsets, src_token, inv_perm, active=None,
+                stream=None):
+    """Routing by a table of token ids, for ``n_tables`` layers in one launch: ``tables`` int64 [n_tables] on the
+    device, the addresses of int32 tables [vocab, top_k].  Fills ``offsets`` [n_tables, n_experts + 1], ``src_token``
+    and ``inv_perm`` [n_tables, T * top_k], ``active`` [n_tables, slots] (None: not wanted) as :func:`moe_align` does
+    for one layer, and ``weights`` [T, top_k] with 1 / top_k."""
+    T = token_ids.numel()
+    call("fx_route_table", _ptr(token_ids), _ptr(tables), int(n_tables), int(vocab), T, int(n_experts), int(top_k),
+         _ptr(weights), _ptr(offsets), _ptr(src_token), _ptr(inv_perm), _ptr(active),
+         active.shape[1] if active is not None else 0, stream if stream is not None else stream_ptr())
+
+
 PAIR_HALVES, PAIR_ADJACENT = 0, 1
 ATTENTION_MAX_KEY_DIM, ATTENTION_MAX_VALUE_DIM = 640, 512    # what the general attention kernels hold of a row
 
@@ -699,7 +757,7 @@ def paged_attention(q, k_pages, v_pages, block_table, page_size, positions, toke
 
 def paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, page_size, positions, token_seq, seq_slot,
                        out, ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim, window, scale, softcap=None, slopes=None,
-                       stream=None, keep_first=0, sinks=None, value_share=1):
+                       stream=None, keep_first=0, sinks=None, value_share=1, chunk=None, gate=None):
     """:func:`paged_attention` in its general form: keys of ``key_dim`` and values of ``value_dim`` elements whose
     positions lie ``ldk`` / ``ldv`` elements apart in their pages (values that are the leading part of the cached
     key rows: the same tensor twice with ldv = ldk); ``q`` and ``out`` are any tensors addressed by a token stride
@@ -707,8 +765,12 @@ def paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pa
     for the query at position i; ``keep_first`` (with a window): the request's first positions stay visible beside
     the window; ``sinks`` (float32 [n_heads], optional): exp(sinks[h]) joins the softmax's denominator once;
     ``value_share``: that many consecutive key heads read one value head (the value pages hold n_kv_heads /
-    value_share heads)."""
+    value_share heads); ``chunk``: a query sees the keys of its own chunk of that many positions only, counted from
+    the request's start; ``gate`` (token rows of n_heads * value_dim, of q's element type, optional): the result is
+    multiplied by sigmoid(gate)."""
     T = positions.numel()
+    if gate is not None and gate.dtype != q.dtype:
+        raise KernelError("paged_attention_ex: the gate has the queries' element type")
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != n_heads):
         raise KernelError("paged_attention_ex: one 32-bit slope per head")
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads):
@@ -716,8 +778,8 @@ def paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pa
     call("fx_paged_attention_ex", _ptr(q), int(ldq), int(ldqh), _ptr(k_pages), _ptr(v_pages), int(ldk), int(ldv), code(q),
          _ptr(block_table), block_table.shape[1], page_size, _ptr(positions), _ptr(token_seq), _ptr(seq_slot), _ptr(out),
          int(ldo), int(ldoh), T, n_heads, n_kv_heads, key_dim, value_dim, int(window or 0), float(scale),
-         float(softcap or 0.0), _ptr(slopes), int(keep_first or 0), _ptr(sinks), int(value_share),
-         stream if stream is not None else stream_ptr())
+         float(softcap or 0.0), _ptr(slopes), int(keep_first or 0), _ptr(sinks), int(value_share), int(chunk or 0),
+         _ptr(gate), _rows(gate) if gate is not None else 0, stream if stream is not None else stream_ptr())
     return out
 
 
@@ -768,7 +830,7 @@ def general_attention_items(entries, n_heads: int, n_kv_heads: int):
 def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, page_size, positions, token_seq, seq_slot,
                       items, out, ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim, window, scale, slopes=None,
                       stream=None, n_splits=1, part_o=None, part_ml=None, kv_strides=None, keep_first=0, softcap=None,
-                      sinks=None, value_share=1):
+                      sinks=None, value_share=1, chunk=None, gate=None):
     """:func:`paged_attention_ex` in bfloat16 on the tensor cores (see :func:`general_attention_ok`).  ``items``: the
     device copy of :func:`general_attention_items`, or None when every entry brings one token (a tile a token and
     kv head; nothing comes from the host, so a captured step replays unchanged).  ``n_splits`` > 1 (without items):
@@ -776,7 +838,10 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pag
     value_dim] and ``part_ml`` float32 [T, heads, n_splits, 2] are scratch, and a second kernel adds the runs up.
     ``kv_strides`` = (k page stride, k head stride, v page stride, v head stride) in elements, for keys and values that
     do not lie [page][kv head][position][ld] (rows that hold all heads side by side); ``ldk`` / ``ldv`` stay the
-    distance between two positions.  ``softcap``, ``sinks``, ``value_share``: as :func:`paged_attention_ex`."""
+    distance between two positions.  ``softcap``, ``sinks``, ``value_share``, ``chunk``, ``gate``: as
+    :func:`paged_attention_ex`."""
+    if gate is not None and gate.dtype != q.dtype:
+        raise KernelError("general_attention: the gate has the queries' element type")
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads):
         raise KernelError("general_attention: one 32-bit sink per head")
     strides = (ctypes.c_long * 4)(*[int(x) for x in kv_strides]) if kv_strides is not None else None
@@ -788,7 +853,8 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pag
          ctypes.cast(strides, c_void_p) if strides is not None else None, _ptr(block_table), block_table.shape[1], page_size, _ptr(positions), _ptr(token_seq), _ptr(seq_slot),
          _ptr(items), n, _ptr(out), int(ldo), int(ldoh), n_heads, n_kv_heads, key_dim, value_dim, int(window or 0),
          float(scale), _ptr(slopes), int(n_splits), _ptr(part_o), _ptr(part_ml), int(keep_first or 0),
-         float(softcap or 0.0), _ptr(sinks), int(value_share), stream if stream is not None else stream_ptr())
+         float(softcap or 0.0), _ptr(sinks), int(value_share), int(chunk or 0), _ptr(gate),
+         _rows(gate) if gate is not None else 0, stream if stream is not None else stream_ptr())
     return out
 
 
@@ -808,6 +874,22 @@ def qk_norm_store(qkv, positions, token_seq, seq_slot, q_weight, k_weight, eps, 
          _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], page_size, qkv.shape[0], n_heads,
          n_kv_heads, key_dim, value_dim, int(write_cache), _ptr(status),
          float(value_norm_eps) if value_norm_eps is not None else -1.0, stream if stream is not None else stream_ptr())
+
+
+def rotary_mix_store(qkv, positions, token_seq, seq_slot, cos_sin, rot_dims, pairing, k_pages, v_pages, block_table,
+                     page_size, n_heads, n_kv_heads, key_dim, value_dim, v_first=None, lam=0.0, write_cache=True,
+                     status=None, stream=None):
+    """Rows of [q heads | k heads | v heads] (widths key_dim, key_dim, value_dim): the first ``rot_dims`` elements of
+    every q head (in place) and k head (into its page) turned by ``cos_sin`` [T, rot_dims / 2, 2] (None: no rotation),
+    the values into their pages, mixed on the way with those of another layer where ``v_first`` (row views [T, kv heads
+    * value_dim]) is given: (1 - lam) v + lam v_first.  The rows' own v stays as projected."""
+    if v_first is not None and (v_first.dtype != qkv.dtype or v_first.shape != (qkv.shape[0], n_kv_heads * value_dim)):
+        raise KernelError("rotary_mix_store: the other layer's values have the shape and element type of this one's")
+    call("fx_rotary_mix_store", _ptr(qkv), code(qkv), _rows(qkv), _ptr(positions), _ptr(token_seq), _ptr(seq_slot),
+         _ptr(cos_sin), int(rot_dims), int(pairing), _ptr(v_first), _rows(v_first) if v_first is not None else 0,
+         float(lam), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], page_size, qkv.shape[0],
+         n_heads, n_kv_heads, key_dim, value_dim, int(write_cache), _ptr(status),
+         stream if stream is not None else stream_ptr())
 
 
 def latent_prep(q, dkv, positions, token_seq, seq_slot, c_weight, eps, cos_sin, rot_dims, q_plain, q_full, pages,
@@ -1312,10 +1394,10 @@ def linear(x, w, out, *, bias=None, accumulate=False, status=None, stream=None, 
 
 def gated_linear(x, w_gu, out, *, status=None, stream=None, activation="silu", bias=None):
     """out = act(x . gate^T (+ b_gate)) * (x . up^T (+ b_up)) with ``w_gu`` = [gate rows ; up rows], ``bias`` =
-    [b_gate ; b_up] or None, and act SiLU or ReLU (``activation``): picks the kernel as :func:`linear` does; the
+    [b_gate ; b_up] or None, and act one of GATE_ACTIVATIONS (``activation``): picks the kernel as :func:`linear` does; the
     gate|up intermediate reaches memory only on the CUDA-core path."""
     T, I = out.shape
-    gated = gated_arg(activation)     # the kernels' argument: 0 plain, 1 SiLU gate, 2 ReLU gate, (3, limit, alpha)
+    gated = gated_arg(activation)     # the kernels' argument: see _gate_args
     if bias is not None and bias.numel() != 2 * I:
         raise KernelError("gated_linear: the bias holds the gate rows' values, then the up rows'")
     if T <= SKINNY_MAX_TOKENS and tc_ok(x, w_gu) and swap_better(T, 2 * I, x.shape[1]):

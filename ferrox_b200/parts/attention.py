@@ -94,17 +94,29 @@ class GqaAttention(Mixer):
         self.value_norm_eps = getattr(s, "value_norm_eps", None)
         self.keep_first = int(getattr(s, "keep_first", 0) or 0) if s.window is not None else 0
         self.gate_name = getattr(s, "output_gate", None)
+        self.chunk = getattr(s, "chunk", None)
+        self.sink_name = getattr(s, "sink", None)
+        self.mix = getattr(s, "value_mix", None)
+        if self.chunk is not None and (self.chunk < 1 or s.window is not None):
+            raise ValueError(f"chunk={self.chunk}: a positive number of positions, without a window")
         if int(getattr(s, "keep_first", 0) or 0) < 0:
             raise ValueError(f"keep_first={s.keep_first}: a number of positions")
-        self.general = bool(self.qk_norm or self.temperature or self.slopes_spec or self.value_dim != s.head_dim
-                            or self.value_norm_eps is not None or self.keep_first or self.gate_name)
+        prepared = bool(self.qk_norm or self.temperature or self.value_norm_eps is not None)    # by qk_norm_store
+        self.general = bool(prepared or self.slopes_spec or self.value_dim != s.head_dim or self.keep_first
+                            or self.gate_name or self.chunk or self.sink_name or self.mix)
+        # in the general form a rotary part's tables serve the kernel that also mixes the values (rotary_mix_store)
+        self.rotates = self.general and s.position is not None and not isinstance(s.position, NoPositionSpec)
         self.v_size = s.n_kv_heads * self.value_dim
         self.o_size = s.n_heads * self.value_dim
         if self.general:
-            if s.position is not None and not isinstance(s.position, NoPositionSpec):
-                raise ValueError("attention with normed queries, keys or values, a query temperature, a distance bias, "
-                                 "kept first positions, an output gate or its own value width takes no rotary "
-                                 "position encoding")
+            if prepared and (self.rotates or self.mix):
+                raise ValueError("attention with normed queries, keys or values or a query temperature takes no rotary "
+                                 "position encoding and no mixing of values")
+            if self.rotates and not hasattr(self.position, "table"):
+                raise ValueError("the general attention form rotates by a table of cos and sin: a rotary position part "
+                                 "or none")
+            if self.rotates and s.position.rotary_dim > s.head_dim:
+                raise ValueError(f"rotary_dim={s.position.rotary_dim} exceeds head_dim={s.head_dim}")
             if s.tied_values or s.softcap:
                 raise ValueError("the general attention form has neither tied values nor a soft cap")
             if self.slopes_spec is not None and len(self.slopes_spec) != s.n_heads:
@@ -128,8 +140,8 @@ class GqaAttention(Mixer):
         if self.value_dim != s.head_dim:
             return CacheSpec(paged=PagedSpec((PagedTensorSpec("k", (s.n_kv_heads, s.head_dim), lead_dims=1),
                                               PagedTensorSpec("v", (s.n_kv_heads, self.value_dim), lead_dims=1)), s.window,
-                                             self.keep_first))
-        return CacheSpec(paged=KvCacheSpec(s.n_kv_heads, s.head_dim, s.window, self.keep_first))
+                                             self.keep_first, self.chunk))
+        return CacheSpec(paged=KvCacheSpec(s.n_kv_heads, s.head_dim, s.window, self.keep_first, self.chunk))
 
     def tensor_decls(self):
         s, n = self.spec, self._names
@@ -144,6 +156,10 @@ class GqaAttention(Mixer):
             d += [TensorDecl(n[key + "_bias"], (sizes[key],)) for key in keys]
         if self.gate_name:
             d.append(TensorDecl(s.prefix + self.gate_name, (self.o_size, s.hidden)))
+        if self.sink_name:
+            d.append(TensorDecl(s.prefix + self.sink_name, (s.n_heads,)))
+        if self.mix:
+            d.append(TensorDecl(s.prefix + self.mix.name, (), optional=self.mix.source))
         return d
 
     def load(self, src, rt):
@@ -171,6 +187,10 @@ class GqaAttention(Mixer):
             self.q_norm_w, self.k_norm_w = (w.to(dt).contiguous() for w in ws)
         if self.slopes_spec is not None:
             self.slopes = torch.tensor([float(x) for x in self.slopes_spec], dtype=torch.float32, device=rt.device)
+        self.sinks = src.get(self.spec.prefix + self.sink_name).to(torch.float32).contiguous() if self.sink_name else None
+        self.lam = 0.0
+        if self.mix and not self.mix.source:
+            self.lam = float(src.get(self.spec.prefix + self.mix.name).to(torch.float32))
         # zeroed scratch of the decode attention kernel that merges its own key ranges (it leaves it zeroed)
         self._range_counters = (torch.zeros(RANGE_COUNTERS, dtype=torch.int32, device=rt.device)
                                 if rt.device.type == "cuda" else None)
@@ -263,36 +283,58 @@ class GqaAttention(Mixer):
 
     def _forward_general(self, x, out, batch, cache, accumulate):
         """The form with normed queries, keys or values, a query temperature, a distance bias, kept first positions,
-        an output gate, values of their own width: fused [q | k | v (| gate)] product; one kernel norms q and k (and
-        v) per head, applies the temperature and stores k and v; attention with the bias and the mask; the gate;
+        chunks, sinks, an output gate, values of their own width or mixed across layers: fused [q | k | v (| gate)]
+        product; one kernel norms q and k (and v) per head, applies the temperature and stores k and v, or rotates q
+        and k, mixes v and stores k and v; attention with the bias and the mask, whose epilogue applies the gate;
         output product."""
         s = self.spec
         T, D, V = x.shape[0], s.head_dim, self.value_dim
         qkv_width = self.q_size + self.kv_size + self.v_size
         qkv = self.rt.empty(T, qkv_width + (self.o_size if self.gate_name else 0))
         ops.linear(x, self.w_qkv, qkv, bias=self.b_qkv, status=batch.status, stream=batch.stream, after_short_kernel=True)
-        eps = self.qk_norm[2] if self.qk_norm else 0.0
-        ops.qk_norm_store(qkv, batch.positions, batch.token_seq, batch.seq_slot, self.q_norm_w, self.k_norm_w, eps,
-                          self.temperature, cache.k, cache.v, cache.block_table, cache.page_size, s.n_heads, s.n_kv_heads,
-                          D, V, write_cache=cache.writes, status=batch.status, stream=batch.stream,
-                          value_norm_eps=self.value_norm_eps)
+        if self.rotates or self.mix:
+            first = self._values_of_first_layer(qkv, qkv_width, batch)
+            ops.rotary_mix_store(qkv, batch.positions, batch.token_seq, batch.seq_slot,
+                                 self.position.table(batch) if self.rotates else None,
+                                 self.position.rotary_dim if self.rotates else 0,
+                                 self.position.pairing if self.rotates else ops.PAIR_HALVES, cache.k, cache.v,
+                                 cache.block_table, cache.page_size, s.n_heads, s.n_kv_heads, D, V, v_first=first,
+                                 lam=self.lam, write_cache=cache.writes, status=batch.status, stream=batch.stream)
+        else:
+            eps = self.qk_norm[2] if self.qk_norm else 0.0
+            ops.qk_norm_store(qkv, batch.positions, batch.token_seq, batch.seq_slot, self.q_norm_w, self.k_norm_w, eps,
+                              self.temperature, cache.k, cache.v, cache.block_table, cache.page_size, s.n_heads,
+                              s.n_kv_heads, D, V, write_cache=cache.writes, status=batch.status, stream=batch.stream,
+                              value_norm_eps=self.value_norm_eps)
         attn = self.rt.empty(T, self.o_size)
         general_attention(qkv, qkv.stride(0), D, cache.k, cache.v, D, V, attn, attn.stride(0), V, batch, cache,
                           s.n_heads, s.n_kv_heads, D, V, s.window, self.scale, self.slopes, self.rt,
-                          keep_first=self.keep_first)
-        if self.gate_name:
-            ops.gate_heads_(attn, qkv[:, qkv_width:], s.n_heads, stream=batch.stream)
+                          keep_first=self.keep_first, sinks=self.sinks, chunk=self.chunk,
+                          gate=qkv[:, qkv_width:] if self.gate_name else None)
         ops.linear(attn, self.w_o, out, accumulate=accumulate, status=batch.status, stream=batch.stream,
                    after_short_kernel=True)
+
+    def _values_of_first_layer(self, qkv, qkv_width, batch):
+        """The step's rows of v_first for a layer that mixes its values with them (None for any other).  The source
+        layer's own rows of its fused product stay as projected: it leaves a view of them for the layers behind it."""
+        if not self.mix:
+            return None
+        key = ("values of the first layer", self.mix.group)
+        if self.mix.source:
+            batch.shared[key] = qkv[:, qkv_width - self.v_size:qkv_width]
+            return None
+        if key not in batch.shared:
+            raise RuntimeError(f"no layer before this one left its values for the group {self.mix.group!r}")
+        return batch.shared[key]
 
 
 def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, batch, cache, n_heads, n_kv_heads,
                       key_dim, value_dim, window, scale, slopes, rt, keep_first=0, softcap=None, sinks=None,
-                      value_share=1):
+                      value_share=1, chunk=None, gate=None):
     """Attention over pages in its general form (keys and values of different widths, strided queries and outputs, an
-    optional distance bias, a window that may keep the request's first positions visible, capped scores, a learned
-    number per head in the softmax's denominator, key heads that share value heads), by the kernel that fits
-    the step: tiles of (token, head) pairs on the tensor cores
+    optional distance bias, a window that may keep the request's first positions visible, chunks, capped scores, a
+    learned number per head in the softmax's denominator, key heads that share value heads, a result multiplied by the
+    sigmoid of a gate), by the kernel that fits the step: tiles of (token, head) pairs on the tensor cores
     in bfloat16, a warp per (token, head) on the CUDA cores in 32-bit and for widths that are no multiple of 16."""
     per_sm = ops.general_attention_ok(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, key_dim, value_dim)
     if per_sm:
@@ -305,6 +347,8 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, 
             reach = cache.block_table.shape[1] * cache.page_size
             if window is not None:
                 reach = min(reach, (window + 63) // 64 * 64 + 64 + (keep_first + 63) // 64 * 64)
+            if chunk is not None:
+                reach = min(reach, (chunk + 63) // 64 * 64 + 64)
             _, n_splits = ops.decode_split_plan(T, tiles, reach, per_sm, single_is_final=True)
             if n_splits > 1:
                 part_o = rt.empty(T, n_heads, n_splits, value_dim, dtype=torch.float32)
@@ -320,11 +364,11 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, 
                                      batch.positions, batch.token_seq, batch.seq_slot, items, out, ldo, ldoh, n_heads,
                                      n_kv_heads, key_dim, value_dim, window, scale, slopes=slopes, stream=batch.stream,
                                      n_splits=n_splits, part_o=part_o, part_ml=part_ml, keep_first=keep_first,
-                                     softcap=softcap, sinks=sinks, value_share=value_share)
+                                     softcap=softcap, sinks=sinks, value_share=value_share, chunk=chunk, gate=gate)
     ops.paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, cache.block_table, cache.page_size, batch.positions,
                            batch.token_seq, batch.seq_slot, out, ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim,
                            window, scale, slopes=slopes, stream=batch.stream, keep_first=keep_first, softcap=softcap,
-                           sinks=sinks, value_share=value_share)
+                           sinks=sinks, value_share=value_share, chunk=chunk, gate=gate)
 
 
 class DifferentialAttention(Mixer):

@@ -45,6 +45,7 @@ class Runtime:
         self._kept = []          # buffers of the last small step, in the order they were asked for
         self._next = -1          # index of the next request; -1: buffers are not kept
         self._kept_bytes = 0
+        self.groups = {}         # what parts of one kind share across a model, under keys of their own choosing
 
     def begin_step(self, n_tokens: int) -> None:
         """An eager step begins (never inside a graph capture: a graph owns its memory)."""
@@ -139,6 +140,12 @@ class FeedForward(Part):
     # ``forward_add(x, h, batch, then_norm=norm)``: it returns that norm's output on the new ``h``, or None if it
     # left the norm to the caller.  Parts without the flag are never given the argument.
     fuses_norm = False
+
+    # A feed-forward whose last kernel can also apply an RMS norm to its own result, add that to the stream and apply the
+    # norm that follows (``post`` and ``then_norm``: norms with ``as_rms()``) sets ``fuses_post_norm`` and has
+    # ``forward_post(x, h, batch, post, then_norm)``: h += post(ffn(x)); returns then_norm's output on the new ``h``, or
+    # None if it left that norm to the caller.
+    fuses_post_norm = False
 
     def forward_add(self, x, h, batch) -> None:  # pragma: no cover - interface
         raise NotImplementedError

@@ -145,9 +145,10 @@ class SandwichNormBlock(Block):
         h += post1(mixer(norm1(h)));   h += post2(ffn(norm2(h)))
 
     (``ffn`` None: the layer ends after the mixer).  The sublayer's output is a 32-bit buffer; one kernel norms it,
-    adds it to the stream and, where the norm that comes next is a layer norm too, applies that to the new row as
-    well (the mixer's post-norm with norm2, the feed-forward's post-norm with the next block's norm1).  A mixer
-    that is a weighted sum of mixers hands its parts over, and the same kernel takes the sum."""
+    adds it to the stream and, where the norm that comes next is of the same kind (layer norms or RMS norms), applies
+    that to the new row as well (the mixer's post-norm with norm2, the feed-forward's post-norm with the next block's
+    norm1).  A mixer that is a weighted sum of mixers hands its parts over, and the layer norms' kernel takes the sum;
+    experts hand their rows over, and the RMS norms' kernel adds a token's rows up (``fuses_post_norm``)."""
 
     passes_norm = True
 
@@ -165,7 +166,10 @@ class SandwichNormBlock(Block):
         return [p for p in (self.norm1, self.mixer, self.post1, self.norm2, self.ffn, self.post2) if p is not None]
 
     def tensor_decls(self):
-        return [d for p in self._parts() for d in p.tensor_decls()]
+        from ..weights.loader import TensorDecl
+
+        d = [x for p in self._parts() for x in p.tensor_decls()]
+        return d + [TensorDecl(n, tuple(shape), optional=True) for n, shape in getattr(self.spec, "unused_tensors", ())]
 
     def load(self, src, rt):
         super().load(src, rt)
@@ -191,6 +195,11 @@ class SandwichNormBlock(Block):
                 then = (nxt[0], nxt[1], self.rt.empty(h.shape[0], h.shape[1]))
             return ops.layernorm_residual(h, y, ln[0], ln[1], scale=sc, y2=y2, scale2=sc2, then=then,
                                           stream=batch.stream)
+        rms = post.as_rms()
+        if rms is not None and len(outs) == 1 and outs[0][1] == 1.0 and ops.rmsnorm_residual_ok(h):
+            nxt = then_norm.as_rms() if then_norm is not None else None
+            then = (nxt[0], nxt[1], self.rt.empty(h.shape[0], h.shape[1])) if nxt is not None else None
+            return ops.rmsnorm_residual(h, outs[0][0], rms[0], rms[1], then=then, stream=batch.stream)
         # any other norm: sum the parts, norm the sum as a stream of its own, add
         total = outs[0][0]
         if outs[0][1] != 1.0:
@@ -221,6 +230,8 @@ class SandwichNormBlock(Block):
             with ops.trace_scope("norm"):
                 x2 = self.norm2.forward(h)
         with ops.trace_scope("feed-forward"):
+            if self.ffn.fuses_post_norm and self.post2.as_rms() is not None and ops.rmsnorm_residual_ok(h):
+                return self.ffn.forward_post(x2, h, batch, self.post2, then_norm)
             y = self.rt.empty(h.shape[0], h.shape[1], dtype=torch.float32)
             self.ffn.forward_into(x2, y, batch, accumulate=False)
         with ops.trace_scope("norm"):

@@ -16,7 +16,8 @@ def pack_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 
 class SwigluMlp(FeedForward):
-    """down( act(gate x) * (up x) ); ``spec.activation`` names act (SiLU unless the spec says ReLU).  With
+    """down( act(gate x) * (up x) ); ``spec.activation`` names act (SiLU unless the spec says ReLU or the
+    tanh form of GELU).  With
     ``spec.bias_names`` every projection has a bias: down( act(gate x + bg) * (up x + bu) ) + bd; the products'
     epilogues add them."""
 

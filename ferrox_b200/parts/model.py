@@ -104,14 +104,19 @@ class DecoderModel(Part):
         s, rt = self.spec, self.rt
         h = rt.empty(batch.n_tokens, s.hidden, dtype=torch.float32)
         with ops.trace_scope("embedding"):
-            if self.position_table is not None:
+            rms = self.embedding_norm.as_rms() if self.embedding_norm is not None else None
+            fused = rms is not None and self.position_table is None and getattr(s, "embedding_scale", 1.0) == 1.0
+            if fused:
+                # rows looked up and RMS-normed in one kernel
+                ops.embed_norm(self.embedding, batch.token_ids, rms[0], rms[1], h, status=batch.status, stream=batch.stream)
+            elif self.position_table is not None:
                 # a learned position vector is added to every embedding row, in 32 bits
                 ops.embed_pos(self.embedding, batch.token_ids, self.position_table, batch.positions, h,
                               status=batch.status, stream=batch.stream)
             else:
                 ops.embed(self.embedding, batch.token_ids, h, status=batch.status, stream=batch.stream,
                           scale=float(getattr(s, "embedding_scale", 1.0)))
-            if self.embedding_norm is not None:
+            if self.embedding_norm is not None and not fused:
                 self.embedding_norm.forward_in_place(h)
         x = None    # the next block's first norm of h, when the block before it has computed it
         for i, entry in enumerate(s.schedule):

@@ -14,6 +14,9 @@ products' epilogues apply act); ``choice_bias`` (a number per expert added to th
 the weights use the scores without it), ``weight_scale`` (a factor on the final weights) and ``renorm_eps`` (added to
 the sum the kept scores are divided by).
 
+``table``: no router at all.  An integer table names every token id's experts, each with weight 1/top_k; the choice
+depends on the step's token ids alone, so the first such layer of a step sorts the tokens of all of them, in one launch.
+
 Reference: router crates/ferrox-moe/src/lib.rs:333-355, expert :619-659, combine
 :735-752, shared expert and its sigmoid gate crates/ferrox-models/src/decoder.rs:
 2660-2681 and (batched) :1037-1093; tokens bucketed by expert :2792-2890.
@@ -26,7 +29,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from ..weights.loader import TensorDecl
+from ..weights.loader import TensorDecl, WeightsError
 from .base import FeedForward, register_part
 from .mlp import pack_gate_up
 
@@ -54,10 +57,19 @@ def expert_tile_tokens(T: int, K: int, E: int):
 class SoftmaxTopkMoe(FeedForward):
     graph_safe = True
     fuses_norm = True
+    fuses_post_norm = True
 
     def __init__(self, spec):
         super().__init__(spec)
         s = spec
+        self.table_name = getattr(s, "table", None)
+        if self.table_name:
+            if s.vocab < 1 or s.n_experts > ops.ROUTE_TABLE_MAX_EXPERTS:
+                raise ValueError(f"an expert table of {s.vocab} token ids over {s.n_experts} experts (at most "
+                                 f"{ops.ROUTE_TABLE_MAX_EXPERTS})")
+            if s.shared_gate or getattr(s, "choice_bias", None) or getattr(s, "weight_on_input", False):
+                raise ValueError("experts chosen by a table take no choice bias, no shared gate and their weight on the "
+                                 "output")
         self.scores = getattr(s, "scores", "softmax")
         if self.scores not in ("softmax", "sigmoid"):
             raise ValueError(f"router scores {self.scores!r}: softmax or sigmoid")
@@ -89,7 +101,10 @@ class SoftmaxTopkMoe(FeedForward):
 
     def tensor_decls(self):
         s, p = self.spec, self.spec.prefix
-        d = [TensorDecl(self._router_name, (s.n_experts, s.hidden))]
+        if self.table_name:
+            d = [TensorDecl(p + self.table_name, (s.vocab, s.top_k), integer=True, below=s.n_experts)]
+        else:
+            d = [TensorDecl(self._router_name, (s.n_experts, s.hidden))]
         shape = lambda part, inner: (s.hidden, inner) if part == "down" else (inner, s.hidden)
         for e in range(s.n_experts):
             d += [TensorDecl(self._expert_name(e, part), shape(part, s.expert_intermediate)) for part in self._parts]
@@ -107,7 +122,10 @@ class SoftmaxTopkMoe(FeedForward):
     def load(self, src, rt):
         super().load(src, rt)
         s, p = self.spec, self.spec.prefix
-        self.w_router = src.get(self._router_name)
+        if self.table_name:
+            self._load_table(src, rt)
+        else:
+            self.w_router = src.get(self._router_name)
         E, I, H = s.n_experts, s.expert_intermediate, s.hidden
         # If any expert tensor is stored in 32 bits, the packed buffers are 32-bit.
         names = [self._expert_name(e, n) for e in range(E) for n in self._parts]
@@ -137,7 +155,7 @@ class SoftmaxTopkMoe(FeedForward):
         scale, eps = float(getattr(s, "weight_scale", 1.0)), float(getattr(s, "renorm_eps", 0.0))
         self._route_extra = (bias, scale, eps) if (bias is not None or scale != 1.0 or eps != 0.0) else None
         # router rows and the shared expert's gate row share one product: [E (+1), H]
-        self.w_route = self.w_router
+        self.w_route = None if self.table_name else self.w_router
         if self.w_shared_gate is not None:
             dtr = torch.float32 if torch.float32 in (self.w_router.dtype, self.w_shared_gate.dtype) else self.w_router.dtype
             self.w_route = torch.cat([self.w_router.to(dtr), self.w_shared_gate.to(dtr)], dim=0).contiguous()
@@ -145,6 +163,41 @@ class SoftmaxTopkMoe(FeedForward):
         if self.w_shared_gu is not None and rt.device.type == "cuda":
             self._side = torch.cuda.Stream(device=rt.device)
             self._fork, self._join = torch.cuda.Event(), torch.cuda.Event()
+
+    def _load_table(self, src, rt):
+        s = self.spec
+        name = s.prefix + self.table_name
+        t = src.get(name).to(torch.int32).contiguous()
+        row = torch.sort(t, dim=1).values
+        if int(t.min()) < 0 or int(t.max()) >= s.n_experts or bool((row[:, 1:] == row[:, :-1]).any()):
+            raise WeightsError(f"{name}: every row names {s.top_k} different experts of {s.n_experts}")
+        # the tables of one model that one launch sorts tokens for: same sizes, in the order in which they were loaded
+        self.table = t
+        self._table_group = rt.groups.setdefault(("expert tables", s.vocab, s.top_k, s.n_experts), [])
+        self._table_index = len(self._table_group)
+        self._table_group.append(t)
+
+    def _route_by_table(self, batch, T, small):
+        """(weights, offsets, src_token, inv_perm, active) of this layer: the step's first layer of the group asks for
+        all of them at once."""
+        s, rt = self.spec, self.rt
+        group = self._table_group
+        key = ("expert tables", s.vocab, s.top_k, s.n_experts)
+        routed = batch.shared.get(key)
+        if routed is None:
+            L, n, i32 = len(group), T * s.top_k, torch.int32
+            ptrs = rt.groups.get(key + ("addresses",))
+            if ptrs is None or ptrs.numel() != L:
+                ptrs = torch.tensor([t.data_ptr() for t in group], dtype=torch.int64, device=rt.device)
+                rt.groups[key + ("addresses",)] = ptrs
+            # (a step's first layer asks for buffers of this order each time: they are kept from step to step)
+            routed = (rt.empty(T, s.top_k, dtype=torch.float32), rt.empty(L, s.n_experts + 1, dtype=i32),
+                      rt.empty(L, n, dtype=i32), rt.empty(L, n, dtype=i32), rt.empty(L, min(s.n_experts, n), dtype=i32))
+            ops.route_table(batch.token_ids, ptrs, L, s.vocab, s.n_experts, s.top_k, *routed, stream=batch.stream)
+            batch.shared[key] = routed
+        w, offsets, src_token, inv_perm, active = routed
+        l = self._table_index
+        return w, offsets[l], src_token[l], inv_perm[l], active[l] if small else None
 
     def _shared_expert(self, x, batch, st):
         """silu(gate) * up, then down, of the expert that every token visits: [T, H]."""
@@ -168,19 +221,43 @@ class SoftmaxTopkMoe(FeedForward):
         return out
 
     def forward_add(self, x, h, batch, then_norm=None):
+        st = batch.stream
+        y, inv_perm, weights, shared, gate_logit = self._expert_rows(x, batch)
+        K = self.spec.top_k
+        # the combination applies the norm that follows it where that is an RMSNorm over rows it can hold
+        rms = then_norm.as_rms() if then_norm is not None else None
+        if rms is not None and ops.combine_norm_ok(h, y):
+            out = self.rt.empty(h.shape[0], h.shape[1])
+            return ops.moe_combine(h, y, inv_perm, weights, shared, gate_logit, stream=st, norm=(rms[0], rms[1], out),
+                                   top_k=K)
+        ops.moe_combine(h, y, inv_perm, weights, shared, gate_logit, stream=st, top_k=K)
+        return None
+
+    def forward_post(self, x, h, batch, post, then_norm=None):
+        """h += post(ffn(x)): one kernel adds a token's expert rows up, norms the sum, adds it to the stream and applies
+        the norm that follows to the new row."""
+        y, inv_perm, weights, shared, gate_logit = self._expert_rows(x, batch)
+        (w, eps), nxt = post.as_rms(), then_norm.as_rms() if then_norm is not None else None
+        then = (nxt[0], nxt[1], self.rt.empty(h.shape[0], h.shape[1])) if nxt is not None else None
+        return ops.rmsnorm_residual(h, y, w, eps, then=then, expert_rows=(inv_perm, weights, shared, gate_logit),
+                                    stream=batch.stream)
+
+    def _expert_rows(self, x, batch):
+        """The experts' results: (rows in expert order [T * K, H], each (token, rank) pair's row, the weights they are
+        added up with (None: as they are), the shared expert's rows or None, its gate's logits or None)."""
         s, rt, st = self.spec, self.rt, batch.stream
         T, E, K, I, H = x.shape[0], s.n_experts, s.top_k, s.expert_intermediate, s.hidden
         i32 = torch.int32
         # A decode step of a few tokens: the router's product, the routing and the rows in expert order come from ONE
         # kernel (three dependent launches otherwise, each a few microseconds of waiting for the one before).
-        fused = ops.route_fused_ok(x, self.w_route, E, K)
+        table = self.table_name is not None
+        fused = not table and ops.route_fused_ok(x, self.w_route, E, K)
         mode, gated, scaled = self._route_mode, self._gated, self.weight_on_input
         unary, extra = self.plain, self._route_extra
         tc = ops.tc_ok(x, self.w_gu) and I % 8 == 0 and E <= ops.TC_MAX_GROUPS
         tiles = expert_tile_tokens(T, K, E) if tc and T >= SWAP_MIN_TOKENS and E <= ops.TC_SWAP_MAX_GROUPS else None
         small = tiles is None and T <= ops.SKINNY_MAX_TOKENS and ops.skinny_ok(x, self.w_gu) and I % 32 == 0
         big = T > ops.SKINNY_MAX_TOKENS and tc
-        n_route = self.w_route.shape[0]      # E router logits, then the shared expert's gate logit if it has one
         # The shared expert's two products run on a second stream beside the routing and the routed experts; both
         # meet again at the combination.  In a decode step the routed experts' kernels leave most of the machine
         # idle; in a prompt the router's short kernels hide under the shared expert's products.  Measured on a
@@ -193,15 +270,21 @@ class SoftmaxTopkMoe(FeedForward):
             self._fork.record(main)          # the shared expert may start from here on
             if not fused:
                 shared = self._shared_on_side(x, batch)
-        logits = rt.empty(T, n_route, dtype=torch.float32)
-        ids = rt.empty(T, K, dtype=i32)
-        weights = rt.empty(T, K, dtype=torch.float32)
-        offsets = rt.empty(E + 1, dtype=i32)
-        src_token = rt.empty(T * K, dtype=i32)
-        inv_perm = rt.empty(T * K, dtype=i32)
-        active = rt.empty(min(E, T * K), dtype=i32) if small else None
+        if table:
+            weights, offsets, src_token, inv_perm, active = self._route_by_table(batch, T, small)
+        else:
+            # E router logits, then the shared expert's gate logit if it has one
+            logits = rt.empty(T, self.w_route.shape[0], dtype=torch.float32)
+            ids = rt.empty(T, K, dtype=i32)
+            weights = rt.empty(T, K, dtype=torch.float32)
+            offsets = rt.empty(E + 1, dtype=i32)
+            src_token = rt.empty(T * K, dtype=i32)
+            inv_perm = rt.empty(T * K, dtype=i32)
+            active = rt.empty(min(E, T * K), dtype=i32) if small else None
         xp = None
-        if fused:
+        if table:
+            pass
+        elif fused:
             # The cluster's kernel goes first: it needs eight free SMs of one GPC at once, which it finds now and would
             # not find once the shared expert's weight-streaming kernels (enqueued right after it, waiting only for what
             # was before it) fill every SM.
@@ -268,14 +351,7 @@ class SoftmaxTopkMoe(FeedForward):
                 shared = self._shared_expert(x, batch, st)
             if self.w_shared_gate is not None:
                 gate_logit = logits[:, E:]      # [T, 1] view with the logits' row stride
-        # the combination applies the norm that follows it where that is an RMSNorm over rows it can hold
-        rms = then_norm.as_rms() if then_norm is not None else None
-        if rms is not None and ops.combine_norm_ok(h, y):
-            out = rt.empty(T, H)
-            return ops.moe_combine(h, y, inv_perm, None if scaled else weights, shared, gate_logit, stream=st,
-                                   norm=(rms[0], rms[1], out), top_k=K)
-        ops.moe_combine(h, y, inv_perm, None if scaled else weights, shared, gate_logit, stream=st, top_k=K)
-        return None
+        return y, inv_perm, None if scaled else weights, shared, gate_logit
 
 
 register_part("softmax_topk_moe", SoftmaxTopkMoe, replace=True)

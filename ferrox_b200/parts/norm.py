@@ -11,7 +11,8 @@ from .base import Norm, register_part
 
 class RmsNorm(Norm):
     """``one_plus``: the stored weight lies around zero and the norm multiplies by 1 + w (added once, in 32 bits,
-    when the weights are loaded)."""
+    when the weights are loaded).  ``scale_name``: the result is multiplied by one more vector; both factors are one
+    32-bit weight from the loading on."""
 
     graph_safe = True
 
@@ -20,19 +21,29 @@ class RmsNorm(Norm):
 
     def tensor_decls(self):
         one_plus = getattr(self.spec, "one_plus", False)
-        return [TensorDecl(self._name(), (self.spec.size,), init="normal" if one_plus else "ones")]
+        d = [TensorDecl(self._name(), (self.spec.size,), init="normal" if one_plus else "ones")]
+        if getattr(self.spec, "scale_name", None):
+            d.append(TensorDecl(self.spec.scale_name, (self.spec.size,), init="ones"))
+        return d
 
     def load(self, src, rt):
         super().load(src, rt)
         self.weight = src.get(self._name())
         if getattr(self.spec, "one_plus", False):
             self.weight = (1.0 + self.weight.to(torch.float32)).contiguous()
+        if getattr(self.spec, "scale_name", None):
+            self.weight = (self.weight.to(torch.float32) * src.get(self.spec.scale_name).to(torch.float32)).contiguous()
 
     def forward(self, h, rows=None):
         n = h.shape[0] if rows is None else rows.numel()
         out = self.rt.empty(n, self.spec.size)
         return ops.rmsnorm(h, self.weight, self.spec.eps, out, rows=rows)
 
+    def forward_in_place(self, h):
+        """The 32-bit stream normed where it lies."""
+        normed = self.rt.empty(h.shape[0], h.shape[1], dtype=torch.float32)
+        h.copy_(ops.rmsnorm(h, self.weight, self.spec.eps, normed))
+        return h
 
     def as_rms(self):
         return self.weight, self.spec.eps

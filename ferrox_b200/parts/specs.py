@@ -26,6 +26,9 @@ class NormSpec:
     kind: str = "rms_norm"
     name: Optional[str] = None  # the weight tensor's full name, where it is not <prefix>weight
     one_plus: bool = False  # the stored weight lies around zero: the norm multiplies by 1 + w
+    # the full name of a further [size] vector the norm's result is multiplied by, element by element (a layer scale
+    # behind an output norm)
+    scale_name: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -114,6 +117,22 @@ class AttentionSpec:
     # name (after <prefix>) of a [n_heads * value_dim, hidden] matrix g: the concatenated heads are multiplied
     # element by element with sigmoid(g x) before the output projection
     output_gate: Optional[str] = None
+    # a query sees the keys of its own chunk of that many positions only, counted from the request's start
+    chunk: Optional[int] = None
+    # name (after <prefix>) of a [n_heads] vector: exp(sink_h) joins the softmax's denominator
+    sink: Optional[str] = None
+    value_mix: Optional["ValueMixSpec"] = None  # the values take part in the mixing of values across layers
+
+
+@dataclass(frozen=True)
+class ValueMixSpec:
+    """Values mixed across layers: the ``source`` layer's values as projected are v_first, every other layer of the
+    ``group`` caches (1 - lambda) v + lambda v_first of the same token.  ``name``: the [] tensor lambda after the
+    mixer's prefix (a checkpoint may hold one for the source as well, which nothing reads)."""
+
+    name: str
+    source: bool
+    group: str = "values"
 
 
 @dataclass(frozen=True)
@@ -265,7 +284,7 @@ class DenseMlpSpec:
     intermediate: int
     prefix: str  # tensors: <prefix>{gate,up,down}_proj.weight
     kind: str = "swiglu_mlp"
-    activation: str = "silu"  # what the gate passes through: silu or relu
+    activation: str = "silu"  # what the gate passes through: silu, relu or gelu_tanh
     tensor_names: Optional[Tuple[str, str, str]] = None  # (gate, up, down) after <prefix>, if spelled differently
     bias_names: Optional[Tuple[str, str, str]] = None  # (gate, up, down) biases after <prefix>; None: no biases
 
@@ -311,6 +330,10 @@ class MoeSpec:
     weight_scale: float = 1.0  # the final weights are multiplied by this
     renorm_eps: float = 0.0  # added to the sum the kept scores are divided by (norm_topk_prob)
     shared_gate_name: Optional[str] = None  # name after <prefix> of the shared expert's [1, hidden] gate row
+    # no router: the name after <prefix> of an integer table [vocab, top_k] whose rows name each token id's experts
+    # (distinct), all with weight 1 / top_k (scores, norm_topk_prob and the router's other options then do not apply)
+    table: Optional[str] = None
+    vocab: int = 0  # rows of the table
 
 
 @dataclass(frozen=True)
@@ -352,6 +375,7 @@ class SandwichBlockSpec:
     ffn: Optional[object]
     post2: Optional[object]
     kind: str = "sandwich_norm"
+    unused_tensors: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()  # (name, shape) a checkpoint may carry all the same
 
 
 @dataclass(frozen=True)

@@ -34,6 +34,7 @@ class TensorDecl:
     init: str = "normal"  # how the random-weights mode fills it: normal | ones | zeros
     optional: bool = False  # present or absent by the file's choice (e.g. a gate vector)
     integer: bool = False  # an integer table (kept as int32)
+    below: int = 0  # the integers of a row (last dimension) are distinct, from 0 on and below this (random-weights mode)
 
 
 def resident_dtype(stored: torch.dtype, compute: torch.dtype) -> torch.dtype:

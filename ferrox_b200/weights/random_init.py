@@ -129,8 +129,26 @@ def normal(key: int, shape, dtype, mean: float, std: float, device="cpu") -> tor
     return normal_cpu(key, n, mean, std).reshape(tuple(shape)).to(dtype)
 
 
+def distinct_rows(key: int, shape, below: int) -> torch.Tensor:
+    """int32 [rows, n]: every row holds n distinct integers in [0, below), the first n of a shuffle of them: the
+    integers in the order of hashes of (key, row, integer)."""
+    rows, n = shape
+    if n > below:
+        raise ValueError(f"{n} distinct integers below {below}")
+    out = torch.empty(rows, n, dtype=torch.int32)
+    step = max(1, _CHUNK // below)
+    for a in range(0, rows, step):
+        b = min(rows, a + step)
+        i = torch.arange(a * below, b * below, dtype=torch.int64).view(b - a, below)
+        h = _mix64((i + 1) * _i64(_GOLDEN) + _i64(key))
+        out[a:b] = torch.argsort(h, dim=1, stable=True)[:, :n].to(torch.int32)
+    return out
+
+
 def random_tensor(decl: TensorDecl, seed: int, dtype, std: float, norm_init: str, device="cpu") -> torch.Tensor:
     if decl.integer:
+        if decl.below:
+            return distinct_rows(tensor_key(seed, decl.name), decl.shape, decl.below).to(device)
         return torch.zeros(decl.shape, dtype=torch.int32, device=device)
     if decl.init == "zeros":
         return torch.zeros(decl.shape, dtype=dtype, device=device)
