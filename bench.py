@@ -5,6 +5,7 @@
     python bench.py --designs        (the Safepel design beside the dense decoder at equal sizes; its own JSON line)
     python bench.py --designs bobepel   (the Bobepel design beside the Qwen2-MoE decoder at equal sizes)
     python bench.py --designs zanezen   (the Zanezen design beside Bobepel at equal sizes)
+    python bench.py --designs balelorn   (the Balelorn design beside the Qwen2-MoE decoder at equal sizes)
 
 Default workload: the layer sizes of the Qwen1.5-MoE-A2.7B shape (24 layers, hidden
 2048, 16 heads of 128, 60 experts top-4 of width 1408, shared expert 5632, vocab
@@ -265,6 +266,19 @@ def zanezen_shape(width, layers, vocab=32768):
             "layers": [(mlstm, att(moe), att(dense), lat)[i % 4] for i in range(layers)]}
 
 
+def balelorn_shape(width, layers, vocab=32768, chunk=1024):
+    """Layer sizes that resemble a real model's: heads of 128 on a quarter as many key heads, half of each head
+    rotated, chunks of 1,024 positions, values mixed with the first layer's, an output gate; 60 experts of which a
+    token uses 4, as wide as the Qwen2-MoE shape's, chosen by a table."""
+    h = width // 128
+    mlp = {"kind": "moe", "expert": {"ff": width * 11 // 16 // 64 * 64, "limit": 7.0}, "router": {"experts": 60, "top": 4}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": chunk},
+        "rot": {"dims": 64, "base": 1000000.0}, "v_mix": True}}
+    return {"architecture": "Balelorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "max_positions": CONTEXT,
+            "layers": [att] * layers}
+
+
 def compare_designs(args) -> int:
     """Prefill and decode throughput of a design and of the closest existing decoder at a few equal sizes (random
     bfloat16 weights), with the device time of every class of kernel from a traced pass beside them."""
@@ -290,7 +304,7 @@ def compare_designs(args) -> int:
         torch.cuda.synchronize()
         return a.elapsed_time(b)
 
-    def measure(cfg):
+    def measure(cfg, random_ids=False):
         n_pages = (PREFILL_TOKENS + steps + 80) // ps * (batch + 1) + 8
         kw = dict(seed=0, dtype="bfloat16", on_device=True, page_size=ps, n_pages=n_pages, max_slots=batch + 1,
                   max_positions=CONTEXT)
@@ -322,6 +336,8 @@ def compare_designs(args) -> int:
                 nonlocal ids
                 logits = eng.step([StepEntry(s, [t], want=[0]) for s, t in zip(slots, ids)], check=False)
                 ids = ops.argmax(logits, dev).tolist()
+                if random_ids:      # experts that follow from the token ids: the choices of a random model are alike
+                    ids = prompt(b)
 
             for _ in range(max(3, args.warmup)):
                 one_step()
@@ -391,6 +407,15 @@ def compare_designs(args) -> int:
                           "prompt_tokens": PREFILL_TOKENS, "decode_steps_timed": steps, "peaks": pk,
                           "data": "synthetic: random N(0,0.02) weights, uniform random token ids", "sizes": rows}))
         return 0
+    if args.designs == "balelorn":
+        for width, layers, _ in sizes:
+            a, b = balelorn_shape(width, layers), dict(moe_like(width, layers), shared_expert_intermediate_size=0)
+            rows.append({"width": width, "layers": layers, "expert_ff": b["moe_intermediate_size"],
+                         "balelorn": measure(a, random_ids=True), "qwen2_moe": measure(b, random_ids=True)})
+        print(json.dumps({"designs": "Balelorn beside the Qwen2-MoE decoder (no shared expert) at equal size", "dtype": "bf16",
+                          "batch": batch, "prompt_tokens": PREFILL_TOKENS, "decode_steps_timed": steps, "peaks": pk,
+                          "data": "synthetic: random N(0,0.02) weights, uniform random token ids", "sizes": rows}))
+        return 0
     if args.designs == "bobepel":
         for width, layers, _ in sizes:
             a, b = bobepel_shape(width, layers), moe_like(width, layers)
@@ -423,11 +448,12 @@ def main() -> int:
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--page-size", type=int, default=64)
     ap.add_argument("--repeats", type=int, default=3, help="timed regions of --steps steps each; the median counts")
-    ap.add_argument("--designs", nargs="?", const="safepel", default=None, choices=["safepel", "bobepel", "sesuzen", "sesuzen-moe", "zanezen"],
+    ap.add_argument("--designs", nargs="?", const="safepel", default=None, choices=["safepel", "bobepel", "sesuzen", "sesuzen-moe", "zanezen", "balelorn"],
                     help="instead of the default workload: prefill and decode of a design beside the closest existing "
                          "decoder at a few equal sizes, with device time per class of kernel (safepel: beside the dense "
                          "Qwen2 decoder; bobepel: beside the Qwen2-MoE decoder; sesuzen: dense feed-forwards, beside "
-                         "Safepel; sesuzen-moe: experts, beside the Qwen2-MoE decoder without its shared expert; zanezen: beside Bobepel)")
+                         "Safepel; sesuzen-moe: experts, beside the Qwen2-MoE decoder without its shared expert; zanezen: beside Bobepel; balelorn: beside the Qwen2-MoE decoder without its "
+                         "shared expert)")
     ap.add_argument("--widths", default="", help="--designs: only these widths (commas), e.g. 2048")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -70,8 +70,8 @@ int fx_general_attention(const void* q, long ldq, long ldqh, const void* k_pages
 
 int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                             const int* block_table, int table_width, int page_size, const int* items, int n_items,
-                            const int* seq_slot, void* out, long ldo, int n_heads, int n_kv_heads, int head_dim,
-                            int window, float scale, int* status, float* part_o, float* part_ml, const int* merges,
+                            const int* seq_slot, void* out, long ldo, int n_heads, int n_kv_heads, int head_dim, int value_dim,
+                            int window, int chunk, float scale, const float* sinks, const void* gate, long ldg, int* status, float* part_o, float* part_ml, const int* merges,
                             int n_merges, void* stream);
 int fx_prefill_attention(const void* q, long ldq, const void* k_pages, const void* v_pages, const int* block_table,
                          int table_width, int page_size, const int* tiles, int n_tiles, const int* seq_slot, void* out,
@@ -151,12 +151,24 @@ int fx_decode_split_mma(const void* q, long ldq, const void* k_pages, const void
                         float* part_acc, float* part_ml, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                         int window, float scale, int split_len, int n_splits, int fresh_positions, float softcap,
                         void* stream);
+// Options of the decode attention kernel that streams pages by TMA (bfloat16; the other decode kernels refuse them).
+typedef struct DecodeExtras {
+    int chunk;               // > 0: a query sees the keys of its own chunk of that many positions only
+    int rot;                 // store_new: the first rot elements of a head are rotated (0: the whole head)
+    const float* sinks;      // one per head: exp(sinks[h]) joins the softmax's denominator once
+    const void* gate;        // token rows of n_heads * head_dim, ldg elements apart: the result times sigmoid(gate)
+    long ldg;
+    const void* v_first;     // store_new: the value that is stored is (1 - lambda) v + lambda v_first, v_first token
+    long ld_first;           //            rows of n_kv_heads * head_dim
+    float lambda;
+} DecodeExtras;
+
 int fx_decode_split_tma(const void* q, long ldq, const void* k_pages, const void* v_pages, int n_pages,
                         const int* block_table, int table_width, int page_size, const int* positions,
                         const int* token_seq, const int* seq_slot, float* part_acc, float* part_ml, int n_tokens,
                         int n_heads, int n_kv_heads, int head_dim, int window, float scale, int split_len,
                         int n_splits, int* status, void* out, long ldo, int* counters, int fresh_positions,
-                        int store_new, int write_pages, const float* cos_sin, void* stream);
+                        int store_new, int write_pages, const float* cos_sin, const DecodeExtras* extras, void* stream);
 // n_pages > 0 (the number of pages behind k_pages / v_pages) lets bfloat16 take the TMA kernel; status: the step's
 // status word (may be null).
 // fresh_positions: 0 makes no assumption about the kernel launched before this one on the stream: nothing is read until
@@ -174,7 +186,8 @@ int fx_decode_attention(const void* q, long ldq, const void* k_pages, const void
                         const int* token_seq, const int* seq_slot, void* out, long ldo, float* part_acc,
                         float* part_ml, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int window,
                         float scale, int split_len, int n_splits, int* status, int* counters, int fresh_positions,
-                        int store_new, int write_pages, const float* cos_sin, float softcap, void* stream);
+                        int store_new, int write_pages, const float* cos_sin, float softcap, const DecodeExtras* extras,
+                        void* stream);
 // attention_prep.cu: what mixers with normed queries and keys, a query temperature, keys and values of different
 // widths, or a latent cache do between their projections and the attention kernel
 int fx_qk_norm_store(void* qkv, int dtype, long ld, const int* positions, const int* token_seq, const int* seq_slot,

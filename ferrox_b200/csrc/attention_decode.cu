@@ -254,20 +254,25 @@ __global__ void __launch_bounds__(NTHREADS) decode_split_kernel(
 template <typename T>
 __global__ void merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                              const int* __restrict__ positions, T* __restrict__ out, long ldo, int n_heads,
-                             int head_dim, int n_splits, int split_len, int window)
+                             int head_dim, int n_splits, int split_len, int window, DecodeExtras x)
 {
     fx_pdl_wait();
     const int tkn = blockIdx.x, h = blockIdx.y;
     const long base = ((long)tkn * n_heads + h) * n_splits;
     // the splits that hold visible keys of this token (the others were not written)
     const int pos = positions[tkn];
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = fx_first_key(pos, window, x.chunk);
     auto has_keys = [&](int s) { int b, e; fx_split_range(pos, lo, s, n_splits, split_len, b, e); return b < e; };
     float mm = -INFINITY;
     for (int s = 0; s < n_splits; ++s)
         if (has_keys(s)) mm = fmaxf(mm, part_ml[(base + s) * 2]);
+    float sunk = 0.f;        // the head's sink: a term of the denominator that no range holds
+    if (x.sinks && mm != -INFINITY) {
+        mm = fmaxf(mm, x.sinks[h]);
+        sunk = fx_exp<T>(x.sinks[h] - mm);
+    }
     for (int e = threadIdx.x; e < head_dim; e += blockDim.x) {
-        float ll = 0.f, a = 0.f;
+        float ll = sunk, a = 0.f;
         for (int s = 0; s < n_splits; ++s) {
             if (!has_keys(s)) continue;
             const float ms = part_ml[(base + s) * 2];
@@ -276,7 +281,9 @@ __global__ void merge_kernel(const float* __restrict__ part_acc, const float* __
             ll += part_ml[(base + s) * 2 + 1] * w;
             a += part_acc[(base + s) * head_dim + e] * w;
         }
-        out[(long)tkn * ldo + (long)h * head_dim + e] = from_f32<T>(ll > 0.f ? a / ll : 0.f);
+        float v = ll > 0.f ? a / ll : 0.f;
+        if (x.gate) v *= fx_sigmoid_fast(to_f32(reinterpret_cast<const T*>(x.gate)[(long)tkn * x.ldg + (long)h * head_dim + e]));
+        out[(long)tkn * ldo + (long)h * head_dim + e] = from_f32<T>(v);
     }
 }
 
@@ -316,8 +323,12 @@ int run(const void* q, long ldq, const void* k_pages, const void* v_pages, int n
         int table_width, int page_size, const int* positions, const int* token_seq, const int* seq_slot, void* out,
         long ldo, float* part_acc, float* part_ml, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int window,
         float scale, int split_len, int n_splits, int* status, int* counters, int fresh, int store_new, int write_pages,
-        const float* cos_sin, float softcap, cudaStream_t s)
+        const float* cos_sin, float softcap, const DecodeExtras* extras, cudaStream_t s)
 {
+    // (chunks, sinks and gates are options of the kernel that streams pages by TMA: the others refuse them)
+    const DecodeExtras x = extras ? *extras : DecodeExtras{};
+    const bool plain = x.chunk == 0 && !x.sinks && !x.gate && !x.v_first && x.rot == 0;
+    if (!plain && (sizeof(T) != 2 || softcap > 0.f || n_pages <= 0)) return FX_ERR_SIZE;
     if (softcap > 0.f && store_new) return FX_ERR_SIZE;   // the kernel that stores the step's keys itself takes no cap
     constexpr int N = Vec<T>::N;
     if (head_dim % N || head_dim > MAX_D || head_dim <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads) return FX_ERR_SIZE;
@@ -331,18 +342,18 @@ int run(const void* q, long ldq, const void* k_pages, const void* v_pages, int n
             rc_mma = fx_decode_split_tma(q, ldq, k_pages, v_pages, n_pages, block_table, table_width, page_size,
                                          positions, token_seq, seq_slot, part_acc, part_ml, n_tokens, n_heads,
                                          n_kv_heads, head_dim, window, scale, split_len, n_splits, status, out, ldo,
-                                         counters, fresh, store_new, write_pages, cos_sin, (void*)s);
+                                         counters, fresh, store_new, write_pages, cos_sin, extras, (void*)s);
             if (rc_mma == FX_OK && (counters || n_splits == 1)) return FX_OK;   // merged by the kernel's last blocks
         }
         // only the kernel above rotates and stores the step's own keys and values itself
-        if (store_new && rc_mma != FX_OK) return rc_mma;
+        if ((store_new || !plain) && rc_mma != FX_OK) return rc_mma;
         if (rc_mma < 0)
             rc_mma = fx_decode_split_mma(q, ldq, k_pages, v_pages, block_table, table_width, page_size, positions,
                                          token_seq, seq_slot, part_acc, part_ml, n_tokens, n_heads, n_kv_heads,
                                          head_dim, window, scale, split_len, n_splits, fresh, softcap, (void*)s);
         if (rc_mma == FX_OK) {
             fx_launch_pdl(merge_kernel<T>, dim3(n_tokens, n_heads), 64, 0, s, part_acc, part_ml, positions, (T*)out, ldo,
-                          n_heads, head_dim, n_splits, split_len, window);
+                          n_heads, head_dim, n_splits, split_len, window, x);
             return fx_launch_status();
         }
         if (rc_mma > 0) return rc_mma;   // a CUDA error; a refusal (< 0) falls through to the CUDA-core kernel
@@ -369,7 +380,7 @@ int run(const void* q, long ldq, const void* k_pages, const void* v_pages, int n
 #undef FX_GO
     if (rc != FX_OK) return rc;
     fx_launch_pdl(merge_kernel<T>, dim3(n_tokens, n_heads), 64, 0, s, part_acc, part_ml, positions, (T*)out, ldo, n_heads, head_dim,
-                                                          n_splits, split_len, window);
+                                                          n_splits, split_len, window, x);
     return fx_launch_status();
 }
 
@@ -382,7 +393,7 @@ extern "C" int fx_decode_attention(const void* q, long ldq, const void* k_pages,
                                    float* part_acc, float* part_ml, int n_tokens, int n_heads, int n_kv_heads,
                                    int head_dim, int window, float scale, int split_len, int n_splits, int* status,
                                    int* counters, int fresh_positions, int store_new, int write_pages,
-                                   const float* cos_sin, float softcap, void* stream)
+                                   const float* cos_sin, float softcap, const DecodeExtras* extras, void* stream)
 {
     if (n_tokens <= 0) return FX_OK;
     if (split_len < 0 || n_splits <= 0) return FX_ERR_SIZE;
@@ -390,11 +401,11 @@ extern "C" int fx_decode_attention(const void* q, long ldq, const void* k_pages,
     if (dtype == FX_F32)
         return run<float>(q, ldq, k_pages, v_pages, n_pages, block_table, table_width, page_size, positions, token_seq,
                           seq_slot, out, ldo, part_acc, part_ml, n_tokens, n_heads, n_kv_heads, head_dim, window, scale,
-                          split_len, n_splits, status, counters, fresh_positions, store_new, write_pages, cos_sin, softcap, s);
+                          split_len, n_splits, status, counters, fresh_positions, store_new, write_pages, cos_sin, softcap, extras, s);
     if (dtype == FX_BF16)
         return run<bf16>(q, ldq, k_pages, v_pages, n_pages, block_table, table_width, page_size, positions, token_seq,
                          seq_slot, out, ldo, part_acc, part_ml, n_tokens, n_heads, n_kv_heads, head_dim, window, scale,
-                         split_len, n_splits, status, counters, fresh_positions, store_new, write_pages, cos_sin, softcap, s);
+                         split_len, n_splits, status, counters, fresh_positions, store_new, write_pages, cos_sin, softcap, extras, s);
     return FX_ERR_DTYPE;
 }
 
@@ -449,10 +460,10 @@ extern "C" int fx_decode_attention_noalloc(const void* q, long ldq, const void* 
     if (dtype == FX_F32)
         return run<float>(q, ldq, k_pages, v_pages, 0, block_table, table_width, page_size, positions, token_seq, seq_slot,
                           out, ldo, part_acc, part_ml, n_tokens, n_heads, n_kv_heads, head_dim, window, scale,
-                          split_len, n_splits, nullptr, nullptr, 0, 0, 0, nullptr, 0.f, s);
+                          split_len, n_splits, nullptr, nullptr, 0, 0, 0, nullptr, 0.f, nullptr, s);
     if (dtype == FX_BF16)
         return run<bf16>(q, ldq, k_pages, v_pages, 0, block_table, table_width, page_size, positions, token_seq, seq_slot,
                          out, ldo, part_acc, part_ml, n_tokens, n_heads, n_kv_heads, head_dim, window, scale,
-                         split_len, n_splits, nullptr, nullptr, 0, 0, 0, nullptr, 0.f, s);
+                         split_len, n_splits, nullptr, nullptr, 0, 0, 0, nullptr, 0.f, nullptr, s);
     return FX_ERR_DTYPE;
 }

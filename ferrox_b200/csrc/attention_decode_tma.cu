@@ -28,6 +28,9 @@
 //
 // Every wait on a barrier is bounded; a block that gives up raises the status word.
 //
+// Options (DecodeExtras in api.h): chunks, a number per head in the softmax's denominator, an output gate; with
+// store_new also a rotation of part of a head and values mixed with another layer's.
+//
 // Reference: crates/ferrox-core/src/attention.rs:146-175 (online softmax), :484-524
 // (window), :572-610 (pages).
 #include "tc_common.cuh"
@@ -57,14 +60,30 @@ struct DecArgs {
     // token is written to `out` at once if that is given.
     bf16* out; long ldo; int* counters;
     // store_new: the rows of q are the fused [q | k | v] rows of the step as the projection left them, one token a
-    // request.  The kernel then rotates the queries itself (split-half pairs over the whole head, cos and sin from
-    // cos_sin [tokens][head_dim / 2][2]; null: no rotation), and the block that holds a token's own position rotates
-    // that token's key, puts it and the value into its copy of their tile, and (one block per kv head, if
+    // request.  The kernel then rotates the queries itself (split-half pairs over the first rot elements of a head, cos
+    // and sin from cos_sin [tokens][rot / 2][2]; null: no rotation), and the block that holds a token's own position rotates
+    // that token's key, mixes its value (x.v_first), puts both into its copy of their tile, and (one block per kv head, if
     // write_pages) into the cache pages: the work of the rotary kernel without its launch.
     int store_new, write_pages;
-    const float* cos_sin;
+    const float* cos_sin; int rot;
     bf16* k_pages; bf16* v_pages;
+    DecodeExtras x;
 };
+
+// acc / (l + the head's sink): the result of a head whose sums are relative to e^mx; then the output gate.
+__device__ __forceinline__ float finish(const DecArgs& a, float acc, float l, float mx, int tkn, int head, int e)
+{
+    float v = 0.f;
+    if (l > 0.f) {
+        if (a.x.sinks) {
+            const float sk = a.x.sinks[head], mm = fmaxf(mx, sk), f = __expf(mx - mm);
+            v = acc * f / (l * f + __expf(sk - mm));
+        } else v = acc / l;
+    }
+    if (a.x.gate)
+        v *= fx_sigmoid_fast(__bfloat162float(reinterpret_cast<const bf16*>(a.x.gate)[(long)tkn * a.x.ldg + (long)head * a.head_dim + e]));
+    return v;
+}
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, int src_bytes) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
@@ -106,7 +125,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
     const int tkn = blockIdx.y, split = blockIdx.z;
     const int pos = a.positions[tkn];
     const int seq = a.token_seq[tkn];                 // (asked for beside the position: the table row hangs on it)
-    const int lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+    const int lo = fx_first_key(pos, a.window, a.x.chunk);
     int k_begin, k_end;
     fx_split_range(pos, lo, split, a.n_splits, a.split_len, k_begin, k_end);
     if (k_begin >= k_end) return;   // nothing of this range is visible: `merge` skips it by the same rule
@@ -178,7 +197,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
         // ---------------- four scoring warps ----------------
         const int g = lane >> 2, t4 = lane & 3;
         const int chunks_row = head_dim / 8;                   // 16-byte chunks per row
-        const int half_d = head_dim >> 1;
+        const int half_d = a.rot >> 1;                         // pairs of a head that are rotated
         // store_new: the warp whose 16 keys of the last tile hold the token's own position prepares that key and value
         const bool owns_new = a.store_new && pos >= k_begin && pos < k_end && warp == ((pos % TK) >> 4);
         const bool writes_page = owns_new && a.write_pages && blockIdx.x % chunks == 0;
@@ -206,9 +225,13 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
                 const int e = lane + 32 * u;
                 if (e < head_dim) {
                     new_v[u] = vrow[e];
+                    if (a.x.v_first) {
+                        const float first = __bfloat162float(reinterpret_cast<const bf16*>(a.x.v_first)[(long)tkn * a.x.ld_first + (long)kvh * head_dim + e]);
+                        new_v[u] = __float2bfloat16_rn((1.0f - a.x.lambda) * __bfloat162float(new_v[u]) + a.x.lambda * first);
+                    }
                     float x = __bfloat162float(krow[e]);
-                    if (a.cos_sin) {
-                        // element e pairs with e +- head_dim / 2; the same arithmetic as the rotary kernel's
+                    if (a.cos_sin && e < a.rot) {
+                        // element e pairs with e +- rot / 2; the same arithmetic as the rotary kernel's
                         const int i = e < half_d ? e : e - half_d;
                         const float2 cs = *reinterpret_cast<const float2*>(a.cos_sin + ((long)tkn * half_d + i) * 2);
                         const float other = __bfloat162float(krow[e < half_d ? e + half_d : e - half_d]);
@@ -232,7 +255,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         consumers_sync();
         if (rotates_q) {
-            // the queries as projected: rotate them where they lie (pairs i, i + head_dim / 2 of every head)
+            // the queries as projected: rotate them where they lie (pairs i, i + rot / 2 of every head)
             bf16* q_s = reinterpret_cast<bf16*>(smem_raw + (q_u - smem_u32(smem_raw)));
             for (int idx = threadIdx.x; idx < nq * half_d; idx += NCONSUMERS) {
                 const int r = idx / half_d, i = idx - r * half_d;
@@ -377,7 +400,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
                 }
                 if (a.n_splits == 1 && a.out) {
                     // the only key range of its token: this is the result
-                    a.out[(long)tkn * a.ldo + (long)(h0 + h) * head_dim + e] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+                    a.out[(long)tkn * a.ldo + (long)(h0 + h) * head_dim + e] = __float2bfloat16(finish(a, acc, ll, mm * a.scale, tkn, h0 + h, e));
                     continue;
                 }
                 const long slot = ((long)tkn * n_heads + (h0 + h)) * a.n_splits + split;
@@ -451,7 +474,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
                                 acc += part[u] * wgt;
                             }
                         }
-                        a.out[(long)tkn * a.ldo + (long)(h0 + h) * head_dim + e] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+                        a.out[(long)tkn * a.ldo + (long)(h0 + h) * head_dim + e] = __float2bfloat16(finish(a, acc, ll, mm, tkn, h0 + h, e));
                     }
                 }
             }
@@ -509,7 +532,8 @@ extern "C" int fx_decode_split_tma(const void* q, long ldq, const void* k_pages,
                                    const int* token_seq, const int* seq_slot, float* part_acc, float* part_ml,
                                    int n_tokens, int n_heads, int n_kv_heads, int head_dim, int window, float scale,
                                    int split_len, int n_splits, int* status, void* out, long ldo, int* counters,
-                                   int fresh_positions, int store_new, int write_pages, const float* cos_sin, void* stream)
+                                   int fresh_positions, int store_new, int write_pages, const float* cos_sin,
+                                   const DecodeExtras* extras, void* stream)
 {
     if (n_tokens <= 0) return FX_OK;
     if (counters && (n_splits > 32 || !out || ldo % 2)) return FX_ERR_SIZE;
@@ -540,7 +564,11 @@ extern "C" int fx_decode_split_tma(const void* q, long ldq, const void* k_pages,
     a.scale_log2e = scale * 1.4426950408889634f; a.scale = scale;
     a.split_len = split_len; a.n_splits = n_splits; a.stages = stages; a.status = status;
     a.fresh = fresh_positions;
-    a.store_new = store_new; a.write_pages = write_pages; a.cos_sin = cos_sin;
+    a.store_new = store_new; a.write_pages = write_pages; a.cos_sin = cos_sin; a.rot = head_dim;
+    a.x = DecodeExtras{};
+    if (extras) a.x = *extras;
+    if (a.x.rot > 0) a.rot = a.x.rot;
+    if (a.x.chunk < 0 || a.rot % 2 || a.rot > head_dim) return FX_ERR_SIZE;
     a.k_pages = (bf16*)const_cast<void*>(k_pages); a.v_pages = (bf16*)const_cast<void*>(v_pages);
     a.out = (bf16*)out; a.ldo = ldo; a.counters = counters;
     if (n_splits > 1 && !counters) a.out = nullptr;   // partial results only

@@ -80,8 +80,6 @@ struct GArgs {
     const bf16* gate; long ldg;   // (optional) token rows of n_heads * value_dim: the result times sigmoid(gate)
 };
 
-__device__ __forceinline__ float sigmoid_of(float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); }
-
 // DVMAX: most value columns one warp accumulates.  NSPLIT: sets of 4 warps that share out the value columns.
 // BKEY: keys a block of the loop holds.
 template <int DVMAX, int NSPLIT, int BKEY>
@@ -323,7 +321,7 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
             if (a.gate) {      // the output gate, on the 32-bit result
                 const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g0 + col));
                 const float2 gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g1 + col));
-                x0 *= sigmoid_of(ga.x); x1 *= sigmoid_of(ga.y); x2 *= sigmoid_of(gb.x); x3 *= sigmoid_of(gb.y);
+                x0 *= fx_sigmoid_fast(ga.x); x1 *= fx_sigmoid_fast(ga.y); x2 *= fx_sigmoid_fast(gb.x); x3 *= fx_sigmoid_fast(gb.y);
             }
             if (r0 < rows) *reinterpret_cast<uint32_t*>(o0 + col) = pack_bf16(x0, x1);
             if (r1 < rows) *reinterpret_cast<uint32_t*>(o1 + col) = pack_bf16(x2, x3);
@@ -363,7 +361,7 @@ __global__ void general_merge_kernel(const float* __restrict__ part_o, const flo
             acc += part_o[(base + s) * value_dim + e] * w;
         }
         float x = ll > 0.f ? acc / ll : 0.f;
-        if (gate) x *= sigmoid_of(__bfloat162float(gate[(long)tkn * ldg + (long)h * value_dim + e]));
+        if (gate) x *= fx_sigmoid_fast(__bfloat162float(gate[(long)tkn * ldg + (long)h * value_dim + e]));
         out[(long)tkn * ldo + (long)h * ldoh + e] = __float2bfloat16_rn(x);
     }
 }

@@ -1,5 +1,6 @@
-// Attention for prompt portions on the 5th-generation tensor cores (bfloat16, head_dim 64 or 128,
-// pages of 64 positions or a multiple).
+// Attention for prompt portions on the 5th-generation tensor cores (bfloat16, keys and values of up to 128
+// elements a head in steps of 8, pages of 64 positions or a multiple).  Key and value widths may differ; in shared
+// and tensor memory both are rounded up to 64 or 128 (D and V below), the rest filled with zeros by the TMA.
 //
 // One CTA takes up to 256 query tokens of one request and one head, as two sub-tiles of 128 rows, and
 // walks that request's keys in blocks of 128 positions (earlier steps' keys and the portion's own alike,
@@ -36,6 +37,10 @@
 // it has (the unnormalised sums in 32 bits, and each row's reference maximum and sum of weights) into
 // scratch memory, and a second kernel (prefill_merge_kernel) adds a tile's runs up in their order.
 //
+// Options: `chunk` (a query sees the keys of its own chunk of that many positions only, counted from the request's
+// start), `sinks` (one number per head: exp(sink_h) joins the softmax's denominator once, at the end or in the merge),
+// `gate` (token rows of n_heads * value_dim: the result is multiplied by sigmoid(gate) before it is rounded).
+//
 // Reference: crates/ferrox-core/src/attention.rs:531-563 (query t over keys 0..=t), :146-175 (online
 // softmax), :484-524 (window), :572-610 (pages), :432-449 (grouped heads).  The mma.sync kernel of
 // attention_prefill.cu remains for other head sizes and page sizes.
@@ -62,28 +67,39 @@ struct AttnArgs {
     const int* tiles; const int* seq_slot;
     bf16* out; long ldo;
     float* part_o; float* part_ml;   // partial results of items that hold a run of their tile's key blocks only
-    int n_heads, n_kv_heads, window;
+    int n_heads, n_kv_heads, window, chunk;
+    int value_dim;                   // elements of a value head (V: rounded up)
+    const float* sinks;              // (optional) one per head
+    const bf16* gate; long ldg;      // (optional) token rows of n_heads * value_dim
     float scale_log2e;
     int* status;
 };
 
-template <int D>
+// What a row's sums are multiplied with at the end: 1 / (l + the head's sink), l being relative to 2^ref.
+__device__ __forceinline__ float inverse_sum(float l, float ref, const float* sinks, int head) {
+    if (!(l > 0.f)) return 0.f;
+    if (!sinks) return 1.f / l;
+    const float sk = sinks[head] * 1.4426950408889634f, mm = fmaxf(ref, sk), f = fast_exp2(ref - mm);
+    return f / (l * f + fast_exp2(sk - mm));
+}
+
+template <int D, int V>
 struct Smem {
-    static constexpr int HALVES = D / 64;                  // 64-element (128-byte) slices of the head dimension
+    static constexpr int HALVES = D / 64, V_HALVES = V / 64;   // 64-element (128-byte) slices of a key's, a value's row
     static constexpr int SUB = 128 * 128;                  // bytes of a [128 rows x 128 bytes] piece
-    static constexpr int Q_BYTES = HALVES * SUB, KV_BYTES = HALVES * SUB;
-    static constexpr int Q_OFF = 0, K_OFF = 2 * Q_BYTES, V_OFF = K_OFF + 2 * KV_BYTES;
-    static constexpr int BAR_OFF = V_OFF + 2 * KV_BYTES;
+    static constexpr int Q_BYTES = HALVES * SUB, K_BYTES = HALVES * SUB, V_BYTES = V_HALVES * SUB;
+    static constexpr int Q_OFF = 0, K_OFF = 2 * Q_BYTES, V_OFF = K_OFF + 2 * K_BYTES;
+    static constexpr int BAR_OFF = V_OFF + 2 * V_BYTES;
     static constexpr int TOTAL = BAR_OFF + 128 + 1024;     // barriers, alignment slack
 };
 
-template <int D>
+template <int D, int V>
 __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                            const __grid_constant__ CUtensorMap map_k,
                                                                            const __grid_constant__ CUtensorMap map_v,
                                                                            AttnArgs a)
 {
-    using L = Smem<D>;
+    using L = Smem<D, V>;
     extern __shared__ uint8_t smem_raw[];
     __shared__ int abort_flag_s;
     __shared__ uint32_t tmem_base_s;
@@ -101,8 +117,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
     const int nt = rows > BQ ? 2 : 1;
     auto rows_of = [&](int t) { return min(BQ, rows - t * BQ); };
     auto blk_lo = [&](int t) {
-        const int p = pos0 + t * BQ;
-        return (a.window > 0 && p - a.window + 1 > 0 ? p - a.window + 1 : 0) / BKEY;
+        return fx_first_key(pos0 + t * BQ, a.window, a.chunk) / BKEY;
     };
     auto blk_hi = [&](int t) { return (pos0 + t * BQ + rows_of(t) - 1) / BKEY; };
     // the key blocks of sub-tile t inside this item's run: lo_t[t] .. hi_t[t] (none if lo > hi)
@@ -155,7 +170,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
             mbar_expect_tx(q_full, nt * L::Q_BYTES);
             for (int t = 0; t < nt; ++t)
                 for (int h = 0; h < L::HALVES; ++h)
-                    tma_load_2d(base + L::Q_OFF + t * L::Q_BYTES + h * L::SUB, &map_q, head * D + h * 64, tok0 + t * BQ, q_full);
+                    tma_load_3d(base + L::Q_OFF + t * L::Q_BYTES + h * L::SUB, &map_q, h * 64, head, tok0 + t * BQ, q_full);
             const int* table = a.block_table + (long)a.seq_slot[entry] * a.table_width;
             int issued = 0;
             for (int j = first_blk; j <= last_blk; ++j) {
@@ -168,15 +183,15 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                     page[hk] = p >= 0 ? p : 0;      // no page (beyond the request, or before its window): masked anyway
                     off[hk] = p >= 0 ? key % a.page_size : 0;
                 }
-                mbar_expect_tx(k_full(b), L::KV_BYTES);
+                mbar_expect_tx(k_full(b), L::K_BYTES);
                 for (int h = 0; h < L::HALVES; ++h)
                     for (int hk = 0; hk < 2; ++hk)
-                        tma_load_4d(base + L::K_OFF + b * L::KV_BYTES + h * L::SUB + hk * 8192, &map_k, h * 64, off[hk], kvh,
+                        tma_load_4d(base + L::K_OFF + b * L::K_BYTES + h * L::SUB + hk * 8192, &map_k, h * 64, off[hk], kvh,
                                     page[hk], k_full(b));
-                mbar_expect_tx(v_full(b), L::KV_BYTES);
-                for (int h = 0; h < L::HALVES; ++h)
+                mbar_expect_tx(v_full(b), L::V_BYTES);
+                for (int h = 0; h < L::V_HALVES; ++h)
                     for (int hk = 0; hk < 2; ++hk)
-                        tma_load_4d(base + L::V_OFF + b * L::KV_BYTES + h * L::SUB + hk * 8192, &map_v, h * 64, off[hk], kvh,
+                        tma_load_4d(base + L::V_OFF + b * L::V_BYTES + h * L::SUB + hk * 8192, &map_v, h * 64, off[hk], kvh,
                                     page[hk], v_full(b));
                 issued = i + 1;
             }
@@ -190,7 +205,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
         // ---------------- tensor-core issue ----------------
         if (lane == 0) {
             constexpr uint32_t idesc_s = instr_desc_ex(BQ, BKEY, 0);   // S: B = K tile, K-major
-            constexpr uint32_t idesc_o = instr_desc_ex(BQ, D, 1);      // O: B = V tile, N-major
+            constexpr uint32_t idesc_o = instr_desc_ex(BQ, V, 1);      // O: B = V tile, N-major
             int k_ready = first_blk - 1;   // the last block whose K is known to have landed
             bool ok = mbar_wait(q_full, 0, abort_flag);
             auto issue_s = [&](int t, int j) {
@@ -203,7 +218,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
 #pragma unroll
                 for (int h = 0; h < L::HALVES; ++h) {
                     const uint64_t dq = smem_desc(base + L::Q_OFF + t * L::Q_BYTES + h * L::SUB);
-                    const uint64_t dk = smem_desc(base + L::K_OFF + b * L::KV_BYTES + h * L::SUB);
+                    const uint64_t dk = smem_desc(base + L::K_OFF + b * L::K_BYTES + h * L::SUB);
 #pragma unroll
                     for (int k = 0; k < 4; ++k) tc_mma(tmem_s(t), dq + 2u * k, dk + 2u * k, idesc_s, (h | k) != 0);
                 }
@@ -227,7 +242,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                         // 64-element slices of the head dimension lie SUB bytes apart (the leading operand).
 #pragma unroll
                         for (int ks = 0; ks < BKEY / 16; ++ks) {
-                            const uint64_t dv = smem_desc_lbo_sbo(base + L::V_OFF + b * L::KV_BYTES + ks * 2048, L::SUB, 1024);
+                            const uint64_t dv = smem_desc_lbo_sbo(base + L::V_OFF + b * L::V_BYTES + ks * 2048, L::SUB, 1024);
                             tc_mma_ts(tmem_o(t), tmem_s(t) + 8u * ks, dv, idesc_o, (n_p[t] | ks) != 0);
                         }
                         ++n_p[t];
@@ -247,7 +262,8 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
             const int rows_t = rows_of(t);
             const int pos0_t = pos0 + t * BQ;
             const int p_r = pos0_t + r;                  // absolute position of this row
-            const int lo_r = a.window > 0 ? p_r - a.window + 1 : 0;
+            const int lo_r = fx_first_key(p_r, a.window, a.chunk);
+            const int lo_last = fx_first_key(pos0_t + BQ - 1, a.window, a.chunk);     // the largest of the sub-tile's rows
             const uint32_t lane_off = (uint32_t)(quad * 32) << 16;
             const uint32_t ts = tmem_s(t) + lane_off, to = tmem_o(t) + lane_off;
             const float sl2 = a.scale_log2e;
@@ -261,7 +277,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                 tc_fence_after();
                 const int kb = j * BKEY;
                 // every key of the block visible to every row of the sub-tile: no masking (most blocks)
-                const bool interior = kb + BKEY - 1 <= pos0_t && (a.window <= 0 || kb >= pos0_t + BQ - a.window);
+                const bool interior = kb + BKEY - 1 <= pos0_t && kb >= lo_last;
                 // The row of S is read in chunks of 32 columns into two register buffers in turn: the load of the
                 // next chunk is in flight while the current one is worked on.
                 uint32_t ca[32], cb[32], pk[32];
@@ -297,7 +313,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                     m = mn;
                     if (cnt > 0) {   // the sums so far of this row, in tensor memory, take the new reference too
 #pragma unroll
-                        for (int c = 0; c < D / 32; ++c) {
+                        for (int c = 0; c < V / 32; ++c) {
                             tc_ld32(to + c * 32, cb);
                             tc_ld_wait_for(cb);
 #pragma unroll
@@ -344,9 +360,9 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                 const long slot = ((long)part * a.n_heads + head) * (2 * BQ) + t * BQ + r;
                 if (r < rows_t) { a.part_ml[slot * 2] = has_blocks ? m : -INFINITY; a.part_ml[slot * 2 + 1] = has_blocks ? l : 0.f; }
                 if (has_blocks) {
-                    float* dst = a.part_o + slot * D;
+                    float* dst = a.part_o + slot * V;
 #pragma unroll
-                    for (int c = 0; c < D / 32; ++c) {
+                    for (int c = 0; c < V / 32; ++c) {
                         uint32_t ob[32];
                         tc_ld32(to + c * 32, ob);
                         tc_ld_wait();
@@ -359,24 +375,28 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                 }
             } else if (ok && has_blocks) {
                 tc_fence_after();
-                const float inv = l > 0.f ? 1.f / l : 0.f;
-                bf16* dst = a.out + (long)(tok0 + t * BQ + r) * a.ldo + (long)head * D;
+                const float inv = inverse_sum(l, m * sl2, a.sinks, head);
+                bf16* dst = a.out + (long)(tok0 + t * BQ + r) * a.ldo + (long)head * a.value_dim;
+                const bf16* gate = a.gate ? a.gate + (long)(tok0 + t * BQ + r) * a.ldg + (long)head * a.value_dim : nullptr;
 #pragma unroll
-                for (int c = 0; c < D / 32; ++c) {
+                for (int c = 0; c < V / 32; ++c) {
                     uint32_t ob[32];
                     tc_ld32(to + c * 32, ob);
                     tc_ld_wait();
                     if (r < rows_t) {
 #pragma unroll
                         for (int k = 0; k < 32; k += 8) {
-                            uint4 v;
-                            __nv_bfloat162 p0 = __floats2bfloat162_rn(__uint_as_float(ob[k]) * inv, __uint_as_float(ob[k + 1]) * inv);
-                            __nv_bfloat162 p1 = __floats2bfloat162_rn(__uint_as_float(ob[k + 2]) * inv, __uint_as_float(ob[k + 3]) * inv);
-                            __nv_bfloat162 p2 = __floats2bfloat162_rn(__uint_as_float(ob[k + 4]) * inv, __uint_as_float(ob[k + 5]) * inv);
-                            __nv_bfloat162 p3 = __floats2bfloat162_rn(__uint_as_float(ob[k + 6]) * inv, __uint_as_float(ob[k + 7]) * inv);
-                            v.x = *reinterpret_cast<uint32_t*>(&p0); v.y = *reinterpret_cast<uint32_t*>(&p1);
-                            v.z = *reinterpret_cast<uint32_t*>(&p2); v.w = *reinterpret_cast<uint32_t*>(&p3);
-                            *reinterpret_cast<uint4*>(dst + c * 32 + k) = v;
+                            if (c * 32 + k >= a.value_dim) continue;      // (zeros beyond the value's width)
+                            float x[8];
+#pragma unroll
+                            for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(ob[k + e]) * inv;
+                            if (gate) {
+                                float g[8];
+                                Pack<bf16>::load(gate + c * 32 + k, g);
+#pragma unroll
+                                for (int e = 0; e < 8; ++e) x[e] *= fx_sigmoid_fast(g[e]);
+                            }
+                            Pack<bf16>::store(dst + c * 32 + k, x);
                         }
                     }
                 }
@@ -398,17 +418,19 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
 // relative to the reference m_c) and the sum of weights l_c; with M = max m_c the result is
 // sum_c o_c 2^((m_c - M) s) / sum_c l_c 2^((m_c - M) s), the runs taken in their order.  A run without visible keys
 // for the row has m_c = -inf and is skipped.  merges: int32 [n, 4] = (first flat token, rows, first part, runs).
-template <int D>
+template <int V>
 __global__ void __launch_bounds__(128) prefill_merge_kernel(const int* __restrict__ merges, const float* __restrict__ part_o,
                                                             const float* __restrict__ part_ml, bf16* __restrict__ out, long ldo,
-                                                            int n_heads, float scale_log2e)
+                                                            int n_heads, float scale_log2e, int value_dim,
+                                                            const float* __restrict__ sinks,
+                                                            const bf16* __restrict__ gate, long ldg)
 {
     fx_pdl_wait();
     const int* mg = merges + (long)blockIdx.x * 4;
     const int tok0 = mg[0], rows = mg[1], part0 = mg[2], runs = mg[3];
     const int head = blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    constexpr int PER = D / 32;   // elements of a row per lane
+    constexpr int PER = V / 32;   // elements of a row per lane
     const int r = blockIdx.z * 4 + warp;   // a warp a row: all of a row's loads are on their way together
     if (r >= rows) return;
     const long slot0 = ((long)part0 * n_heads + head) * (2 * BQ) + r;
@@ -430,14 +452,20 @@ __global__ void __launch_bounds__(128) prefill_merge_kernel(const int* __restric
         const float w = __shfl_sync(0xffffffffu, w_c, c);
         l = fmaf(__shfl_sync(0xffffffffu, l_c, c), w, l);
         if (w == 0.f) continue;    // a run without visible keys for this row wrote no sums
-        const float* src = part_o + (slot0 + c * run_stride) * D + lane * PER;
+        const float* src = part_o + (slot0 + c * run_stride) * V + lane * PER;
 #pragma unroll
         for (int i = 0; i < PER; ++i) acc[i] = fmaf(src[i], w, acc[i]);
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    bf16* dst = out + (long)(tok0 + r) * ldo + (long)head * D + lane * PER;
+    if (lane * PER >= value_dim) return;
+    const float inv = inverse_sum(l, mx * scale_log2e, sinks, head);
+    bf16* dst = out + (long)(tok0 + r) * ldo + (long)head * value_dim + lane * PER;
+    const bf16* g = gate ? gate + (long)(tok0 + r) * ldg + (long)head * value_dim + lane * PER : nullptr;
 #pragma unroll
-    for (int i = 0; i < PER; ++i) dst[i] = __float2bfloat16_rn(acc[i] * inv);
+    for (int i = 0; i < PER; ++i) {
+        float x = acc[i] * inv;
+        if (g) x *= fx_sigmoid_fast(__bfloat162float(g[i]));
+        dst[i] = __float2bfloat16_rn(x);
+    }
 }
 
 bool encode(CUtensorMap* map, const void* ptr, int rank, const cuuint64_t* dims, const cuuint64_t* strides, const cuuint32_t* box)
@@ -450,17 +478,21 @@ bool encode(CUtensorMap* map, const void* ptr, int rank, const cuuint64_t* dims,
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int D>
-int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnArgs& a, dim3 grid, cudaStream_t s)
+template <int D, int V>
+int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnArgs& a, dim3 grid, const int* merges,
+           int n_merges, cudaStream_t s)
 {
-    auto kern = prefill_attention_tc_kernel<D>;
+    auto kern = prefill_attention_tc_kernel<D, V>;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<D>::TOTAL);
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<D, V>::TOTAL);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    fx_launch_pdl(kern, grid, NTHREADS, Smem<D>::TOTAL, s, mq, mk, mv, a);
+    fx_launch_pdl(kern, grid, NTHREADS, Smem<D, V>::TOTAL, s, mq, mk, mv, a);
+    if (n_merges > 0)
+        fx_launch_pdl(prefill_merge_kernel<V>, dim3(n_merges, a.n_heads, 2 * BQ / 4), 128, 0, s, merges, (const float*)a.part_o,
+                      (const float*)a.part_ml, a.out, a.ldo, a.n_heads, a.scale_log2e, a.value_dim, a.sinks, a.gate, a.ldg);
     return fx_launch_status();
 }
 
@@ -469,7 +501,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 // items: int32 [n_items, 8] = (first flat token, rows <= 256, entry index, absolute position of the first row, first
 // key block of 128 positions, end of the key blocks, part or -1, unused), the heavy ones first.  An item with part -1
 // holds every key block its tile sees and writes the tile's output; the items of a tile that was cut write their
-// partial results to part_o [parts, n_heads, 256, head_dim] and part_ml [parts, n_heads, 256, 2] (32-bit), and
+// partial results to part_o [parts, n_heads, 256, value_dim rounded up to 64 or 128] and part_ml [parts, n_heads, 256, 2] (32-bit), and
 // merges: int32 [n_merges, 4] = (first flat token, rows, first part, runs) tells the second kernel which to add up
 // (a tile's runs have consecutive parts, in the order of their keys).
 // q is the fused [tokens, ldq] buffer whose rows start with the query heads; n_tokens its number of rows.
@@ -477,46 +509,46 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 extern "C" int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, const void* k_pages, const void* v_pages,
                                        int n_pages, const int* block_table, int table_width, int page_size,
                                        const int* tiles, int n_tiles, const int* seq_slot, void* out, long ldo,
-                                       int n_heads, int n_kv_heads, int head_dim, int window, float scale, int* status,
+                                       int n_heads, int n_kv_heads, int head_dim, int value_dim, int window, int chunk,
+                                       float scale, const float* sinks, const void* gate, long ldg, int* status,
                                        float* part_o, float* part_ml, const int* merges, int n_merges, void* stream)
 {
     if (n_tiles <= 0) return FX_OK;
     if (n_merges > 0 && (!part_o || !part_ml || !merges || (uintptr_t)part_o % 16)) return FX_ERR_ALIGN;
-    if ((head_dim != 64 && head_dim != 128) || page_size < 64 || page_size % 64 || n_kv_heads <= 0 || n_heads % n_kv_heads)
+    if (head_dim <= 0 || head_dim > 128 || head_dim % 8 || value_dim <= 0 || value_dim > 128 || value_dim % 8 ||
+        page_size < 64 || page_size % 64 || n_kv_heads <= 0 || n_heads % n_kv_heads || chunk < 0 || !(scale > 0.f))
         return FX_ERR_SIZE;
     if (ldq % 8 || ldo % 8 || (uintptr_t)q % 16 || (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16 || (uintptr_t)out % 16)
         return FX_ERR_ALIGN;
+    if (gate && (ldg % 8 || (uintptr_t)gate % 16)) return FX_ERR_ALIGN;
     if (n_tiles > 65535) return FX_ERR_SIZE;
     CUtensorMap mq, mk, mv;
     {
-        cuuint64_t dims[2] = {(cuuint64_t)n_heads * head_dim, (cuuint64_t)n_tokens};
-        cuuint64_t strides[1] = {(cuuint64_t)ldq * 2};
-        cuuint32_t box[2] = {64, 128};
-        if (!encode(&mq, q, 2, dims, strides, box)) return FX_ERR_SIZE;
+        cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)n_heads, (cuuint64_t)n_tokens};
+        cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, (cuuint64_t)ldq * 2};
+        cuuint32_t box[3] = {64, 1, 128};
+        if (!encode(&mq, q, 3, dims, strides, box)) return FX_ERR_SIZE;
     }
-    {
-        cuuint64_t dims[4] = {(cuuint64_t)head_dim, (cuuint64_t)page_size, (cuuint64_t)n_kv_heads, (cuuint64_t)n_pages};
-        cuuint64_t strides[3] = {(cuuint64_t)head_dim * 2, (cuuint64_t)page_size * head_dim * 2,
-                                 (cuuint64_t)n_kv_heads * page_size * head_dim * 2};
+    for (int v = 0; v < 2; ++v) {
+        const int width = v ? value_dim : head_dim;
+        cuuint64_t dims[4] = {(cuuint64_t)width, (cuuint64_t)page_size, (cuuint64_t)n_kv_heads, (cuuint64_t)n_pages};
+        cuuint64_t strides[3] = {(cuuint64_t)width * 2, (cuuint64_t)page_size * width * 2,
+                                 (cuuint64_t)n_kv_heads * page_size * width * 2};
         cuuint32_t box[4] = {64, 64, 1, 1};
-        if (!encode(&mk, k_pages, 4, dims, strides, box) || !encode(&mv, v_pages, 4, dims, strides, box)) return FX_ERR_SIZE;
+        if (!encode(v ? &mv : &mk, v ? v_pages : k_pages, 4, dims, strides, box)) return FX_ERR_SIZE;
     }
     AttnArgs a;
     a.block_table = block_table; a.table_width = table_width; a.page_size = page_size;
     a.tiles = tiles; a.seq_slot = seq_slot; a.out = (bf16*)out; a.ldo = ldo;
-    a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.window = window;
+    a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.window = window; a.chunk = chunk; a.value_dim = value_dim;
+    a.sinks = sinks; a.gate = (const bf16*)gate; a.ldg = ldg;
     a.scale_log2e = scale * 1.4426950408889634f; a.status = status;
     a.part_o = part_o; a.part_ml = part_ml;
     dim3 grid(n_heads, n_tiles);
     cudaStream_t s = (cudaStream_t)stream;
-    const int rc = head_dim == 64 ? launch<64>(mq, mk, mv, a, grid, s) : launch<128>(mq, mk, mv, a, grid, s);
-    if (rc != FX_OK || n_merges <= 0) return rc;
-    dim3 mgrid(n_merges, n_heads, 2 * BQ / 4);
-    if (head_dim == 64)
-        fx_launch_pdl(prefill_merge_kernel<64>, mgrid, 128, 0, s, merges, (const float*)part_o, (const float*)part_ml, (bf16*)out,
-                      ldo, n_heads, a.scale_log2e);
-    else
-        fx_launch_pdl(prefill_merge_kernel<128>, mgrid, 128, 0, s, merges, (const float*)part_o, (const float*)part_ml,
-                      (bf16*)out, ldo, n_heads, a.scale_log2e);
-    return fx_launch_status();
+    if (head_dim <= 64)
+        return value_dim <= 64 ? launch<64, 64>(mq, mk, mv, a, grid, merges, n_merges, s)
+                               : launch<64, 128>(mq, mk, mv, a, grid, merges, n_merges, s);
+    return value_dim <= 64 ? launch<128, 64>(mq, mk, mv, a, grid, merges, n_merges, s)
+                           : launch<128, 128>(mq, mk, mv, a, grid, merges, n_merges, s);
 }

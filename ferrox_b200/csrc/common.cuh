@@ -111,8 +111,7 @@ template <bool FAST>
 __device__ __forceinline__ float fx_clamped_glu(float g, float u, float limit, float alpha) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
-    const float e = FAST ? __expf(-alpha * g) : expf(-alpha * g);
-    return g / (1.0f + e) * (u + 1.0f);
+    return (FAST ? __fdividef(g, 1.0f + __expf(-alpha * g)) : g / (1.0f + expf(-alpha * g))) * (u + 1.0f);
 }
 
 // z * (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) / 2, the tanh form of GELU, written with 1 + tanh(y) = 2 / (1 + e^(-2y)).
@@ -131,6 +130,26 @@ __device__ __forceinline__ float fx_gate(float g, float u, int act, float limit,
     if (act == 3) return fx_gelu_tanh<FAST>(g) * u;
     return (FAST ? __fdividef(g, 1.0f + __expf(-g)) : g / (1.0f + expf(-g))) * u;
 }
+
+// The same over 32 pairs in registers, the choice of the unit made once: x[j] <- act(x[j]) * u[j].
+__device__ __forceinline__ void fx_gate_32(float* x, const uint32_t* u, int act, float limit, float alpha) {
+    if (act == 2) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) x[j] = fx_clamped_glu<true>(x[j], __uint_as_float(u[j]), limit, alpha);
+    } else if (act == 0) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) x[j] = __fdividef(x[j], 1.0f + __expf(-x[j])) * __uint_as_float(u[j]);
+    } else if (act == 1) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) x[j] = fmaxf(x[j], 0.f) * __uint_as_float(u[j]);
+    } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) x[j] = fx_gelu_tanh<true>(x[j]) * __uint_as_float(u[j]);
+    }
+}
+
+// sigmoid(g) with the hardware's exponential and quotient, for the attention kernels' output gates.
+__device__ __forceinline__ float fx_sigmoid_fast(float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); }
 
 // The first key the query at position pos may see: of a window of the last `window` positions (0: no window) and of
 // chunks of `chunk` positions counted from the request's start (0: no chunks), in which a query sees its own chunk only.

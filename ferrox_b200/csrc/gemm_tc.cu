@@ -281,10 +281,10 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_tc_kernel(const __grid_const
                     float x = __uint_as_float(r[j]);
                     if (a.bias) x += bias_s[quad][c * 32 + j];
                     if (GATED && a.bias) u[j] = __float_as_uint(__uint_as_float(u[j]) + bias_up_s[quad][c * 32 + j]);
-                    if (GATED) x = fx_gate<true>(x, __uint_as_float(u[j]), a.act, a.act_limit, a.act_alpha);
-                    else if (a.act) x = fx_unary(x, a.act);     // a plain product with an activation on its result
+                    if (!GATED && a.act) x = fx_unary(x, a.act);     // a plain product with an activation on its result
                     v[j] = x;
                 }
+                if (GATED) fx_gate_32(v, u, a.act, a.act_limit, a.act_alpha);
                 if (fast) {
                     const long row0 = tc.m0 + quad * 32;
                     if (a.c_dtype == FX_F32) {

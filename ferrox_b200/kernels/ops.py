@@ -91,15 +91,15 @@ _SIGNATURES = {
     "fx_softcap": [_P, _L, _F, _P],
     "fx_relu_square": [_P, _I, _L, _I, _I, _P],
     "fx_prefill_attention": [_P, _L, _P, _P, _P, _I, _I, _P, _I, _P, _P, _L, _I, _I, _I, _I, _F, _F, _P],
-    "fx_prefill_attention_tc": [_P, _L, _I, _P, _P, _I, _P, _I, _I, _P, _I, _P, _P, _L, _I, _I, _I, _I, _F, _P, _P, _P,
-                                _P, _I, _P],
+    "fx_prefill_attention_tc": [_P, _L, _I, _P, _P, _I, _P, _I, _I, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I, _I, _F, _P, _P, _L,
+                                _P, _P, _P, _P, _I, _P],
     "fx_router_topk": [_P, _L, _I, _I, _I, _I, _P, _P, _P, _F, _F, _P],
     "fx_moe_align": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _P],
     "fx_gemm_slab_ok": [_I, _I, _I],
     "fx_gemm_slab": [_P, _L, _P, _L, _P, _I, _P, _I, _L, _I, _I, _I, _I, _P, _P],
     "fx_gemm_skinny": [_P, _L, _P, _P, _L, _L, _P, _I, _P, _I, _L, _I, _I, _I, _I, _I, _I, _F, _F, _P, _P, _I, _I, _I, _P],
     "fx_decode_attention": [_P, _L, _P, _P, _I, _I, _P, _I, _I, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _F, _I,
-                            _I, _P, _P, _I, _I, _I, _P, _F, _P],
+                            _I, _P, _P, _I, _I, _I, _P, _F, _P, _P],
     "fx_argmax": [_P, _L, _I, _I, _P, _P],
     "fx_repetition_penalty": [_P, _L, _I, _I, _P, _P, _P, _P],
     "fx_sample": [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P],
@@ -963,10 +963,12 @@ def prefill_ok(q, out, k_pages, head_dim) -> bool:
             and q.stride(0) % 8 == 0 and out.stride(0) % 2 == 0 and q.data_ptr() % 16 == 0 and k_pages.data_ptr() % 16 == 0)
 
 
-def prefill_tc_ok(q, out, k_pages, page_size, head_dim) -> bool:
-    """Whether the tcgen05 prompt attention kernel takes these operands."""
-    return (q.dtype == torch.bfloat16 and k_pages.dtype == torch.bfloat16 and head_dim in (64, 128)
-            and page_size >= 64 and page_size % 64 == 0 and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
+def prefill_tc_ok(q, out, k_pages, page_size, head_dim, value_dim=None, scale=1.0) -> bool:
+    """Whether the tcgen05 prompt attention kernel takes these operands: keys (and values, where their width differs)
+    of up to 128 elements in steps of 8."""
+    widths = (head_dim, value_dim or head_dim)
+    return (q.dtype == torch.bfloat16 and k_pages.dtype == torch.bfloat16 and all(0 < d <= 128 and d % 8 == 0 for d in widths)
+            and scale > 0 and page_size >= 64 and page_size % 64 == 0 and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
             and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0)
 
 
@@ -1009,7 +1011,18 @@ def _prefill_makespan(items, parts: int, n_heads: int, sms: int) -> float:
     return est + (PREFILL_MERGE_COST if parts else 0)
 
 
-def prefill_tc_plan(entries, window, n_heads: int, sms: int = 0, run_blocks: int = -1):
+def prefill_value_width(value_dim: int) -> int:
+    """Elements a value head takes in the tcgen05 prompt attention kernel's scratch."""
+    return 64 if value_dim <= 64 else 128
+
+
+def first_key(pos: int, window=None, chunk=None) -> int:
+    """The first key that the query at ``pos`` may see (``fx_first_key``)."""
+    lo = max(0, pos - int(window) + 1) if window else 0
+    return max(lo, pos // int(chunk) * int(chunk)) if chunk else lo
+
+
+def prefill_tc_plan(entries, window, n_heads: int, sms: int = 0, run_blocks: int = -1, chunk=None):
     """The work items of the tcgen05 prompt attention kernel for a step.  ``entries``: (tokens, first position) of
     each entry, in the order of the flattened batch.  A tile is up to 256 queries of one entry; it sees the key blocks
     (of 128 positions) from its first query's first visible key to its last query's own.  Tiles with many key blocks
@@ -1022,12 +1035,11 @@ def prefill_tc_plan(entries, window, n_heads: int, sms: int = 0, run_blocks: int
     import numpy as np
 
     sms = sms or sm_count()
-    W = int(window or 0)
     tiles, flat = [], 0
     for b, (n, start) in enumerate(entries):
         for i in range(0, n, WIDE_PREFILL_TILE):
             rows, pos0 = min(WIDE_PREFILL_TILE, n - i), start + i
-            first = (max(0, pos0 - W + 1) if W > 0 else 0) // PREFILL_KEY_BLOCK
+            first = first_key(pos0, window, chunk) // PREFILL_KEY_BLOCK
             end = (pos0 + rows - 1) // PREFILL_KEY_BLOCK + 1
             tiles.append((flat + i, rows, b, pos0, first, end))
         flat += n
@@ -1048,10 +1060,12 @@ def prefill_tc_plan(entries, window, n_heads: int, sms: int = 0, run_blocks: int
 
 
 def prefill_attention_tc(q, k_pages, v_pages, block_table, page_size, items, seq_slot, out, n_heads, n_kv_heads,
-                         head_dim, window, scale, status=None, stream=None, merges=None, part_o=None, part_ml=None):
-    """Flash attention of prompt portions on the tcgen05 tensor cores (bfloat16, head_dim 64 or 128, pages of a
-    multiple of 64 positions).  ``items``, ``merges``: device copies of what :func:`prefill_tc_plan` returns;
-    ``part_o`` float32 [parts, n_heads, 256, head_dim] and ``part_ml`` float32 [parts, n_heads, 256, 2]: scratch for the
+                         head_dim, window, scale, status=None, stream=None, merges=None, part_o=None, part_ml=None,
+                         value_dim=None, chunk=None, sinks=None, gate=None):
+    """Flash attention of prompt portions on the tcgen05 tensor cores (bfloat16, keys and values of up to 128 elements
+    in steps of 8, pages of a multiple of 64 positions).  ``value_dim``, ``chunk``, ``sinks``, ``gate``: as
+    :func:`paged_attention_ex`.  ``items``, ``merges``: device copies of what :func:`prefill_tc_plan` returns;
+    ``part_o`` float32 [parts, n_heads, 256, :func:`prefill_value_width`] and ``part_ml`` float32 [parts, n_heads, 256, 2]: scratch for the
     tiles that were cut into runs of key blocks (a second kernel adds the runs up)."""
     global _launches
     n_merges = merges.shape[0] if merges is not None else 0
@@ -1059,7 +1073,8 @@ def prefill_attention_tc(q, k_pages, v_pages, block_table, page_size, items, seq
         _launches += 1
     call("fx_prefill_attention_tc", _ptr(q), _rows(q), q.shape[0], _ptr(k_pages), _ptr(v_pages), k_pages.shape[0],
          _ptr(block_table), block_table.shape[1], page_size, _ptr(items), items.shape[0], _ptr(seq_slot), _ptr(out),
-         _rows(out), n_heads, n_kv_heads, head_dim, int(window or 0), float(scale), _ptr(status),
+         _rows(out), n_heads, n_kv_heads, head_dim, int(value_dim or head_dim), int(window or 0), int(chunk or 0), float(scale),
+         _ptr(sinks), _ptr(gate), _rows(gate) if gate is not None else 0, _ptr(status),
          _ptr(part_o) if n_merges else None, _ptr(part_ml) if n_merges else None, _ptr(merges) if n_merges else None,
          n_merges, stream if stream is not None else stream_ptr())
     return out
@@ -1196,11 +1211,31 @@ def decode_store_ok(qkv, k_pages, head_dim: int, page_size: int) -> bool:
             and qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0 and k_pages.data_ptr() % 16 == 0)
 
 
+class DecodeExtras(ctypes.Structure):
+    """Options of the decode attention kernel that streams pages by TMA (csrc/api.h): ``chunk``, ``sinks``, ``gate`` as
+    :func:`paged_attention_ex`; with ``store_new`` the first ``rot`` elements of a head are rotated (0: all of it) and
+    the stored value is (1 - lam) v + lam v_first as :func:`rotary_mix_store` says."""
+
+    _fields_ = [("chunk", c_int), ("rot", c_int), ("sinks", c_void_p), ("gate", c_void_p), ("ldg", c_long),
+                ("v_first", c_void_p), ("ld_first", c_long), ("lam", c_float)]
+
+    @classmethod
+    def of(cls, chunk=None, sinks=None, gate=None, rot=0, v_first=None, lam=0.0):
+        if sinks is not None and sinks.dtype != torch.float32:
+            raise KernelError("decode_attention: one 32-bit sink per head")
+        for t in (gate, v_first):
+            if t is not None and t.dtype != torch.bfloat16:
+                raise KernelError("decode_attention: the gate and the other layer's values are bfloat16 rows")
+        return cls(int(chunk or 0), int(rot), _ptr(sinks), _ptr(gate), _rows(gate) if gate is not None else 0,
+                   _ptr(v_first), _rows(v_first) if v_first is not None else 0, float(lam))
+
+
 def decode_attention(q, k_pages, v_pages, block_table, page_size, positions, token_seq, seq_slot, out, n_heads,
                      n_kv_heads, head_dim, window, scale, split_len, n_splits, part_acc, part_ml, status=None,
                      counters=None, stream=None, fresh_positions=0, store_new=False, write_pages=True, cos_sin=None,
-                     softcap=None):
-    """``softcap`` c: the scaled scores pass through c * tanh(s / c) (the kernel that streams pages by TMA does not
+                     softcap=None, extras=None):
+    """``extras`` (:class:`DecodeExtras` or None): options of the kernel that streams pages by TMA, which has to be the
+    one that runs (:func:`decode_store_ok`).  ``softcap`` c: the scaled scores pass through c * tanh(s / c) (the kernel that streams pages by TMA does not
     take one: the call goes to the others).  ``counters``: zeroed int32 scratch that the call leaves zeroed, at least tokens x ceil(group / 16) x kv heads;
     with it the kernel that streams pages by TMA merges the key ranges itself (one kernel instead of two).
     ``fresh_positions``: 0 assumes nothing about the kernel launched just before on the stream.  N > 0 promises that
@@ -1225,7 +1260,7 @@ def decode_attention(q, k_pages, v_pages, block_table, page_size, positions, tok
          _ptr(block_table), block_table.shape[1], page_size, _ptr(positions), _ptr(token_seq), _ptr(seq_slot),
          _ptr(out), _rows(out), _ptr(part_acc), _ptr(part_ml), T, n_heads, n_kv_heads, head_dim, int(window or 0),
          float(scale), split_len, n_splits, _ptr(status), _ptr(counters), int(fresh_positions), int(store_new),
-         int(write_pages), _ptr(cos_sin), float(softcap or 0.0), stream if stream is not None else stream_ptr())
+         int(write_pages), _ptr(cos_sin), float(softcap or 0.0), ctypes.byref(extras) if extras is not None else None, stream if stream is not None else stream_ptr())
     return out
 
 

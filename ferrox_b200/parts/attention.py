@@ -53,13 +53,14 @@ def query_tiles(batch, rows: int) -> torch.Tensor:
     return t
 
 
-def prefill_tc_plan(batch, window, n_heads: int):
+def prefill_tc_plan(batch, window, n_heads: int, chunk=None):
     """This step's work items for the tcgen05 prompt attention kernel (``ops.prefill_tc_plan``) on the device: made
-    once a step for each window and shared by the layers that have it."""
-    key = ("attention tcgen05 items", window, n_heads)
+    once a step for each window and chunk and shared by the layers that have it."""
+    key = ("attention tcgen05 items", window, n_heads, chunk)
     plan = batch.shared.get(key)
     if plan is None:
-        items, merges, parts = ops.prefill_tc_plan([(len(e.tokens), e.start) for e in batch.entries], window, n_heads)
+        items, merges, parts = ops.prefill_tc_plan([(len(e.tokens), e.start) for e in batch.entries], window, n_heads,
+                                                   chunk=chunk)
         both = torch.from_numpy(np.concatenate([items.reshape(-1), merges.reshape(-1)])).to(batch.token_ids.device)
         plan = (both[:items.size].view(-1, 8), both[items.size:].view(-1, 4) if merges.size else None, parts)
         batch.shared[key] = plan
@@ -292,14 +293,24 @@ class GqaAttention(Mixer):
         qkv_width = self.q_size + self.kv_size + self.v_size
         qkv = self.rt.empty(T, qkv_width + (self.o_size if self.gate_name else 0))
         ops.linear(x, self.w_qkv, qkv, bias=self.b_qkv, status=batch.status, stream=batch.stream, after_short_kernel=True)
+        gate = qkv[:, qkv_width:] if self.gate_name else None
+        # keys and values of one width, no distance bias, no kept positions: the kernels that stream pages by TMA
+        direct = V == D and not self.slopes_spec and not self.keep_first and qkv.dtype == torch.bfloat16
+        few = batch.max_new <= DECODE_ATTENTION_MAX_NEW
+        by_tma = direct and few and ops.decode_store_ok(qkv, cache.k, D, cache.page_size)
+        in_kernel = False
+        first = self._values_of_first_layer(qkv, qkv_width, batch)
         if self.rotates or self.mix:
-            first = self._values_of_first_layer(qkv, qkv_width, batch)
-            ops.rotary_mix_store(qkv, batch.positions, batch.token_seq, batch.seq_slot,
-                                 self.position.table(batch) if self.rotates else None,
-                                 self.position.rotary_dim if self.rotates else 0,
-                                 self.position.pairing if self.rotates else ops.PAIR_HALVES, cache.k, cache.v,
-                                 cache.block_table, cache.page_size, s.n_heads, s.n_kv_heads, D, V, v_first=first,
-                                 lam=self.lam, write_cache=cache.writes, status=batch.status, stream=batch.stream)
+            cos_sin = self.position.table(batch) if self.rotates else None
+            rot = self.position.rotary_dim if self.rotates else 0
+            pairing = self.position.pairing if self.rotates else ops.PAIR_HALVES
+            in_kernel = (by_tma and batch.max_new == 1 and T <= ROTARY_IN_DECODE_KERNEL_MAX_TOKENS
+                         and pairing == ops.PAIR_HALVES)
+            if not in_kernel:
+                ops.rotary_mix_store(qkv, batch.positions, batch.token_seq, batch.seq_slot, cos_sin, rot, pairing, cache.k,
+                                     cache.v, cache.block_table, cache.page_size, s.n_heads, s.n_kv_heads, D, V,
+                                     v_first=first, lam=self.lam, write_cache=cache.writes, status=batch.status,
+                                     stream=batch.stream)
         else:
             eps = self.qk_norm[2] if self.qk_norm else 0.0
             ops.qk_norm_store(qkv, batch.positions, batch.token_seq, batch.seq_slot, self.q_norm_w, self.k_norm_w, eps,
@@ -307,16 +318,50 @@ class GqaAttention(Mixer):
                               s.n_kv_heads, D, V, write_cache=cache.writes, status=batch.status, stream=batch.stream,
                               value_norm_eps=self.value_norm_eps)
         attn = self.rt.empty(T, self.o_size)
-        general_attention(qkv, qkv.stride(0), D, cache.k, cache.v, D, V, attn, attn.stride(0), V, batch, cache,
-                          s.n_heads, s.n_kv_heads, D, V, s.window, self.scale, self.slopes, self.rt,
-                          keep_first=self.keep_first, sinks=self.sinks, chunk=self.chunk,
-                          gate=qkv[:, qkv_width:] if self.gate_name else None)
+        if by_tma:
+            extras = ops.DecodeExtras.of(self.chunk, self.sinks, gate, *((rot, first, self.lam) if in_kernel else ()))
+            self._decode_by_tma(qkv, attn, batch, cache, in_kernel, cos_sin if in_kernel else None, extras)
+        elif (not few and not self.slopes_spec and not self.keep_first
+              and ops.prefill_tc_ok(qkv, attn, cache.k, cache.page_size, D, V, self.scale)):
+            items, merges, parts = prefill_tc_plan(batch, s.window, s.n_heads, self.chunk)
+            part_o = part_ml = None
+            if parts:
+                part_o = self.rt.empty(parts, s.n_heads, ops.WIDE_PREFILL_TILE, ops.prefill_value_width(V), dtype=torch.float32)
+                part_ml = self.rt.empty(parts, s.n_heads, ops.WIDE_PREFILL_TILE, 2, dtype=torch.float32)
+            ops.prefill_attention_tc(qkv, cache.k, cache.v, cache.block_table, cache.page_size, items, batch.seq_slot, attn,
+                                     s.n_heads, s.n_kv_heads, D, s.window, self.scale, status=batch.status,
+                                     stream=batch.stream, merges=merges, part_o=part_o, part_ml=part_ml, value_dim=V,
+                                     chunk=self.chunk, sinks=self.sinks, gate=gate)
+        else:
+            general_attention(qkv, qkv.stride(0), D, cache.k, cache.v, D, V, attn, attn.stride(0), V, batch, cache,
+                              s.n_heads, s.n_kv_heads, D, V, s.window, self.scale, self.slopes, self.rt,
+                              keep_first=self.keep_first, sinks=self.sinks, chunk=self.chunk, gate=gate)
         ops.linear(attn, self.w_o, out, accumulate=accumulate, status=batch.status, stream=batch.stream,
                    after_short_kernel=True)
 
+    def _decode_by_tma(self, qkv, attn, batch, cache, store_new, cos_sin, extras):
+        """Steps of few tokens a request: the kernel that streams pages by TMA, every token's keys cut into runs."""
+        s, T = self.spec, qkv.shape[0]
+        per_sm = ops.decode_tma_blocks_per_sm(qkv.dtype, s.head_dim, cache.page_size)
+        reach = cache.block_table.shape[1] * cache.page_size
+        for limit in (s.window, self.chunk):
+            if limit is not None:
+                reach = min(reach, (limit + 63) // 64 * 64 + 64)
+        split_len, n_splits = ops.decode_split_plan(
+            T, s.n_kv_heads * -(-(s.n_heads // s.n_kv_heads) // 16), reach, per_sm, single_is_final=True,
+            run_latency=ops.DECODE_RUN_LATENCY)
+        part_acc = self.rt.empty(T, s.n_heads, n_splits, s.head_dim, dtype=torch.float32)
+        part_ml = self.rt.empty(T, s.n_heads, n_splits, 2, dtype=torch.float32)
+        ops.decode_attention(
+            qkv, cache.k, cache.v, cache.block_table, cache.page_size, batch.positions, batch.token_seq, batch.seq_slot,
+            attn, s.n_heads, s.n_kv_heads, s.head_dim, s.window, self.scale, split_len, n_splits, part_acc, part_ml,
+            status=batch.status, counters=self._range_counters, stream=batch.stream, fresh_positions=batch.max_new,
+            store_new=store_new, write_pages=cache.writes, cos_sin=cos_sin, extras=extras)
+
     def _values_of_first_layer(self, qkv, qkv_width, batch):
         """The step's rows of v_first for a layer that mixes its values with them (None for any other).  The source
-        layer's own rows of its fused product stay as projected: it leaves a view of them for the layers behind it."""
+        layer's own value rows of its fused product stay as projected: it leaves a view of them for the layers behind
+        it."""
         if not self.mix:
             return None
         key = ("values of the first layer", self.mix.group)

@@ -878,15 +878,15 @@ def test_prefill_attention_tcgen05(case, run_blocks):
 
 def test_prefill_attention_tcgen05_refuses_other_sizes():
     o = ops()
-    q = rnd(4, 3 * 48, dtype=torch.bfloat16)
-    kp = torch.zeros(2, 1, 64, 48, dtype=torch.bfloat16, device=DEV)
-    out = torch.zeros(4, 48, dtype=torch.bfloat16, device=DEV)
-    assert not o.prefill_tc_ok(q, out, kp, 64, 48)
+    q = rnd(4, 3 * 136, dtype=torch.bfloat16)
+    kp = torch.zeros(2, 1, 64, 136, dtype=torch.bfloat16, device=DEV)
+    out = torch.zeros(4, 136, dtype=torch.bfloat16, device=DEV)
+    assert not o.prefill_tc_ok(q, out, kp, 64, 136)
     tiles = torch.tensor([[0, 4, 0, 0, 0, 1, -1, 0]], dtype=torch.int32, device=DEV)
     table = torch.zeros(1, 2, dtype=torch.int32, device=DEV)
     slots = torch.zeros(1, dtype=torch.int32, device=DEV)
     with pytest.raises(o.KernelError):
-        o.prefill_attention_tc(q, kp, kp, table, 64, tiles, slots, out, 1, 1, 48, 0, 1.0)
+        o.prefill_attention_tc(q, kp, kp, table, 64, tiles, slots, out, 1, 1, 136, 0, 1.0)
 
 
 def test_gemm_skinny_transposed_store_and_linear_picks_it_for_narrow_outputs():
