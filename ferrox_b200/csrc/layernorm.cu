@@ -85,6 +85,22 @@ template <> struct Row<bf16, 8> : Pack<bf16> {};
 
 constexpr int RMS_THREADS = 512;   // at most
 
+// N weights of either element type (N > 1: 16-byte aligned vectors of them)
+template <int N> __device__ __forceinline__ void load_weights(const void* w, int dtype, int i, float* o) {
+    if (N == 1) { o[0] = load_any(w, dtype, i); return; }
+    if (dtype == FX_F32) {
+#pragma unroll
+        for (int e = 0; e + 3 < N; e += 4) Pack<float>::load(reinterpret_cast<const float*>(w) + i + e, o + e);
+    } else {
+#pragma unroll
+        for (int e = 0; e + 3 < N; e += 4) {
+            const uint2 t = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(w) + i + e);
+            o[e] = __uint_as_float(t.x << 16); o[e + 1] = __uint_as_float(t.x & 0xffff0000u);
+            o[e + 2] = __uint_as_float(t.y << 16); o[e + 3] = __uint_as_float(t.y & 0xffff0000u);
+        }
+    }
+}
+
 struct RmsArgs {
     float* h; const void* y;
     const int* place; const float* weight; int top_k;         // place == nullptr: z is the token's own row of y
@@ -98,6 +114,13 @@ template <typename T, typename OT, int N, int CH>
 __global__ void __launch_bounds__(RMS_THREADS) rms_residual_kernel(RmsArgs a)
 {
     __shared__ float scratch[33];
+    // a thread with one item holds its weights from before the wait for the kernel before this one (which wrote none)
+    constexpr bool EARLY = CH == 1;
+    float wp[N], wn[N];
+    if (EARLY && (int)threadIdx.x * N < a.hidden) {
+        load_weights<N>(a.w_post, a.wp_dtype, threadIdx.x * N, wp);
+        if (a.w_next) load_weights<N>(a.w_next, a.wn_dtype, threadIdx.x * N, wn);
+    }
     fx_pdl_wait();
     const int t = blockIdx.x;
     const T* y = reinterpret_cast<const T*>(a.y);
@@ -120,6 +143,7 @@ __global__ void __launch_bounds__(RMS_THREADS) rms_residual_kernel(RmsArgs a)
         if (a.place) {
 #pragma unroll
             for (int e = 0; e < N; ++e) z[c][e] = 0.f;
+#pragma unroll 4
             for (int k = 0; k < a.top_k; ++k) {
                 const long r = a.place[(long)t * a.top_k + k];
                 const float w = a.weight ? a.weight[(long)t * a.top_k + k] : 1.f;
@@ -147,9 +171,10 @@ __global__ void __launch_bounds__(RMS_THREADS) rms_residual_kernel(RmsArgs a)
     for (int c = 0; c < CH; ++c) {
         const int i = (c * blockDim.x + threadIdx.x) * N;
         if (i >= a.hidden) continue;
+        if (!EARLY) load_weights<N>(a.w_post, a.wp_dtype, i, wp);
 #pragma unroll
         for (int e = 0; e < N; ++e) {
-            hv[c][e] += z[c][e] * r * load_any(a.w_post, a.wp_dtype, i + e);
+            hv[c][e] += z[c][e] * r * wp[e];
             ss = fmaf(hv[c][e], hv[c][e], ss);
         }
         if (N == 1) hr[i] = hv[c][0];
@@ -166,9 +191,10 @@ __global__ void __launch_bounds__(RMS_THREADS) rms_residual_kernel(RmsArgs a)
     for (int c = 0; c < CH; ++c) {
         const int i = (c * blockDim.x + threadIdx.x) * N;
         if (i >= a.hidden) continue;
+        if (!EARLY) load_weights<N>(a.w_next, a.wn_dtype, i, wn);
         float v[N];
 #pragma unroll
-        for (int e = 0; e < N; ++e) v[e] = hv[c][e] * rn * load_any(a.w_next, a.wn_dtype, i + e);
+        for (int e = 0; e < N; ++e) v[e] = hv[c][e] * rn * wn[e];
         if (N == 1) o[i] = from_f32<OT>(v[0]);
         else if (sizeof(OT) == 4) {
 #pragma unroll
@@ -243,7 +269,7 @@ extern "C" int fx_rmsnorm_residual(float* h, const void* y, int y_dtype, const i
     a.eps_next = eps_next; a.x_out = x_out; a.hidden = hidden;
     const int vw = y_dtype == FX_F32 ? 4 : 8;
     const bool vec = hidden % vw == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)shared % 16 == 0 &&
-                     (uintptr_t)x_out % 16 == 0;
+                     (uintptr_t)x_out % 16 == 0 && (uintptr_t)w_post % 16 == 0 && (uintptr_t)w_next % 16 == 0;
     const int items = vec ? hidden / vw : hidden;
     // few rows (a decode step): a block's trips through its row are the kernel's time, so an item a thread
     int nt = 64;

@@ -85,7 +85,7 @@ def attention(m, W, p, h, first):
     if rot and rot.get("dims"):
         q, k = rotate_halves(q, rot["dims"], rot["base"]), rotate_halves(k, rot["dims"], rot["base"])
     if first is not None:
-        v = mixed_values(v, first, W[p + "vmix"])
+        v = mixed_values(v, first.reshape(v.shape), W[p + "vmix"])    # (element by element of the rows [kv head][vdim])
     q, k, v = _r(q), _r(k), _r(v)
     mask = chunk_mask(n, m["mask"]["size"] if m.get("mask") else None)
     o = torch.zeros(n, H, V, dtype=h.dtype)
