@@ -110,12 +110,12 @@ struct RmsArgs {
     void* x_out; int hidden;
 };
 
-template <typename T, typename OT, int N, int CH>
-__global__ void __launch_bounds__(RMS_THREADS) rms_residual_kernel(RmsArgs a)
+// EARLY (steps of few rows; CH = 1): a thread holds its weights from before the wait for the kernel before this one (which
+// wrote none); with many rows the registers are worth more as blocks an SM holds.
+template <typename T, typename OT, int N, int CH, bool EARLY>
+__global__ void __launch_bounds__(RMS_THREADS, EARLY ? 1 : (N * CH <= 4 ? 3 : N * CH <= 16 ? 2 : 1)) rms_residual_kernel(RmsArgs a)
 {
     __shared__ float scratch[33];
-    // a thread with one item holds its weights from before the wait for the kernel before this one (which wrote none)
-    constexpr bool EARLY = CH == 1;
     float wp[N], wn[N];
     if (EARLY && (int)threadIdx.x * N < a.hidden) {
         load_weights<N>(a.w_post, a.wp_dtype, threadIdx.x * N, wp);
@@ -280,7 +280,10 @@ extern "C" int fx_rmsnorm_residual(float* h, const void* y, int y_dtype, const i
     if (ch > max_ch) return FX_ERR_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     const bool out32 = !w_next || x_dtype == FX_F32;
-#define FX_GO(T, OT, N, CH) fx_launch_pdl(rms_residual_kernel<T, OT, N, CH>, n_rows, nt, 0, s, a)
+    const bool early = ch <= 1 && n_rows < 256;
+#define FX_GO(T, OT, N, CH)                                                                                          \
+    do { if (early) fx_launch_pdl(rms_residual_kernel<T, OT, N, CH, CH == 1>, n_rows, nt, 0, s, a);                 \
+         else fx_launch_pdl(rms_residual_kernel<T, OT, N, CH, false>, n_rows, nt, 0, s, a); } while (0)
 #define FX_CH(T, OT, N)                                                                                              \
     do { if (ch <= 1) FX_GO(T, OT, N, 1); else if (ch <= 2) FX_GO(T, OT, N, 2); else if (ch <= 4) FX_GO(T, OT, N, 4); \
          else if (ch <= 8) FX_GO(T, OT, N, (N == 8 ? 4 : 8)); else FX_GO(T, OT, N, (N == 1 ? 16 : 4)); } while (0)

@@ -76,8 +76,6 @@ class GqaAttention(Mixer):
     def __init__(self, spec):
         super().__init__(spec)
         s = spec
-        if s.head_dim % 2 or s.head_dim > 256:
-            raise ValueError(f"head_dim={s.head_dim}: must be even and at most 256")
         if s.window is not None and s.window < 1:
             raise ValueError(f"window={s.window}: a window holds at least the query's own position")
         if s.n_heads % s.n_kv_heads:
@@ -107,6 +105,12 @@ class GqaAttention(Mixer):
                             or self.gate_name or self.chunk or self.sink_name or self.mix)
         # in the general form a rotary part's tables serve the kernel that also mixes the values (rotary_mix_store)
         self.rotates = self.general and s.position is not None and not isinstance(s.position, NoPositionSpec)
+        if self.general:
+            if s.head_dim > ops.ATTENTION_MAX_KEY_DIM or self.value_dim > ops.ATTENTION_MAX_VALUE_DIM:
+                raise ValueError(f"head_dim={s.head_dim}, value_dim={self.value_dim}: at most {ops.ATTENTION_MAX_KEY_DIM} and "
+                                 f"{ops.ATTENTION_MAX_VALUE_DIM}")
+        elif s.head_dim % 2 or s.head_dim > 256:
+            raise ValueError(f"head_dim={s.head_dim}: must be even and at most 256")
         self.v_size = s.n_kv_heads * self.value_dim
         self.o_size = s.n_heads * self.value_dim
         if self.general:
