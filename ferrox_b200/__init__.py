@@ -13,6 +13,7 @@ from .models import bobepel as _bobepel  # noqa: F401  (registers the architectu
 from .models import sesuzen as _sesuzen  # noqa: F401  (registers the architecture)
 from .models import zanezen as _zanezen  # noqa: F401  (registers the architecture)
 from .models import balelorn as _balelorn  # noqa: F401  (registers the architecture)
+from .models import dubazen as _dubazen  # noqa: F401  (registers the architecture)
 from .parts.base import register_part  # noqa: F401
 from .weights.loader import WeightsError  # noqa: F401
 from .weights.random_init import write_random_model  # noqa: F401

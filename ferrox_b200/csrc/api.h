@@ -52,8 +52,9 @@ int fx_paged_attention_ex(const void* q, long ldq, long ldqh, const void* k_page
                           const int* token_seq, const int* seq_slot, void* out, long ldo, long ldoh, int n_tokens,
                           int n_heads, int n_kv_heads, int key_dim, int value_dim, int window, float scale, float softcap,
                           const float* slopes, int keep_first, const float* sinks, int value_share, int chunk,
-                          const void* gate, long ldg, void* stream);
-// chunk > 0: a query sees the keys of its own chunk of that many positions only.  gate (optional, token rows of n_heads *
+                          const void* gate, long ldg, const float* turn, void* stream);
+// turn (optional, [tokens][value_dim / 2] (cos, sin)): pair (2m, 2m + 1) of every head's result is turned by minus that
+// angle, before the gate.  chunk > 0: a query sees the keys of its own chunk of that many positions only.  gate (optional, token rows of n_heads *
 // value_dim): the result is multiplied by sigmoid(gate).
 // sinks (optional, one per head): exp(sinks[h]) joins the softmax's denominator once.  value_share >= 1: that many
 // consecutive key heads read one value head (the value pages hold n_kv_heads / value_share heads).
@@ -66,13 +67,14 @@ int fx_general_attention(const void* q, long ldq, long ldqh, const void* k_pages
                          const int* token_seq, const int* seq_slot, const int* items, int n_items, void* out, long ldo,
                          long ldoh, int n_heads, int n_kv_heads, int key_dim, int value_dim, int window, float scale,
                          const float* slopes, int n_splits, float* part_o, float* part_ml, int keep_first, float softcap,
-                         const float* sinks, int value_share, int chunk, const void* gate, long ldg, void* stream);
+                         const float* sinks, int value_share, int chunk, const void* gate, long ldg,
+                         const float* turn, void* stream);
 
 int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                             const int* block_table, int table_width, int page_size, const int* items, int n_items,
                             const int* seq_slot, void* out, long ldo, int n_heads, int n_kv_heads, int head_dim, int value_dim,
-                            int window, int chunk, float scale, const float* sinks, const void* gate, long ldg, int* status, float* part_o, float* part_ml, const int* merges,
-                            int n_merges, void* stream);
+                            int window, int chunk, float scale, const float* sinks, const void* gate, long ldg, const float* turn,
+                            int* status, float* part_o, float* part_ml, const int* merges, int n_merges, void* stream);
 int fx_prefill_attention(const void* q, long ldq, const void* k_pages, const void* v_pages, const int* block_table,
                          int table_width, int page_size, const int* tiles, int n_tiles, const int* seq_slot, void* out,
                          long ldo, int n_heads, int n_kv_heads, int head_dim, int window, float scale, float softcap,
@@ -161,6 +163,7 @@ typedef struct DecodeExtras {
     const void* v_first;     // store_new: the value that is stored is (1 - lambda) v + lambda v_first, v_first token
     long ld_first;           //            rows of n_kv_heads * head_dim
     float lambda;
+    const float* turn;       // [tokens][head_dim / 2] (cos, sin): pair (2m, 2m + 1) of the result turned back, before the gate
 } DecodeExtras;
 
 int fx_decode_split_tma(const void* q, long ldq, const void* k_pages, const void* v_pages, int n_pages,
@@ -194,6 +197,12 @@ int fx_qk_norm_store(void* qkv, int dtype, long ld, const int* positions, const 
                      const void* wq, const void* wk, int w_dtype, float eps, float temp_coef, int temp_every, void* k_pages,
                      void* v_pages, const int* block_table, int table_width, int page_size, int n_tokens, int n_heads,
                      int n_kv_heads, int key_dim, int value_dim, int write_cache, int* status, float v_eps, void* stream);
+// the first rot elements of every q and k head turned, then (eps >= 0) each divided by its root mean square; values
+// turned on neighbouring pairs by v_cos_sin (optional); k and v into their pages, q in place
+int fx_rotary_norm_store(void* qkv, int dtype, long ld, const int* positions, const int* token_seq, const int* seq_slot,
+                         const float* cos_sin, int rot, int pairing, float eps, const float* v_cos_sin, void* k_pages,
+                         void* v_pages, const int* block_table, int table_width, int page_size, int n_tokens, int n_heads,
+                         int n_kv_heads, int key_dim, int value_dim, int write_cache, int* status, void* stream);
 int fx_latent_prep(void* q, long ldq, const void* dkv, long ld_dkv, int dtype, const int* positions,
                    const int* token_seq, const int* seq_slot, const void* wc, int w_dtype, float eps, const float* cos_sin,
                    int rot_dims, void* q_plain, void* q_full, void* pages, const int* block_table, int table_width,
@@ -266,7 +275,8 @@ int fx_general_delta_scan(const float* r, long ldr, const float* k, long ldk, co
 // update_tail: every entry brings exactly one token and the kernel moves the tail on itself.
 int fx_input_conv(const void* x, int dtype, long ldx, const void* w, int w_dtype, int taps, float* tail,
                   const int* token_seq, const int* seq_slot, void* out, long ldo, int n_tokens, int channels,
-                  int update_tail, int add_input, void* stream);   // add_input 0: out[t] = the sum alone
+                  int update_tail, int add_input, const void* bias, int b_dtype, int act, void* stream);
+// add_input 0: the sum alone; bias (optional, [channels]) added to it; act 1: SiLU of the result
 // out[t] = table[ids[t]] + pos_table[positions[t]] in 32 bits; status 1: an id outside the vocabulary, 4: a position
 // outside the table.
 int fx_embed_pos(const void* table, int dtype, const int* ids, const void* pos_table, int pos_dtype, const int* positions,
@@ -299,6 +309,47 @@ int fx_conv_rotary_store(const void* proj, int dtype, long ldp, const void* w, i
                          int* status, void* stream);
 int fx_diff_combine(const void* attn, long lda, void* out, long ldo, int dtype, int n_tokens, int n_heads, int group,
                     int value_dim, float lambda, float eps, float post, void* stream);
+
+// A residual of several streams [token][stream][hidden], 32-bit (streams.cu): see there.  write 0: the streams stay as
+// they are and coef[j][0] weighs result j in what is read.
+#define FX_MAX_STREAMS 8
+typedef struct StreamStep {
+    float* streams;
+    const int* rows;           // (optional, write 0) the tokens that are read, one a block
+    const float* y[3];         // n_terms results, [tokens][hidden]
+    const void* expert_rows;   // (with place) rows in expert order, [.][hidden]
+    const int* place;          // [tokens][top_k] row of each of the token's experts
+    const float* weight;       // [tokens][top_k] (null: 1)
+    const void* shared;        // (optional) [tokens][hidden], added with weight 1 or sigmoid(shared_gate)
+    const float* shared_gate; long gate_ld;
+    const void* w;             // (with x_out) [hidden] norm weight
+    void* x_out;               // (optional) [rows][hidden] = rms(u) * w
+    int expert_dtype, w_dtype, x_dtype, top_k, n_terms, write, hidden;
+    float eps;
+    float mix[FX_MAX_STREAMS][FX_MAX_STREAMS];   // [from][to]
+    float coef[4][FX_MAX_STREAMS];               // of y[0], y[1], y[2] and the experts' sum, for every stream
+    float in[FX_MAX_STREAMS];
+} StreamStep;
+int fx_stream_step(const StreamStep* step, int n_streams, int n_rows, void* stream);
+int fx_embed_streams(const void* table, int dtype, const int* ids, float* out, int n_tokens, int hidden, int vocab,
+                     int streams, float scale, int* status, void* stream);
+
+// Linear attention with a decay per key channel (channel_decay.cu): alpha = sigmoid(w2 . low + bias)^(1/tau), then over
+// every entry's tokens in order S <- diag(alpha) S + k v^T, out = q_scale S^T q; state [slots, H, D(key), V] 32-bit.
+int fx_channel_decay_prep(const float* low, long ldl, const void* w2, int w2_dtype, const void* bias, int b_dtype,
+                          float inv_tau, float* alpha, int n_tokens, int channels, int rank, void* stream);
+int fx_channel_decay_scan(const float* q, long ldq, const float* k, long ldk, const float* v, long ldv, const float* alpha,
+                          float q_scale, float* state, float* out, long ldo, const int* token_seq, const int* seq_slot,
+                          int n_tokens, int n_entries, int H, int D, int V, void* stream);
+
+// Selective state space (selective_scan.cu): dt = softplus(dt + dt_bias), S[c, n] <- exp(dt A) S + dt x B_n,
+// out = (sum_n S C_n + D x) silu(z), A = -exp(A_log); state [slots, inner, n_state] 32-bit.
+int fx_selective_scan(const float* dt, long ldt, const void* dt_bias, int db_dtype, const void* x, long ldx, const void* z,
+                      long ldz, int dtype, const float* bc, long ldbc, const float* a_log, const float* d_skip,
+                      float* state, void* out, long ldo, const int* token_seq, const int* seq_slot, int n_tokens,
+                      int n_entries, int inner, int n_state, void* stream);
+// out row = [hi | lo] in bfloat16, hi + lo = x to 16 bits of mantissa; each half `pad` columns wide, zeros beyond n
+int fx_split_rows(const float* x, long ldx, void* out, long ldo, int n_tokens, int n, int pad, void* stream);
 
 #ifdef __cplusplus
 }

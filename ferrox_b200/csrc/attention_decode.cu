@@ -271,9 +271,11 @@ __global__ void merge_kernel(const float* __restrict__ part_acc, const float* __
         mm = fmaxf(mm, x.sinks[h]);
         sunk = fx_exp<T>(x.sinks[h] - mm);
     }
-    for (int e = threadIdx.x; e < head_dim; e += blockDim.x) {
+    for (int e0 = 0; e0 < head_dim; e0 += blockDim.x) {      // (every lane takes every trip: partners of a pair meet)
+        const int e = e0 + threadIdx.x;
+        const bool in = e < head_dim;
         float ll = sunk, a = 0.f;
-        for (int s = 0; s < n_splits; ++s) {
+        for (int s = 0; s < n_splits && in; ++s) {
             if (!has_keys(s)) continue;
             const float ms = part_ml[(base + s) * 2];
             if (ms == -INFINITY) continue;
@@ -282,6 +284,11 @@ __global__ void merge_kernel(const float* __restrict__ part_acc, const float* __
             a += part_acc[(base + s) * head_dim + e] * w;
         }
         float v = ll > 0.f ? a / ll : 0.f;
+        if (x.turn) {
+            const float2 cs = in ? *reinterpret_cast<const float2*>(x.turn + (long)tkn * head_dim + (e & ~1)) : make_float2(1.f, 0.f);
+            v = fx_turn_back_lane(v, cs, e & 1);
+        }
+        if (!in) continue;
         if (x.gate) v *= fx_sigmoid_fast(to_f32(reinterpret_cast<const T*>(x.gate)[(long)tkn * x.ldg + (long)h * head_dim + e]));
         out[(long)tkn * ldo + (long)h * head_dim + e] = from_f32<T>(v);
     }
@@ -327,7 +334,7 @@ int run(const void* q, long ldq, const void* k_pages, const void* v_pages, int n
 {
     // (chunks, sinks and gates are options of the kernel that streams pages by TMA: the others refuse them)
     const DecodeExtras x = extras ? *extras : DecodeExtras{};
-    const bool plain = x.chunk == 0 && !x.sinks && !x.gate && !x.v_first && x.rot == 0;
+    const bool plain = x.chunk == 0 && !x.sinks && !x.gate && !x.turn && !x.v_first && x.rot == 0;
     if (!plain && (sizeof(T) != 2 || softcap > 0.f || n_pages <= 0)) return FX_ERR_SIZE;
     if (softcap > 0.f && store_new) return FX_ERR_SIZE;   // the kernel that stores the step's keys itself takes no cap
     constexpr int N = Vec<T>::N;

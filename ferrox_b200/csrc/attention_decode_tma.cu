@@ -80,6 +80,8 @@ __device__ __forceinline__ float finish(const DecArgs& a, float acc, float l, fl
             v = acc * f / (l * f + __expf(sk - mm));
         } else v = acc / l;
     }
+    if (a.x.turn)      // (whole warps come here together, neighbouring lanes with neighbouring elements)
+        v = fx_turn_back_lane(v, *reinterpret_cast<const float2*>(a.x.turn + (long)tkn * a.head_dim + (e & ~1)), e & 1);
     if (a.x.gate)
         v *= fx_sigmoid_fast(__bfloat162float(reinterpret_cast<const bf16*>(a.x.gate)[(long)tkn * a.x.ldg + (long)head * a.head_dim + e]));
     return v;

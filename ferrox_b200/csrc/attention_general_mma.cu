@@ -78,6 +78,7 @@ struct GArgs {
     int value_share;      // consecutive key heads that read one value head
     int chunk;            // > 0: a query sees the keys of its own chunk of that many positions only
     const bf16* gate; long ldg;   // (optional) token rows of n_heads * value_dim: the result times sigmoid(gate)
+    const float* turn;    // (optional) [tokens][value_dim / 2] (cos, sin): the result's pairs (2m, 2m + 1) turned back
 };
 
 // DVMAX: most value columns one warp accumulates.  NSPLIT: sets of 4 warps that share out the value columns.
@@ -318,6 +319,10 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
         const int col = i * 8 + 2 * t4;
         if (col < my_cols) {
             float x0 = o[i][0] * inv0, x1 = o[i][1] * inv0, x2 = o[i][2] * inv1, x3 = o[i][3] * inv1;
+            if (a.turn) {
+                fx_turn_back(x0, x1, *reinterpret_cast<const float2*>(a.turn + (long)(tok0 + min(r0, rows - 1) / n_h) * a.value_dim + col0 + col));
+                fx_turn_back(x2, x3, *reinterpret_cast<const float2*>(a.turn + (long)(tok0 + min(r1, rows - 1) / n_h) * a.value_dim + col0 + col));
+            }
             if (a.gate) {      // the output gate, on the 32-bit result
                 const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g0 + col));
                 const float2 gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g1 + col));
@@ -333,7 +338,8 @@ __global__ void __launch_bounds__(128 * NSPLIT) general_attention_kernel(GArgs a
 __global__ void general_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                      const int* __restrict__ positions, bf16* __restrict__ out, long ldo, long ldoh,
                                      int n_heads, int value_dim, int n_splits, int window, const float* __restrict__ sinks,
-                                     int chunk, const bf16* __restrict__ gate, long ldg)
+                                     int chunk, const bf16* __restrict__ gate, long ldg,
+                                     const float* __restrict__ turn)
 {
     fx_pdl_wait();
     const int tkn = blockIdx.x, h = blockIdx.y;
@@ -350,9 +356,11 @@ __global__ void general_merge_kernel(const float* __restrict__ part_o, const flo
         mm = fmaxf(mm, sk);
         sunk = exp2f(sk - mm);
     }
-    for (int e = threadIdx.x; e < value_dim; e += blockDim.x) {
+    for (int e0 = 0; e0 < value_dim; e0 += blockDim.x) {      // (every lane takes every trip: partners of a pair meet)
+        const int e = e0 + threadIdx.x;
+        const bool in = e < value_dim;
         float ll = sunk, acc = 0.f;
-        for (int s = 0; s < n_splits; ++s) {
+        for (int s = 0; s < n_splits && in; ++s) {
             if (!has_keys(s)) continue;
             const float ms = part_ml[(base + s) * 2];
             if (ms == -INFINITY) continue;
@@ -361,6 +369,11 @@ __global__ void general_merge_kernel(const float* __restrict__ part_o, const flo
             acc += part_o[(base + s) * value_dim + e] * w;
         }
         float x = ll > 0.f ? acc / ll : 0.f;
+        if (turn) {
+            const float2 cs = in ? *reinterpret_cast<const float2*>(turn + (long)tkn * value_dim + (e & ~1)) : make_float2(1.f, 0.f);
+            x = fx_turn_back_lane(x, cs, e & 1);
+        }
+        if (!in) continue;
         if (gate) x *= fx_sigmoid_fast(__bfloat162float(gate[(long)tkn * ldg + (long)h * value_dim + e]));
         out[(long)tkn * ldo + (long)h * ldoh + e] = __float2bfloat16_rn(x);
     }
@@ -378,7 +391,7 @@ int launch(dim3 grid, size_t smem, cudaStream_t s, const GArgs& a)
     if (a.n_splits > 1)
         fx_launch_pdl(general_merge_kernel, dim3(grid.x, a.n_heads), dim3(64), 0, s, (const float*)a.part_o,
                       (const float*)a.part_ml, a.positions, a.out, a.ldo, a.ldoh, a.n_heads, a.value_dim, a.n_splits,
-                      a.window, a.sinks, a.chunk, a.gate, a.ldg);
+                      a.window, a.sinks, a.chunk, a.gate, a.ldg, a.turn);
     return fx_launch_status();
 }
 
@@ -411,6 +424,8 @@ extern "C" int fx_general_attention_ok(int key_dim, int value_dim, int alias)
 // tokens x heads <= 64; or nullptr: one token a tile, n_items = tokens.  bfloat16 only.
 // chunk > 0: a query sees the keys of its own chunk of that many positions (counted from the request's start) only.
 // gate (optional): token rows of n_heads * value_dim, ldg elements apart; the result is multiplied by sigmoid(gate).
+// turn (optional): [tokens][value_dim / 2] (cos, sin); pair (2m, 2m + 1) of every head's result is turned by minus that
+// angle before the gate.
 // softcap c > 0: the scaled scores pass through c tanh(s / c) before bias and softmax.  sinks (optional, one per
 // head): exp(sinks[h]) joins the denominator once (with runs: in the merge).  value_share >= 1: that many consecutive
 // key heads read one value head (value head = key head / value_share).
@@ -423,7 +438,7 @@ extern "C" int fx_general_attention(const void* q, long ldq, long ldqh, const vo
                                     int key_dim, int value_dim, int window, float scale, const float* slopes,
                                     int n_splits, float* part_o, float* part_ml, int keep_first, float softcap,
                                     const float* sinks, int value_share, int chunk, const void* gate, long ldg,
-                                    void* stream)
+                                    const float* turn, void* stream)
 {
     if (n_items <= 0) return FX_OK;
     if (value_share < 1) value_share = 1;
@@ -452,6 +467,8 @@ extern "C" int fx_general_attention(const void* q, long ldq, long ldqh, const vo
     if (chunk < 0 || (chunk > 0 && a.keep_first > 0)) return FX_ERR_SIZE;
     if (gate && (ldg % 2 || (uintptr_t)gate % 4)) return FX_ERR_ALIGN;
     a.chunk = chunk; a.gate = (const bf16*)gate; a.ldg = ldg;
+    if ((uintptr_t)turn % 8) return FX_ERR_ALIGN;
+    a.turn = turn;
     a.n_splits = n_splits > 1 ? n_splits : 1; a.part_o = part_o; a.part_ml = part_ml;
     if (a.n_splits > 1 && (items || !part_o || !part_ml || a.n_splits > 65535)) return FX_ERR_SIZE;
     const int bkey = general_bkey(key_dim, value_dim, alias);

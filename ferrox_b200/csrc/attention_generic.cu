@@ -34,6 +34,8 @@
 // the value pages hold n_kv_heads / value_share heads), for attention maps of their own keys over shared values.
 // `chunk` (> 0): a query sees only the keys of its own chunk of that many positions, counted from the request's start.
 // `gate` (optional, token rows of n_heads * value_dim): the result is multiplied element by element by sigmoid(gate).
+// `turn` (optional, [tokens][value_dim / 2] (cos, sin); value_dim even): pair (2m, 2m + 1) of every head's result is
+// turned by minus that angle before the gate.
 #include "common.cuh"
 #include "api.h"
 
@@ -50,7 +52,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
     const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
     T* __restrict__ out, long ldo, long ldoh, int n_heads, int n_kv_heads, int key_dim, int value_dim, int window,
     float scale, float softcap, const float* __restrict__ slopes, int keep_first, const float* __restrict__ sinks,
-    int value_share, int chunk, const T* __restrict__ gate, long ldg)
+    int value_share, int chunk, const T* __restrict__ gate, long ldg, const float* __restrict__ turn)
 {
     __shared__ float q_s[WARPS][MAX_DK];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -129,8 +131,12 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int d = lane + 32 * i;
+        float v = acc[i] * inv;
+        if (turn) {      // (partners of a pair lie in neighbouring lanes: the whole warp takes part)
+            const float2 cs = d < value_dim ? *reinterpret_cast<const float2*>(turn + (long)t * value_dim + (d & ~1)) : make_float2(1.f, 0.f);
+            v = fx_turn_back_lane(v, cs, d & 1);
+        }
         if (d < value_dim) {
-            float v = acc[i] * inv;
             if (gate) v *= 1.0f / (1.0f + expf(-to_f32(gate[(long)t * ldg + (long)h * value_dim + d])));
             o[d] = from_f32<T>(v);
         }
@@ -142,14 +148,15 @@ int launch_paged(const void* q, long ldq, long ldqh, const void* k_pages, const 
                  const int* block_table, int table_width, int page_size, const int* positions, const int* token_seq,
                  const int* seq_slot, void* out, long ldo, long ldoh, int n_tokens, int n_heads, int n_kv_heads,
                  int key_dim, int value_dim, int window, float scale, float softcap, const float* slopes, int keep_first,
-                 const float* sinks, int value_share, int chunk, const void* gate, long ldg, cudaStream_t s)
+                 const float* sinks, int value_share, int chunk, const void* gate, long ldg,
+                 const float* turn, cudaStream_t s)
 {
     dim3 grid(n_tokens, (unsigned)fx_cdiv(n_heads, WARPS));
 #define FX_GO(NV)                                                                                                     \
     paged_attention_kernel<T, NV><<<grid, WARPS * 32, 0, s>>>((const T*)q, ldq, ldqh, (const T*)k_pages,              \
         (const T*)v_pages, ldk, ldv, block_table, table_width, page_size, positions, token_seq, seq_slot, (T*)out,    \
         ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks,        \
-        value_share, chunk, (const T*)gate, ldg)
+        value_share, chunk, (const T*)gate, ldg, turn)
     if (value_dim <= 64) FX_GO(2);
     else if (value_dim <= 128) FX_GO(4);
     else if (value_dim <= 256) FX_GO(8);
@@ -168,13 +175,14 @@ extern "C" int fx_paged_attention_ex(const void* q, long ldq, long ldqh, const v
                                      void* out, long ldo, long ldoh, int n_tokens, int n_heads, int n_kv_heads,
                                      int key_dim, int value_dim, int window, float scale, float softcap,
                                      const float* slopes, int keep_first, const float* sinks, int value_share,
-                                     int chunk, const void* gate, long ldg, void* stream)
+                                     int chunk, const void* gate, long ldg, const float* turn, void* stream)
 {
     if (n_tokens <= 0) return FX_OK;
     if (value_share < 1) value_share = 1;
     if (n_kv_heads % value_share) return FX_ERR_SIZE;
     if (keep_first < 0 || window <= 0) keep_first = 0;
     if (chunk < 0 || (chunk > 0 && keep_first > 0)) return FX_ERR_SIZE;
+    if (turn && (value_dim % 2 || (uintptr_t)turn % 8)) return FX_ERR_ALIGN;
     if (key_dim > MAX_DK || value_dim > MAX_DV || key_dim <= 0 || value_dim <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || ldk < key_dim || ldv < value_dim)
         return FX_ERR_SIZE;
@@ -182,11 +190,11 @@ extern "C" int fx_paged_attention_ex(const void* q, long ldq, long ldqh, const v
     if (dtype == FX_F32)
         return launch_paged<float>(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, table_width, page_size,
                                    positions, token_seq, seq_slot, out, ldo, ldoh, n_tokens, n_heads, n_kv_heads,
-                                   key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, chunk, gate, ldg, s);
+                                   key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, chunk, gate, ldg, turn, s);
     if (dtype == FX_BF16)
         return launch_paged<bf16>(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, table_width, page_size,
                                   positions, token_seq, seq_slot, out, ldo, ldoh, n_tokens, n_heads, n_kv_heads,
-                                  key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, chunk, gate, ldg, s);
+                                  key_dim, value_dim, window, scale, softcap, slopes, keep_first, sinks, value_share, chunk, gate, ldg, turn, s);
     return FX_ERR_DTYPE;
 }
 
@@ -199,5 +207,5 @@ extern "C" int fx_paged_attention(const void* q, long ldq, const void* k_pages, 
 {
     return fx_paged_attention_ex(q, ldq, head_dim, k_pages, v_pages, head_dim, head_dim, dtype, block_table, table_width,
                                  page_size, positions, token_seq, seq_slot, out, ldo, head_dim, n_tokens, n_heads,
-                                 n_kv_heads, head_dim, head_dim, window, scale, softcap, nullptr, 0, nullptr, 1, 0, nullptr, 0, stream);
+                                 n_kv_heads, head_dim, head_dim, window, scale, softcap, nullptr, 0, nullptr, 1, 0, nullptr, 0, nullptr, stream);
 }

@@ -39,7 +39,8 @@
 //
 // Options: `chunk` (a query sees the keys of its own chunk of that many positions only, counted from the request's
 // start), `sinks` (one number per head: exp(sink_h) joins the softmax's denominator once, at the end or in the merge),
-// `gate` (token rows of n_heads * value_dim: the result is multiplied by sigmoid(gate) before it is rounded).
+// `gate` (token rows of n_heads * value_dim: the result is multiplied by sigmoid(gate) before it is rounded), `turn`
+// ([tokens][value_dim / 2] (cos, sin): pair (2m, 2m + 1) of the result is turned by minus that angle before the gate).
 //
 // Reference: crates/ferrox-core/src/attention.rs:531-563 (query t over keys 0..=t), :146-175 (online
 // softmax), :484-524 (window), :572-610 (pages), :432-449 (grouped heads).  The mma.sync kernel of
@@ -71,6 +72,7 @@ struct AttnArgs {
     int value_dim;                   // elements of a value head (V: rounded up)
     const float* sinks;              // (optional) one per head
     const bf16* gate; long ldg;      // (optional) token rows of n_heads * value_dim
+    const float* turn;               // (optional) [tokens][value_dim / 2] (cos, sin)
     float scale_log2e;
     int* status;
 };
@@ -378,6 +380,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                 const float inv = inverse_sum(l, m * sl2, a.sinks, head);
                 bf16* dst = a.out + (long)(tok0 + t * BQ + r) * a.ldo + (long)head * a.value_dim;
                 const bf16* gate = a.gate ? a.gate + (long)(tok0 + t * BQ + r) * a.ldg + (long)head * a.value_dim : nullptr;
+                const float* turn = a.turn ? a.turn + (long)(tok0 + t * BQ + r) * a.value_dim : nullptr;
 #pragma unroll
                 for (int c = 0; c < V / 32; ++c) {
                     uint32_t ob[32];
@@ -390,6 +393,12 @@ __global__ void __launch_bounds__(NTHREADS, 1) prefill_attention_tc_kernel(const
                             float x[8];
 #pragma unroll
                             for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(ob[k + e]) * inv;
+                            if (turn) {
+                                const float4 c0 = *reinterpret_cast<const float4*>(turn + c * 32 + k);
+                                const float4 c1 = *reinterpret_cast<const float4*>(turn + c * 32 + k + 4);
+                                fx_turn_back(x[0], x[1], make_float2(c0.x, c0.y)); fx_turn_back(x[2], x[3], make_float2(c0.z, c0.w));
+                                fx_turn_back(x[4], x[5], make_float2(c1.x, c1.y)); fx_turn_back(x[6], x[7], make_float2(c1.z, c1.w));
+                            }
                             if (gate) {
                                 float g[8];
                                 Pack<bf16>::load(gate + c * 32 + k, g);
@@ -423,7 +432,8 @@ __global__ void __launch_bounds__(128) prefill_merge_kernel(const int* __restric
                                                             const float* __restrict__ part_ml, bf16* __restrict__ out, long ldo,
                                                             int n_heads, float scale_log2e, int value_dim,
                                                             const float* __restrict__ sinks,
-                                                            const bf16* __restrict__ gate, long ldg)
+                                                            const bf16* __restrict__ gate, long ldg,
+                                                            const float* __restrict__ turn)
 {
     fx_pdl_wait();
     const int* mg = merges + (long)blockIdx.x * 4;
@@ -460,6 +470,12 @@ __global__ void __launch_bounds__(128) prefill_merge_kernel(const int* __restric
     const float inv = inverse_sum(l, mx * scale_log2e, sinks, head);
     bf16* dst = out + (long)(tok0 + r) * ldo + (long)head * value_dim + lane * PER;
     const bf16* g = gate ? gate + (long)(tok0 + r) * ldg + (long)head * value_dim + lane * PER : nullptr;
+    static_assert(PER % 2 == 0, "a lane holds whole pairs");
+    if (turn) {
+#pragma unroll
+        for (int i = 0; i < PER; i += 2)
+            fx_turn_back(acc[i], acc[i + 1], *reinterpret_cast<const float2*>(turn + (long)(tok0 + r) * value_dim + lane * PER + i));
+    }
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         float x = acc[i] * inv;
@@ -492,7 +508,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     fx_launch_pdl(kern, grid, NTHREADS, Smem<D, V>::TOTAL, s, mq, mk, mv, a);
     if (n_merges > 0)
         fx_launch_pdl(prefill_merge_kernel<V>, dim3(n_merges, a.n_heads, 2 * BQ / 4), 128, 0, s, merges, (const float*)a.part_o,
-                      (const float*)a.part_ml, a.out, a.ldo, a.n_heads, a.scale_log2e, a.value_dim, a.sinks, a.gate, a.ldg);
+                      (const float*)a.part_ml, a.out, a.ldo, a.n_heads, a.scale_log2e, a.value_dim, a.sinks, a.gate, a.ldg, a.turn);
     return fx_launch_status();
 }
 
@@ -510,7 +526,8 @@ extern "C" int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, co
                                        int n_pages, const int* block_table, int table_width, int page_size,
                                        const int* tiles, int n_tiles, const int* seq_slot, void* out, long ldo,
                                        int n_heads, int n_kv_heads, int head_dim, int value_dim, int window, int chunk,
-                                       float scale, const float* sinks, const void* gate, long ldg, int* status,
+                                       float scale, const float* sinks, const void* gate, long ldg, const float* turn,
+                                       int* status,
                                        float* part_o, float* part_ml, const int* merges, int n_merges, void* stream)
 {
     if (n_tiles <= 0) return FX_OK;
@@ -520,7 +537,7 @@ extern "C" int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, co
         return FX_ERR_SIZE;
     if (ldq % 8 || ldo % 8 || (uintptr_t)q % 16 || (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16 || (uintptr_t)out % 16)
         return FX_ERR_ALIGN;
-    if (gate && (ldg % 8 || (uintptr_t)gate % 16)) return FX_ERR_ALIGN;
+    if ((gate && (ldg % 8 || (uintptr_t)gate % 16)) || (uintptr_t)turn % 16) return FX_ERR_ALIGN;
     if (n_tiles > 65535) return FX_ERR_SIZE;
     CUtensorMap mq, mk, mv;
     {
@@ -541,7 +558,7 @@ extern "C" int fx_prefill_attention_tc(const void* q, long ldq, int n_tokens, co
     a.block_table = block_table; a.table_width = table_width; a.page_size = page_size;
     a.tiles = tiles; a.seq_slot = seq_slot; a.out = (bf16*)out; a.ldo = ldo;
     a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.window = window; a.chunk = chunk; a.value_dim = value_dim;
-    a.sinks = sinks; a.gate = (const bf16*)gate; a.ldg = ldg;
+    a.sinks = sinks; a.gate = (const bf16*)gate; a.ldg = ldg; a.turn = turn;
     a.scale_log2e = scale * 1.4426950408889634f; a.status = status;
     a.part_o = part_o; a.part_ml = part_ml;
     dim3 grid(n_heads, n_tiles);

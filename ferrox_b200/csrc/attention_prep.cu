@@ -165,6 +165,97 @@ __global__ void rotary_mix_store_kernel(T* __restrict__ qkv, long ld, const int*
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Rows of [q heads | k heads | v heads] (head widths D, D, V) of an attention that norms its queries and keys behind the
+// rotation and caches its values turned by their position:
+//   q, k: the first rot elements of a head turned by the token's angles (cos_sin [tokens][rot / 2][2]; pairing as above;
+//   nullptr: none), then, eps >= 0, x / sqrt(mean(x^2) + eps) over the head; q in place, k into its page;
+//   v: pairs (2m, 2m + 1) of the whole head turned by v_cos_sin [tokens][V / 2][2] (nullptr: as it is), into its page.
+// The rows' own k and v stay as projected.  A warp a head (the head's row as 32-bit values in shared memory), gridDim.y
+// blocks a token; items of N elements.
+template <> struct Items<bf16, 4> {
+    static __device__ __forceinline__ void load(const bf16* p, float* o) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        o[0] = __uint_as_float(v.x << 16); o[1] = __uint_as_float(v.x & 0xffff0000u);
+        o[2] = __uint_as_float(v.y << 16); o[3] = __uint_as_float(v.y & 0xffff0000u);
+    }
+    static __device__ __forceinline__ void store(bf16* p, const float* o) {
+        __nv_bfloat162 a = __floats2bfloat162_rn(o[0], o[1]), b = __floats2bfloat162_rn(o[2], o[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+    }
+};
+
+constexpr int RN_WARPS = 8;
+
+template <typename T, int N>
+__global__ void __launch_bounds__(RN_WARPS * 32) rotary_norm_store_kernel(
+    T* __restrict__ qkv, long ld, const int* __restrict__ positions, const int* __restrict__ token_seq,
+    const int* __restrict__ seq_slot, const float* __restrict__ cos_sin, int rot, int pairing, float eps,
+    const float* __restrict__ v_cos_sin, T* __restrict__ k_pages, T* __restrict__ v_pages,
+    const int* __restrict__ block_table, int table_width, int page_size, int H, int G, int D, int V, int write_cache,
+    int* __restrict__ status)
+{
+    extern __shared__ __align__(16) float rn_s[];
+    fx_pdl_wait();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int pos = positions[t];
+    T* row = qkv + (long)t * ld;
+    long place = -1;      // (page, kv head 0, position in the page) as one index
+    if (write_cache) {
+        const int page = block_table[(long)seq_slot[token_seq[t]] * table_width + pos / page_size];
+        if (page < 0) { if (threadIdx.x == 0 && status) atomicExch(status, 2); }
+        else place = (long)page * G * page_size + (pos % page_size);
+    }
+    float* x_s = rn_s + warp * (((D > V ? D : V) + 3) & ~3);
+    const int half = rot >> 1;
+    const float* cs = cos_sin ? cos_sin + (long)t * half * 2 : nullptr;
+    const float* vcs = v_cos_sin ? v_cos_sin + (long)t * V : nullptr;
+    const int units = H + 2 * G;
+    for (int u = blockIdx.y * RN_WARPS + warp; u < units; u += gridDim.y * RN_WARPS) {
+        const bool is_q = u < H, is_v = u >= H + G;
+        if (!is_q && place < 0) continue;
+        const int width = is_v ? V : D;
+        T* x = row + (is_v ? (long)(H + G) * D + (long)(u - H - G) * V : (long)u * D);
+        T* dst = is_q ? x : is_v ? v_pages + (place + (long)(u - H - G) * page_size) * V
+                                 : k_pages + (place + (long)(u - H) * page_size) * D;
+        float ss = 0.f;
+        for (int i = lane * N; i < width; i += 32 * N) {
+            float a[N];
+            Items<T, N>::load(x + i, a);
+#pragma unroll
+            for (int e = 0; e < N; ++e) { x_s[i + e] = a[e]; ss = fmaf(a[e], a[e], ss); }
+        }
+        __syncwarp();
+        // (a rotation leaves the sum of squares as it is)
+        const float r = is_v || eps < 0.f ? 1.f : 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
+        for (int i = lane * N; i < width; i += 32 * N) {
+            float a[N];
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                const int j = i + e;
+                const float own = x_s[j];
+                float y = own;
+                if (is_v) {
+                    if (vcs) {
+                        const float2 f = *reinterpret_cast<const float2*>(vcs + (j & ~1));
+                        const float other = x_s[j ^ 1];
+                        y = j & 1 ? own * f.x + other * f.y : own * f.x - other * f.y;
+                    }
+                } else if (cs && j < rot) {
+                    const bool second = pairing ? j & 1 : j >= half;
+                    const int p = pairing ? j >> 1 : (second ? j - half : j);
+                    const float2 f = *reinterpret_cast<const float2*>(cs + p * 2);
+                    const float other = x_s[pairing ? j ^ 1 : (second ? j - half : j + half)];
+                    y = second ? own * f.x + other * f.y : own * f.x - other * f.y;
+                }
+                a[e] = y * r;
+            }
+            Items<T, N>::store(dst + i, a);
+        }
+        __syncwarp();
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // The latent form.  Per token: `dkv` = [C latent | R rotated key part] as projected, `q` = H heads of [D | R].
 //   c <- dkv[:C] / sqrt(mean(dkv[:C]^2) + eps) * wc            -> pages[position][0:C]
 //   k_rot <- pairs (2i, 2i+1) of the first rot_dims of dkv[C:] turned by the position's angles, the rest as it is
@@ -332,6 +423,40 @@ extern "C" int fx_rotary_mix_store(void* qkv, int dtype, long ld, const int* pos
                   table_width, page_size, n_heads, n_kv_heads, key_dim, value_dim, write_cache, status)
     if (dtype == FX_F32) { if (vec) FX_GO(float, 4); else FX_GO(float, 1); }
     else if (dtype == FX_BF16) { if (vec) FX_GO(bf16, 8); else FX_GO(bf16, 1); }
+    else return FX_ERR_DTYPE;
+#undef FX_GO
+    return fx_launch_status();
+}
+
+// eps < 0: queries and keys are not normed.  Refuses (FX_ERR_SIZE) heads wider than the shared memory holds.
+extern "C" int fx_rotary_norm_store(void* qkv, int dtype, long ld, const int* positions, const int* token_seq,
+                                    const int* seq_slot, const float* cos_sin, int rot, int pairing, float eps,
+                                    const float* v_cos_sin, void* k_pages, void* v_pages, const int* block_table,
+                                    int table_width, int page_size, int n_tokens, int n_heads, int n_kv_heads,
+                                    int key_dim, int value_dim, int write_cache, int* status, void* stream)
+{
+    if (n_tokens <= 0) return FX_OK;
+    if (key_dim <= 0 || value_dim <= 0 || page_size <= 0 || n_heads <= 0 || n_kv_heads <= 0 || pairing < 0 || pairing > 1)
+        return FX_ERR_SIZE;
+    if (!cos_sin) rot = 0;
+    if (rot < 0 || rot % 2 || rot > key_dim || (v_cos_sin && value_dim % 2)) return FX_ERR_SIZE;
+    if ((uintptr_t)cos_sin % 8 || (uintptr_t)v_cos_sin % 8) return FX_ERR_ALIGN;
+    const int widest = ((key_dim > value_dim ? key_dim : value_dim) + 3) & ~3;
+    const size_t smem = (size_t)RN_WARPS * widest * 4;
+    if (smem > 48 * 1024) return FX_ERR_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int item = dtype == FX_F32 ? 16 : 8;     // bytes of four elements
+    const bool vec = key_dim % 4 == 0 && value_dim % 4 == 0 && ld % 4 == 0 && (uintptr_t)qkv % item == 0 &&
+                     (uintptr_t)k_pages % item == 0 && (uintptr_t)v_pages % item == 0;
+    // few tokens (a decode step): a token's heads are shared out over blocks
+    const int units = n_heads + 2 * n_kv_heads;
+    dim3 grid(n_tokens, n_tokens < 256 ? (unsigned)fx_cdiv(units, RN_WARPS) : 1u);
+#define FX_GO(T, N)                                                                                                   \
+    fx_launch_pdl(rotary_norm_store_kernel<T, N>, grid, RN_WARPS * 32, smem, s, (T*)qkv, ld, positions, token_seq,   \
+                  seq_slot, cos_sin, rot, pairing, eps, v_cos_sin, (T*)k_pages, (T*)v_pages, block_table, table_width, \
+                  page_size, n_heads, n_kv_heads, key_dim, value_dim, write_cache, status)
+    if (dtype == FX_F32) { if (vec) FX_GO(float, 4); else FX_GO(float, 1); }
+    else if (dtype == FX_BF16) { if (vec) FX_GO(bf16, 4); else FX_GO(bf16, 1); }
     else return FX_ERR_DTYPE;
 #undef FX_GO
     return fx_launch_status();

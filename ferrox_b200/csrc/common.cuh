@@ -151,6 +151,20 @@ __device__ __forceinline__ void fx_gate_32(float* x, const uint32_t* u, int act,
 // sigmoid(g) with the hardware's exponential and quotient, for the attention kernels' output gates.
 __device__ __forceinline__ float fx_sigmoid_fast(float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); }
 
+// A head's result turned back: pair (x0, x1) of neighbours 2m, 2m + 1 by minus the angle whose cos and sin are cs, for
+// attention whose values were turned by their own positions before they were cached.
+__device__ __forceinline__ void fx_turn_back(float& x0, float& x1, float2 cs) {
+    const float a = x0;
+    x0 = a * cs.x + x1 * cs.y;
+    x1 = x1 * cs.x - a * cs.y;
+}
+
+// The same where the two elements of a pair lie in neighbouring lanes (even lane: x0): called by whole warps.
+__device__ __forceinline__ float fx_turn_back_lane(float x, float2 cs, bool odd) {
+    const float other = __shfl_xor_sync(0xffffffffu, x, 1);
+    return odd ? x * cs.x - other * cs.y : x * cs.x + other * cs.y;
+}
+
 // The first key the query at position pos may see: of a window of the last `window` positions (0: no window) and of
 // chunks of `chunk` positions counted from the request's start (0: no chunks), in which a query sees its own chunk only.
 __host__ __device__ __forceinline__ int fx_first_key(int pos, int window, int chunk) {

@@ -3,7 +3,7 @@
 //   out[t, c] = x[t, c] + sum_j w[c, j] * x[t - (taps - 1) + j, c]        (zeros before the request's start)
 //
 // (add_input = 0: the sum alone, for a convolution that stands in its input's place, as the one behind the
-// projections of an attention mixer)
+// projections of an attention mixer; a bias per channel and SiLU of the result are options)
 //
 // over the tokens of one request.  The taps - 1 inputs before a step's first token come from the request's state
 // slot (`tail` [slots, taps - 1, channels], 32-bit, oldest first), so a request may be cut into steps anywhere;
@@ -24,7 +24,7 @@ template <typename T>
 __global__ void __launch_bounds__(CONV_THREADS) input_conv_kernel(
     const T* __restrict__ x, long ldx, const void* __restrict__ w, int w_dtype, int taps, float* tail,
     const int* __restrict__ token_seq, const int* __restrict__ seq_slot, T* __restrict__ out, long ldo, int C,
-    int update_tail, int add_input)
+    int update_tail, int add_input, const void* __restrict__ bias, int b_dtype, int act)
 {
     fx_pdl_wait();
     const int t = blockIdx.x;
@@ -37,6 +37,7 @@ __global__ void __launch_bounds__(CONV_THREADS) input_conv_kernel(
     float* tl = tail + (long)seq_slot[b] * (taps - 1) * C;
     const float xt = to_f32(x[(long)t * ldx + c]);
     float acc = add_input ? xt : 0.f;     // (a convolution that replaces its input: the sum alone)
+    if (bias) acc += load_any(bias, b_dtype, c);
     for (int j = 0; j < taps; ++j) {
         const int back = taps - 1 - j;          // this tap's input lies `back` tokens before t
         float v;
@@ -45,12 +46,71 @@ __global__ void __launch_bounds__(CONV_THREADS) input_conv_kernel(
         else v = tl[(long)(taps - 1 - (back - own)) * C + c];
         acc = fmaf(load_any(w, w_dtype, (long)c * taps + j), v, acc);
     }
+    if (act) acc = acc / (1.0f + expf(-acc));
     out[(long)t * ldo + c] = from_f32<T>(acc);
     // (the caller's promise that every entry brings exactly one token: this thread is then the only reader of the
     // channel's tail in the whole step, and moves it on by the token's input itself)
     if (update_tail && taps > 1) {
         for (int j = 0; j + 1 < taps - 1; ++j) tl[(long)j * C + c] = tl[(long)(j + 1) * C + c];
         tl[(long)(taps - 2) * C + c] = xt;
+    }
+}
+
+// The same for a prompt: a thread takes RUN tokens of two neighbouring channels one after the other and keeps the last
+// TAPS - 1 inputs in registers, so that every input is read once (and TAPS - 1 more at the start of a run).
+constexpr int CONV_RUN = 16;
+
+template <typename T> __device__ __forceinline__ float2 load2(const T* p);
+template <> __device__ __forceinline__ float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> __device__ __forceinline__ float2 load2<bf16>(const bf16* p) {
+    return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+__device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void store2(bf16* p, float2 v) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y);
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CONV_THREADS) input_conv_run_kernel(
+    const T* __restrict__ x, long ldx, const void* __restrict__ w, int w_dtype, const float* __restrict__ tail,
+    const int* __restrict__ token_seq, const int* __restrict__ seq_slot, T* __restrict__ out, long ldo, int n_tokens, int C,
+    int add_input, const void* __restrict__ bias, int b_dtype, int act)
+{
+    fx_pdl_wait();
+    const int t0 = blockIdx.x * CONV_RUN, t1 = min(n_tokens, t0 + CONV_RUN);
+    const int c = (blockIdx.y * CONV_THREADS + threadIdx.x) * 2;
+    if (c >= C) return;
+    float2 wt[TAPS], hist[TAPS];      // hist[j]: the input TAPS - 1 - j tokens before the current one
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+        wt[j] = make_float2(load_any(w, w_dtype, (long)c * TAPS + j), load_any(w, w_dtype, (long)(c + 1) * TAPS + j));
+    float2 b0 = make_float2(0.f, 0.f);
+    if (bias) b0 = make_float2(load_any(bias, b_dtype, c), load_any(bias, b_dtype, c + 1));
+    int seq = -1;
+    for (int t = t0; t < t1; ++t) {
+        const int s = token_seq[t];
+        if (s != seq) {       // the run's first token, or another entry's: its earlier inputs, from rows and tail
+            seq = s;
+            int own = 0;
+            while (own < TAPS - 1 && t - own - 1 >= 0 && token_seq[t - own - 1] == s) ++own;
+            const float* tl = tail + (long)seq_slot[s] * (TAPS - 1) * C + c;
+#pragma unroll
+            for (int j = 1; j < TAPS; ++j) {            // (moved down by one below)
+                const int back = TAPS - j;
+                hist[j] = back <= own ? load2(x + (long)(t - back) * ldx + c)
+                                      : *reinterpret_cast<const float2*>(tl + (long)(TAPS - 1 - (back - own)) * C);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j) hist[j] = hist[j + 1];
+        const float2 xt = load2(x + (long)t * ldx + c);
+        hist[TAPS - 1] = xt;
+        float2 acc = add_input ? xt : make_float2(0.f, 0.f);
+        acc.x += b0.x; acc.y += b0.y;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) { acc.x = fmaf(wt[j].x, hist[j].x, acc.x); acc.y = fmaf(wt[j].y, hist[j].y, acc.y); }
+        if (act) { acc.x = acc.x / (1.0f + expf(-acc.x)); acc.y = acc.y / (1.0f + expf(-acc.y)); }
+        store2(out + (long)t * ldo + c, acc);
     }
 }
 
@@ -97,18 +157,31 @@ __global__ void relu_square_kernel(T* __restrict__ x, long ld, int n)
 
 extern "C" int fx_input_conv(const void* x, int dtype, long ldx, const void* w, int w_dtype, int taps, float* tail,
                              const int* token_seq, const int* seq_slot, void* out, long ldo, int n_tokens, int channels,
-                             int update_tail, int add_input, void* stream)
+                             int update_tail, int add_input, const void* bias, int b_dtype, int act, void* stream)
 {
     if (n_tokens <= 0 || channels <= 0) return FX_OK;
     if (taps < 1 || taps > CONV_MAX_TAPS || x == out) return FX_ERR_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(n_tokens, (unsigned)fx_cdiv(channels, CONV_THREADS));
+    const int es = dtype == FX_F32 ? 8 : 4;      // bytes of two elements
+    if (!update_tail && n_tokens >= 128 && (taps == 3 || taps == 4) && channels % 2 == 0 && ldx % 2 == 0 && ldo % 2 == 0 &&
+        (uintptr_t)x % es == 0 && (uintptr_t)out % es == 0 && (uintptr_t)tail % 8 == 0) {
+        dim3 g((unsigned)fx_cdiv(n_tokens, CONV_RUN), (unsigned)fx_cdiv(channels, 2 * CONV_THREADS));
+#define FX_RUN(T, TAPS)                                                                                              \
+    fx_launch_pdl(input_conv_run_kernel<T, TAPS>, g, CONV_THREADS, 0, s, (const T*)x, ldx, w, w_dtype,               \
+                  (const float*)tail, token_seq, seq_slot, (T*)out, ldo, n_tokens, channels, add_input, bias, b_dtype, act)
+        if (dtype == FX_F32) { if (taps == 4) FX_RUN(float, 4); else FX_RUN(float, 3); }
+        else if (dtype == FX_BF16) { if (taps == 4) FX_RUN(bf16, 4); else FX_RUN(bf16, 3); }
+        else return FX_ERR_DTYPE;
+#undef FX_RUN
+        return fx_launch_status();
+    }
     if (dtype == FX_F32)
         fx_launch_pdl(input_conv_kernel<float>, grid, CONV_THREADS, 0, s, (const float*)x, ldx, w, w_dtype, taps, tail,
-                      token_seq, seq_slot, (float*)out, ldo, channels, update_tail, add_input);
+                      token_seq, seq_slot, (float*)out, ldo, channels, update_tail, add_input, bias, b_dtype, act);
     else if (dtype == FX_BF16)
         fx_launch_pdl(input_conv_kernel<bf16>, grid, CONV_THREADS, 0, s, (const bf16*)x, ldx, w, w_dtype, taps, tail,
-                      token_seq, seq_slot, (bf16*)out, ldo, channels, update_tail, add_input);
+                      token_seq, seq_slot, (bf16*)out, ldo, channels, update_tail, add_input, bias, b_dtype, act);
     else return FX_ERR_DTYPE;
     return fx_launch_status();
 }

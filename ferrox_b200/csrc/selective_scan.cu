@@ -1,0 +1,245 @@
+// The selective state space of a Mamba mixer: per request a state S [inner, n_state], 32-bit, and for every token
+//
+//   dt_c = softplus(dt_c + bias_c),    S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,    A = -exp(A_log)
+//   y_c  = sum_n S[c, n] C_n + D_c x_c,    out_c = y_c silu(z_c)
+//
+// Channels never meet: L lanes share a channel's states (NPL of them each, in runs of four, so that B and C are read
+// from shared memory sixteen bytes at a time) and keep them in registers for the whole step; the tokens of a request are
+// taken in order, in the same order of operations however the request was cut into steps.  A block of 128 threads takes
+// 128 / L channels of one request; the tokens' rows come SC_CH tokens at a time, the next chunk's into registers while
+// this one is worked on.  The step size, the products dt x and the skip and gate are worked out once a (token, channel),
+// not by every lane; the lanes' shares of the read-out meet once a chunk, through shared memory.
+//
+// Everything is 32-bit arithmetic; x and z come in the engine's element type.  A state that decays slowly is multiplied a
+// thousand times by numbers just below 1, so that a bias of half a unit in their last place would show: where the
+// exponent is small the state moves by S (e^a - 1) with e^a - 1 from its Taylor series, whose error is relative to a.
+#include "common.cuh"
+#include "api.h"
+
+namespace {
+
+__device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+
+// e^a S + u for a <= 0.
+__device__ __forceinline__ float decay_add(float S, float a, float u)
+{
+    // a > -1/4: e^a - 1 = a (1 + a/2 (1 + a/3 (1 + a/4 (1 + a/5 (1 + a/6))))), the next term below 5e-8 of the sum
+    float p = fmaf(a, 1.0f / 720.0f, 1.0f / 120.0f);
+    p = fmaf(p, a, 1.0f / 24.0f);
+    p = fmaf(p, a, 1.0f / 6.0f);
+    p = fmaf(p, a, 0.5f);
+    p = fmaf(p, a, 1.0f) * a;
+    const float slow = fmaf(S, p, u) + S;
+    const float fast = fmaf(S, __expf(a), u);
+    return a > -0.25f ? slow : fast;
+}
+
+// first row r with token_seq[r] >= b
+__device__ __forceinline__ int first_row_of(const int* __restrict__ token_seq, int n_tokens, int b)
+{
+    int lo = 0, hi = n_tokens;
+    while (lo < hi) {
+        const int mid = (lo + hi) >> 1;
+        if (token_seq[mid] < b) lo = mid + 1; else hi = mid;
+    }
+    return lo;
+}
+
+constexpr int SC_THREADS = 128;
+constexpr int SC_CH = 16;        // tokens a chunk
+
+struct ScArgs {
+    const float* dt; long ldt; const void* dt_bias; int db_dtype;
+    const void* x; long ldx; const void* z; long ldz;
+    const float* bc; long ldbc;              // [tokens][B (n_state) | C (n_state)]
+    const float* a_log; const float* d_skip; // [inner][n_state], [inner]
+    float* state;                            // [slots, inner, n_state]
+    void* out; long ldo;
+    const int *token_seq, *seq_slot;
+    int n_tokens, inner, n_state;
+};
+
+template <typename T, int L, int NPL>
+__global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs a)
+{
+    constexpr int CB = SC_THREADS / L;                       // channels a block
+    constexpr int NP = L * NPL;                              // states a channel, padded
+    constexpr int EPT = (SC_CH * CB + SC_THREADS - 1) / SC_THREADS;     // (token, channel) pairs a thread
+    constexpr int BPT = (SC_CH * NP + SC_THREADS - 1) / SC_THREADS;     // (token, state) pairs a thread
+    __shared__ float dt_s[SC_CH][CB], dx_s[SC_CH][CB];
+    __shared__ float x_s[SC_CH][CB], z_s[SC_CH][CB];
+    __shared__ __align__(16) float b_s[SC_CH][NP], c_s[SC_CH][NP];
+    __shared__ float rd_s[SC_CH][SC_THREADS];
+    fx_pdl_wait_only();
+    const int b = blockIdx.x;
+    const int r0 = first_row_of(a.token_seq, a.n_tokens, b), r1 = first_row_of(a.token_seq, a.n_tokens, b + 1);
+    if (r1 <= r0) return;
+    const int ch0 = blockIdx.y * CB, I = a.inner, N = a.n_state;
+    const int cl = threadIdx.x / L, part = threadIdx.x % L, ch = ch0 + cl;
+    const bool live = ch < I;
+    float* sp = a.state + ((long)a.seq_slot[b] * I + (live ? ch : 0)) * N;
+    const T* xp = reinterpret_cast<const T*>(a.x);
+    const T* zp = reinterpret_cast<const T*>(a.z);
+
+    float S[NPL], A[NPL];        // the states and their rates
+#pragma unroll
+    for (int i = 0; i < NPL; ++i) {
+        const int n = (i >> 2) * 4 * L + part * 4 + (i & 3);
+        const bool in = live && n < N;
+        S[i] = in ? sp[n] : 0.f;
+        A[i] = in ? -expf(a.a_log[(long)ch * N + n]) : 0.f;
+    }
+    // the channel of this thread's (token, channel) pairs is the same in every chunk: CB divides the block
+    const int pc = threadIdx.x % CB, ptt = threadIdx.x / CB, pch = ch0 + pc;
+    const bool plive = pch < I;
+    const int gch = plive ? pch : I - 1;
+    const float bias = load_any(a.dt_bias, a.db_dtype, gch), skip = a.d_skip[gch];
+
+    float fdt[EPT], fx[EPT], fz[EPT], fb[BPT], fc[BPT];
+    auto fetch = [&](int c0, int nt) {       // every load unconditional, from places clamped into the chunk
+#pragma unroll
+        for (int e = 0; e < EPT; ++e) {
+            const long t = c0 + min(ptt + e * L, nt - 1);
+            fdt[e] = a.dt[t * a.ldt + gch];
+            fx[e] = to_f32(xp[t * a.ldx + gch]);
+            fz[e] = to_f32(zp[t * a.ldz + gch]);
+        }
+#pragma unroll
+        for (int e = 0; e < BPT; ++e) {
+            const int idx = threadIdx.x + e * SC_THREADS;
+            const long t = c0 + min(idx / NP, nt - 1);
+            const int n = min(idx % NP, N - 1);
+            fb[e] = a.bc[t * a.ldbc + n];
+            fc[e] = a.bc[t * a.ldbc + N + n];
+        }
+    };
+    fetch(r0, min(SC_CH, r1 - r0));
+    for (int c0 = r0; c0 < r1; c0 += SC_CH) {
+        const int nt = min(SC_CH, r1 - c0);
+        __syncthreads();             // the chunk before is done with the staged rows
+#pragma unroll
+        for (int e = 0; e < EPT; ++e) {
+            const int tt = ptt + e * L;
+            if (tt < SC_CH) {
+                const float d = softplus_f(fdt[e] + bias);
+                dt_s[tt][pc] = d; dx_s[tt][pc] = d * fx[e];
+                x_s[tt][pc] = fx[e]; z_s[tt][pc] = fz[e];
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < BPT; ++e) {
+            const int idx = threadIdx.x + e * SC_THREADS;
+            if (idx < SC_CH * NP) {
+                const bool in = idx % NP < N;
+                b_s[idx / NP][idx % NP] = in ? fb[e] : 0.f;
+                c_s[idx / NP][idx % NP] = in ? fc[e] : 0.f;
+            }
+        }
+        __syncthreads();
+        if (c0 + SC_CH < r1) fetch(c0 + SC_CH, min(SC_CH, r1 - c0 - SC_CH));
+#pragma unroll 4
+        for (int tt = 0; tt < nt; ++tt) {
+            const float d = dt_s[tt][cl], dx = dx_s[tt][cl];
+            float y0 = 0.f, y1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < NPL; i += 4) {
+                const float4 bb = *reinterpret_cast<const float4*>(&b_s[tt][(i >> 2) * 4 * L + part * 4]);
+                const float4 cc = *reinterpret_cast<const float4*>(&c_s[tt][(i >> 2) * 4 * L + part * 4]);
+                S[i] = decay_add(S[i], d * A[i], dx * bb.x);
+                S[i + 1] = decay_add(S[i + 1], d * A[i + 1], dx * bb.y);
+                S[i + 2] = decay_add(S[i + 2], d * A[i + 2], dx * bb.z);
+                S[i + 3] = decay_add(S[i + 3], d * A[i + 3], dx * bb.w);
+                y0 = fmaf(S[i], cc.x, y0); y1 = fmaf(S[i + 1], cc.y, y1);
+                y0 = fmaf(S[i + 2], cc.z, y0); y1 = fmaf(S[i + 3], cc.w, y1);
+            }
+            rd_s[tt][threadIdx.x] = y0 + y1;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int e = 0; e < EPT; ++e) {
+            const int tt = ptt + e * L;
+            if (tt < nt && plive) {
+                float y = 0.f;
+#pragma unroll
+                for (int l = 0; l < L; ++l) y += rd_s[tt][pc * L + l];
+                y = fmaf(skip, x_s[tt][pc], y);
+                const float zz = z_s[tt][pc];
+                reinterpret_cast<T*>(a.out)[(long)(c0 + tt) * a.ldo + pch] = from_f32<T>(y * (zz / (1.0f + expf(-zz))));
+            }
+        }
+    }
+    fx_pdl_trigger();
+    if (live) {
+#pragma unroll
+        for (int i = 0; i < NPL; ++i) {
+            const int n = (i >> 2) * 4 * L + part * 4 + (i & 3);
+            if (n < N) sp[n] = S[i];
+        }
+    }
+}
+
+template <typename T, int L, int NPL>
+int launch_sc(const ScArgs& a, int n_entries, cudaStream_t s)
+{
+    dim3 grid(n_entries, (unsigned)fx_cdiv(a.inner, SC_THREADS / L));
+    // a prompt's recurrence starts on an empty device (see fx_launch_pdl_if); a decode step's is set up early
+    fx_launch_pdl_if(a.n_tokens < 8 * n_entries, selective_scan_kernel<T, L, NPL>, grid, dim3(SC_THREADS), 0, s, a);
+    return fx_launch_status();
+}
+
+template <typename T>
+int scan_for(const ScArgs& a, int n_entries, cudaStream_t s)
+{
+    const int n = a.n_state;
+    if (n <= 4) return launch_sc<T, 1, 4>(a, n_entries, s);
+    if (n <= 8) return launch_sc<T, 2, 4>(a, n_entries, s);
+    if (n <= 16) return launch_sc<T, 4, 4>(a, n_entries, s);
+    if (n <= 32) return launch_sc<T, 8, 4>(a, n_entries, s);
+    if (n <= 64) return launch_sc<T, 8, 8>(a, n_entries, s);
+    if (n <= 128) return launch_sc<T, 16, 8>(a, n_entries, s);
+    return launch_sc<T, 32, 8>(a, n_entries, s);
+}
+
+__global__ void split_rows_kernel(const float* __restrict__ x, long ldx, bf16* __restrict__ out, long ldo, int n_tokens, int n,
+                                  int pad)
+{
+    fx_pdl_wait();
+    const long total = (long)n_tokens * pad;
+    for (long idx = blockIdx.x * (long)blockDim.x + threadIdx.x; idx < total; idx += (long)gridDim.x * blockDim.x) {
+        const long t = idx / pad;
+        const int i = (int)(idx - t * pad);
+        const float v = i < n ? x[t * ldx + i] : 0.f;
+        const bf16 hi = __float2bfloat16_rn(v);
+        out[t * ldo + i] = hi;
+        out[t * ldo + pad + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+}
+
+}  // namespace
+
+extern "C" int fx_selective_scan(const float* dt, long ldt, const void* dt_bias, int db_dtype, const void* x, long ldx,
+                                 const void* z, long ldz, int dtype, const float* bc, long ldbc, const float* a_log,
+                                 const float* d_skip, float* state, void* out, long ldo, const int* token_seq,
+                                 const int* seq_slot, int n_tokens, int n_entries, int inner, int n_state, void* stream)
+{
+    if (n_tokens <= 0 || n_entries <= 0) return FX_OK;
+    if (inner <= 0 || n_state <= 0 || n_state > 256 || fx_cdiv(inner, 4) > 65535) return FX_ERR_SIZE;
+    ScArgs a;
+    a.dt = dt; a.ldt = ldt; a.dt_bias = dt_bias; a.db_dtype = db_dtype; a.x = x; a.ldx = ldx; a.z = z; a.ldz = ldz;
+    a.bc = bc; a.ldbc = ldbc; a.a_log = a_log; a.d_skip = d_skip; a.state = state; a.out = out; a.ldo = ldo;
+    a.token_seq = token_seq; a.seq_slot = seq_slot; a.n_tokens = n_tokens; a.inner = inner; a.n_state = n_state;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == FX_F32) return scan_for<float>(a, n_entries, s);
+    if (dtype == FX_BF16) return scan_for<bf16>(a, n_entries, s);
+    return FX_ERR_DTYPE;
+}
+
+extern "C" int fx_split_rows(const float* x, long ldx, void* out, long ldo, int n_tokens, int n, int pad, void* stream)
+{
+    if (n_tokens <= 0) return FX_OK;
+    if (n <= 0 || pad < n) return FX_ERR_SIZE;
+    long blocks = fx_cdiv((long)n_tokens * pad, 256);
+    if (blocks > fx_sm_count() * 16L) blocks = fx_sm_count() * 16L;
+    fx_launch_pdl(split_rows_kernel, (unsigned)blocks, 256, 0, (cudaStream_t)stream, x, ldx, (bf16*)out, ldo, n_tokens, n, pad);
+    return fx_launch_status();
+}

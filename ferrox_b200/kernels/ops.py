@@ -50,10 +50,10 @@ _SIGNATURES = {
     "fx_gather_rows": [_P, _L, _P, _P, _L, _I, _I, _I, _P],
     "fx_gather_rows_scaled": [_P, _L, _P, _P, _P, _I, _P, _L, _I, _I, _I, _P],
     "fx_paged_attention_ex": [_P, _L, _L, _P, _P, _L, _L, _I, _P, _I, _I, _P, _P, _P, _P, _L, _L, _I, _I, _I, _I, _I, _I, _F,
-                              _F, _P, _I, _P, _I, _I, _P, _L, _P],
+                              _F, _P, _I, _P, _I, _I, _P, _L, _P, _P],
     "fx_general_attention_ok": [_I, _I, _I],
     "fx_general_attention": [_P, _L, _L, _P, _P, _L, _L, _P, _P, _I, _I, _P, _P, _P, _P, _I, _P, _L, _L, _I, _I, _I, _I, _I,
-                             _F, _P, _I, _P, _P, _I, _F, _P, _I, _I, _P, _L, _P],
+                             _F, _P, _I, _P, _P, _I, _F, _P, _I, _I, _P, _L, _P, _P],
     "fx_rotary_mix_store": [_P, _I, _L, _P, _P, _P, _P, _I, _I, _P, _L, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "fx_route_table": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _I, _P],
     "fx_rmsnorm_residual": [_P, _P, _I, _P, _P, _I, _P, _P, _L, _P, _I, _F, _P, _I, _F, _P, _I, _I, _I, _P],
@@ -80,7 +80,14 @@ _SIGNATURES = {
     "fx_gated_group_norm": [_P, _P, _I, _L, _P, _I, _F, _I, _P, _I, _I, _I, _I, _L, _P],
     "fx_general_delta_prep": [_P, _L, _P, _L, _P, _L, _P, _I, _P, _I, _P, _I, _F, _P, _P, _P, _I, _I, _I, _I, _P],
     "fx_general_delta_scan": [_P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P],
-    "fx_input_conv": [_P, _I, _L, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P],
+    "fx_input_conv": [_P, _I, _L, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P, _I, _I, _P],
+    "fx_rotary_norm_store": [_P, _I, _L, _P, _P, _P, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "fx_stream_step": [_P, _I, _I, _P],
+    "fx_embed_streams": [_P, _I, _P, _P, _I, _I, _I, _I, _F, _P, _P],
+    "fx_channel_decay_prep": [_P, _L, _P, _I, _P, _I, _F, _P, _I, _I, _I, _P],
+    "fx_channel_decay_scan": [_P, _L, _P, _L, _P, _L, _P, _F, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
+    "fx_selective_scan": [_P, _L, _P, _I, _P, _L, _P, _L, _I, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P],
+    "fx_split_rows": [_P, _L, _P, _L, _I, _I, _I, _P],
     "fx_mlstm_column_blocks": [_I, _I],
     "fx_mlstm_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _I, _F, _F, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I,
                       _P],
@@ -92,7 +99,7 @@ _SIGNATURES = {
     "fx_relu_square": [_P, _I, _L, _I, _I, _P],
     "fx_prefill_attention": [_P, _L, _P, _P, _P, _I, _I, _P, _I, _P, _P, _L, _I, _I, _I, _I, _F, _F, _P],
     "fx_prefill_attention_tc": [_P, _L, _I, _P, _P, _I, _P, _I, _I, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I, _I, _F, _P, _P, _L,
-                                _P, _P, _P, _P, _I, _P],
+                                _P, _P, _P, _P, _P, _I, _P],
     "fx_router_topk": [_P, _L, _I, _I, _I, _I, _P, _P, _P, _F, _F, _P],
     "fx_moe_align": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _P],
     "fx_gemm_slab_ok": [_I, _I, _I],
@@ -312,6 +319,80 @@ def embed_norm(table, ids, weight, eps, out, status=None, stream=None):
     T = ids.numel()
     call("fx_embed_norm", _ptr(table), code(table), _ptr(ids), _ptr(weight), code(weight), float(eps), _ptr(out), T,
          table.shape[1], table.shape[0], _ptr(status), stream if stream is not None else stream_ptr())
+    return out
+
+
+def embed_streams(table, ids, out, streams, status=None, stream=None, scale=1.0):
+    """``streams`` copies of table[ids[t]] * scale in 32 bits, side by side in row t of ``out``."""
+    if out.shape[1] != streams * table.shape[1]:
+        raise KernelError("embed_streams: the streams of a token lie side by side")
+    call("fx_embed_streams", _ptr(table), code(table), _ptr(ids), _ptr(out), ids.numel(), table.shape[1], table.shape[0],
+         int(streams), float(scale), _ptr(status), stream if stream is not None else stream_ptr())
+    return out
+
+
+MAX_STREAMS = 8
+
+
+class StreamStep(ctypes.Structure):
+    """The arguments of ``fx_stream_step`` (csrc/api.h), by value."""
+
+    _fields_ = [("streams", c_void_p), ("rows", c_void_p), ("y", c_void_p * 3), ("expert_rows", c_void_p),
+                ("place", c_void_p), ("weight", c_void_p), ("shared", c_void_p), ("shared_gate", c_void_p),
+                ("gate_ld", c_long), ("w", c_void_p), ("x_out", c_void_p), ("expert_dtype", c_int), ("w_dtype", c_int),
+                ("x_dtype", c_int), ("top_k", c_int), ("n_terms", c_int), ("write", c_int), ("hidden", c_int),
+                ("eps", c_float), ("mix", c_float * MAX_STREAMS * MAX_STREAMS), ("coef", c_float * MAX_STREAMS * 4),
+                ("reads", c_float * MAX_STREAMS)]
+
+
+def stream_step(h, n_streams, *, terms=(), experts=None, mix=None, read=None, rows=None, stream=None):
+    """A residual of ``n_streams`` streams, ``h`` [T, n_streams * hidden] 32-bit, updated and read in one kernel
+    (csrc/streams.cu).  ``mix`` [from][to] (a list of lists): X_t <- sum_s mix[s][t] X_s + sum_j c_j[t] y_j.  ``terms``:
+    up to three (y_j [T, hidden] 32-bit, c_j) with c_j a list of one number a stream; ``experts`` = ((rows in expert
+    order, inv_perm, weights or None, shared rows or None, its gate's logits or None), c).  ``mix`` None: the streams stay
+    as they are and every c is [one number], the weight of that result in what is read.  ``read`` = (r, weight, eps, out):
+    out = u / sqrt(mean(u^2) + eps) * weight with u = sum_t r[t] X_t on the new streams (without ``mix``: on the streams
+    as they are, plus the results).  ``rows`` (without ``mix``): the tokens that are read.  Returns ``out`` or None."""
+    S = int(n_streams)
+    if h.dtype != torch.float32 or not h.is_contiguous() or not 1 <= S <= MAX_STREAMS or h.shape[1] % S:
+        raise KernelError(f"stream_step: a contiguous 32-bit residual of 1 to {MAX_STREAMS} streams")
+    W = h.shape[1] // S
+    T = h.shape[0]
+    if len(terms) > 3:
+        raise KernelError("stream_step: at most three results of a sublayer beside the experts'")
+    a = StreamStep(streams=_ptr(h), rows=_ptr(rows), hidden=W, write=int(mix is not None))
+    if mix is not None:
+        for s in range(S):
+            for t in range(S):
+                a.mix[s][t] = mix[s][t]
+    n_coef = S if mix is not None else 1
+    for j, (y, c) in enumerate(terms):
+        if y.dtype != torch.float32 or y.shape != (T, W) or not y.is_contiguous() or len(c) != n_coef:
+            raise KernelError("stream_step: a sublayer's result is contiguous, 32-bit, one row a token, and has one weight a stream")
+        a.y[j] = _ptr(y)
+        for s in range(n_coef):
+            a.coef[j][s] = c[s]
+    a.n_terms = len(terms)
+    if experts is not None:
+        (y, place, wts, shared, gate), c = experts
+        if not y.is_contiguous() or y.shape[-1] != W or len(c) != n_coef or (shared is not None and (
+                shared.dtype != y.dtype or not shared.is_contiguous())):
+            raise KernelError("stream_step: contiguous rows of the experts, the shared one's of their element type")
+        a.expert_rows, a.expert_dtype, a.place, a.weight = _ptr(y), code(y), _ptr(place), _ptr(wts)
+        a.top_k, a.shared, a.shared_gate = place.numel() // T, _ptr(shared), _ptr(gate)
+        a.gate_ld = gate.stride(0) if gate is not None else 0
+        for s in range(n_coef):
+            a.coef[3][s] = c[s]
+    out, n = None, T
+    if read is not None:
+        r, w, eps, out = read
+        for s in range(S):
+            a.reads[s] = r[s]
+        a.w, a.w_dtype, a.eps, a.x_out, a.x_dtype = _ptr(w), code(w), float(eps), _ptr(out), code(out)
+        n = out.shape[0]
+        if n != (rows.numel() if rows is not None else T) or out.shape[1] != W or not out.is_contiguous():
+            raise KernelError("stream_step: one contiguous output row for every token that is read")
+    call("fx_stream_step", ctypes.cast(ctypes.byref(a), c_void_p), S, n, stream if stream is not None else stream_ptr())
     return out
 
 
@@ -542,6 +623,64 @@ def general_delta_scan(r, k, v, u, au, w, state, out, token_seq, seq_slot, n_ent
     return out
 
 
+CHANNEL_DECAY_MAX_DIM = 256
+
+
+def channel_decay_prep(low, w2, bias, tau, alpha, stream=None):
+    """alpha = sigmoid(w2 . low + bias)^(1 / tau): ``low`` 32-bit row views [T, rank], ``w2`` [channels, rank], ``alpha``
+    contiguous 32-bit [T, channels]; all arithmetic 32-bit."""
+    if low.dtype != torch.float32 or alpha.dtype != torch.float32 or not alpha.is_contiguous() or not w2.is_contiguous():
+        raise KernelError("channel_decay_prep: what enters the recurrence is 32-bit, matrices are contiguous")
+    call("fx_channel_decay_prep", _ptr(low), _rows(low), _ptr(w2), code(w2), _ptr(bias), code(bias), 1.0 / float(tau),
+         _ptr(alpha), low.shape[0], w2.shape[0], w2.shape[1], stream if stream is not None else stream_ptr())
+    return alpha
+
+
+def channel_decay_scan(q, k, v, alpha, q_scale, state, out, token_seq, seq_slot, n_entries, H, D, V, stream=None):
+    """Linear attention with a decay per key channel over every entry's tokens in order: S = diag(alpha) S + k v^T,
+    out = q_scale S^T q.  ``q``, ``k`` [T, H*D], ``v`` [T, H*V] 32-bit row views; ``alpha`` contiguous [T, H*D];
+    ``state`` [slots, H, D, V] and ``out`` [T, H*V] 32-bit."""
+    for t in (q, k, v, alpha, state, out):
+        if t.dtype != torch.float32:
+            raise KernelError("channel_decay_scan: the recurrence is 32-bit")
+    call("fx_channel_decay_scan", _ptr(q), _rows(q), _ptr(k), _rows(k), _ptr(v), _rows(v), _ptr(alpha), float(q_scale),
+         _ptr(state), _ptr(out), _rows(out), _ptr(token_seq), _ptr(seq_slot), q.shape[0], int(n_entries), int(H), int(D),
+         int(V), stream if stream is not None else stream_ptr())
+    return out
+
+
+SELECTIVE_SCAN_MAX_STATE = 256
+
+
+def selective_scan(dt, dt_bias, x, z, bc, a_log, d_skip, state, out, token_seq, seq_slot, n_entries, stream=None):
+    """The selective state space over every entry's tokens in order (csrc/selective_scan.cu): ``dt`` [T, inner] 32-bit
+    before bias and softplus, ``x`` and ``z`` row views [T, inner] of the engine's element type, ``bc`` 32-bit row views
+    [T, B | C], ``a_log`` [inner, n_state] and ``d_skip`` [inner] 32-bit, ``state`` [slots, inner, n_state] 32-bit;
+    ``out`` [T, inner] = (S C + D x) silu(z)."""
+    for t in (dt, bc, a_log, d_skip, state):
+        if t.dtype != torch.float32:
+            raise KernelError("selective_scan: the recurrence is 32-bit")
+    if x.dtype != z.dtype or x.dtype != out.dtype:
+        raise KernelError("selective_scan: x, z and the result share one element type")
+    inner, n_state = a_log.shape
+    if not (a_log.is_contiguous() and d_skip.is_contiguous() and bc.shape[1] == 2 * n_state):
+        raise KernelError("selective_scan: contiguous constants, rows of [B | C]")
+    call("fx_selective_scan", _ptr(dt), _rows(dt), _ptr(dt_bias), code(dt_bias), _ptr(x), _rows(x), _ptr(z), _rows(z), code(x),
+         _ptr(bc), _rows(bc), _ptr(a_log), _ptr(d_skip), _ptr(state), _ptr(out), _rows(out), _ptr(token_seq),
+         _ptr(seq_slot), x.shape[0], int(n_entries), int(inner), int(n_state), stream if stream is not None else stream_ptr())
+    return out
+
+
+def split_rows(x, out, stream=None):
+    """``out`` bfloat16 [T, 2 * pad] = [hi | lo] with hi + lo = ``x`` (32-bit row views [T, n], n <= pad; zeros beyond n)
+    to sixteen bits of mantissa: rows for a product on the tensor cores that must not lose them to rounding."""
+    if x.dtype != torch.float32 or out.dtype != torch.bfloat16 or out.shape[1] % 2:
+        raise KernelError("split_rows: 32-bit rows into pairs of bfloat16 halves")
+    call("fx_split_rows", _ptr(x), _rows(x), _ptr(out), _rows(out), x.shape[0], x.shape[1], out.shape[1] // 2,
+         stream if stream is not None else stream_ptr())
+    return out
+
+
 def mlstm_column_blocks(head_dim: int, value_dim: int) -> int:
     """Blocks of value columns :func:`mlstm_scan` shares a head's state out over: the copies of the normaliser and of
     the running maximum that the state keeps.  A function of the two sizes alone, stated here as the kernel's
@@ -605,16 +744,17 @@ def diff_combine(attn, out, n_heads, group, value_dim, lam, eps, post, stream=No
     return out
 
 
-def input_conv(x, weight, taps, tail, token_seq, seq_slot, out, update_tail=False, stream=None, add_input=True):
+def input_conv(x, weight, taps, tail, token_seq, seq_slot, out, update_tail=False, stream=None, add_input=True, bias=None,
+               silu=False):
     """out[t] = x[t] + sum_j weight[:, j] x[t - taps + 1 + j] over the tokens of each request (``weight`` [channels,
     taps]); the inputs before the step come from ``tail`` [slots, taps - 1, channels] 32-bit.  ``update_tail``: only
     when every entry brings exactly one token; the kernel then also moves the tail on (:func:`conv_tail_update`
-    otherwise).  ``add_input`` False: the sum alone."""
+    otherwise).  ``add_input`` False: the sum alone; ``bias`` [channels]: added to it; ``silu``: SiLU of the result."""
     if out.dtype != x.dtype or out.data_ptr() == x.data_ptr():
         raise KernelError("input_conv: an output of its own, of the input's element type")
     call("fx_input_conv", _ptr(x), code(x), _rows(x), _ptr(weight), code(weight), int(taps), _ptr(tail), _ptr(token_seq),
-         _ptr(seq_slot), _ptr(out), _rows(out), x.shape[0], x.shape[1], int(update_tail), int(add_input),
-         stream if stream is not None else stream_ptr())
+         _ptr(seq_slot), _ptr(out), _rows(out), x.shape[0], x.shape[1], int(update_tail), int(add_input), _ptr(bias),
+         code(bias) if bias is not None else 0, int(silu), stream if stream is not None else stream_ptr())
     return out
 
 
@@ -755,9 +895,15 @@ def paged_attention(q, k_pages, v_pages, block_table, page_size, positions, toke
     return out
 
 
+def _check_turn(turn, n_tokens, value_dim):
+    if turn is not None and (turn.dtype != torch.float32 or not turn.is_contiguous() or turn.numel() != n_tokens * value_dim
+                             or value_dim % 2):
+        raise KernelError("attention: the results' angles are contiguous 32-bit (cos, sin) pairs [tokens, value_dim / 2, 2]")
+
+
 def paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, page_size, positions, token_seq, seq_slot,
                        out, ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim, window, scale, softcap=None, slopes=None,
-                       stream=None, keep_first=0, sinks=None, value_share=1, chunk=None, gate=None):
+                       stream=None, keep_first=0, sinks=None, value_share=1, chunk=None, gate=None, turn=None):
     """:func:`paged_attention` in its general form: keys of ``key_dim`` and values of ``value_dim`` elements whose
     positions lie ``ldk`` / ``ldv`` elements apart in their pages (values that are the leading part of the cached
     key rows: the same tensor twice with ldv = ldk); ``q`` and ``out`` are any tensors addressed by a token stride
@@ -766,8 +912,10 @@ def paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pa
     the window; ``sinks`` (float32 [n_heads], optional): exp(sinks[h]) joins the softmax's denominator once;
     ``value_share``: that many consecutive key heads read one value head (the value pages hold n_kv_heads /
     value_share heads); ``chunk``: a query sees the keys of its own chunk of that many positions only, counted from
-    the request's start; ``gate`` (token rows of n_heads * value_dim, of q's element type, optional): the result is
-    multiplied by sigmoid(gate)."""
+    the request's start; ``turn`` (float32 [T, value_dim / 2, 2] (cos, sin), optional): pair (2m, 2m + 1) of every head's
+    result is turned by minus that angle; ``gate`` (token rows of n_heads * value_dim, of q's element type, optional):
+    the result is then multiplied by sigmoid(gate)."""
+    _check_turn(turn, positions.numel(), value_dim)
     T = positions.numel()
     if gate is not None and gate.dtype != q.dtype:
         raise KernelError("paged_attention_ex: the gate has the queries' element type")
@@ -779,7 +927,7 @@ def paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pa
          _ptr(block_table), block_table.shape[1], page_size, _ptr(positions), _ptr(token_seq), _ptr(seq_slot), _ptr(out),
          int(ldo), int(ldoh), T, n_heads, n_kv_heads, key_dim, value_dim, int(window or 0), float(scale),
          float(softcap or 0.0), _ptr(slopes), int(keep_first or 0), _ptr(sinks), int(value_share), int(chunk or 0),
-         _ptr(gate), _rows(gate) if gate is not None else 0, stream if stream is not None else stream_ptr())
+         _ptr(gate), _rows(gate) if gate is not None else 0, _ptr(turn), stream if stream is not None else stream_ptr())
     return out
 
 
@@ -830,7 +978,7 @@ def general_attention_items(entries, n_heads: int, n_kv_heads: int):
 def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, page_size, positions, token_seq, seq_slot,
                       items, out, ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim, window, scale, slopes=None,
                       stream=None, n_splits=1, part_o=None, part_ml=None, kv_strides=None, keep_first=0, softcap=None,
-                      sinks=None, value_share=1, chunk=None, gate=None):
+                      sinks=None, value_share=1, chunk=None, gate=None, turn=None):
     """:func:`paged_attention_ex` in bfloat16 on the tensor cores (see :func:`general_attention_ok`).  ``items``: the
     device copy of :func:`general_attention_items`, or None when every entry brings one token (a tile a token and
     kv head; nothing comes from the host, so a captured step replays unchanged).  ``n_splits`` > 1 (without items):
@@ -838,8 +986,9 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pag
     value_dim] and ``part_ml`` float32 [T, heads, n_splits, 2] are scratch, and a second kernel adds the runs up.
     ``kv_strides`` = (k page stride, k head stride, v page stride, v head stride) in elements, for keys and values that
     do not lie [page][kv head][position][ld] (rows that hold all heads side by side); ``ldk`` / ``ldv`` stay the
-    distance between two positions.  ``softcap``, ``sinks``, ``value_share``, ``chunk``, ``gate``: as
-    :func:`paged_attention_ex`."""
+    distance between two positions.  ``softcap``, ``sinks``, ``value_share``, ``chunk``, ``gate``, ``turn``:
+    as :func:`paged_attention_ex`."""
+    _check_turn(turn, positions.numel(), value_dim)
     if gate is not None and gate.dtype != q.dtype:
         raise KernelError("general_attention: the gate has the queries' element type")
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads):
@@ -854,7 +1003,7 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, block_table, pag
          _ptr(items), n, _ptr(out), int(ldo), int(ldoh), n_heads, n_kv_heads, key_dim, value_dim, int(window or 0),
          float(scale), _ptr(slopes), int(n_splits), _ptr(part_o), _ptr(part_ml), int(keep_first or 0),
          float(softcap or 0.0), _ptr(sinks), int(value_share), int(chunk or 0), _ptr(gate),
-         _rows(gate) if gate is not None else 0, stream if stream is not None else stream_ptr())
+         _rows(gate) if gate is not None else 0, _ptr(turn), stream if stream is not None else stream_ptr())
     return out
 
 
@@ -890,6 +1039,20 @@ def rotary_mix_store(qkv, positions, token_seq, seq_slot, cos_sin, rot_dims, pai
          float(lam), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], page_size, qkv.shape[0],
          n_heads, n_kv_heads, key_dim, value_dim, int(write_cache), _ptr(status),
          stream if stream is not None else stream_ptr())
+
+
+def rotary_norm_store(qkv, positions, token_seq, seq_slot, cos_sin, rot_dims, pairing, eps, v_cos_sin, k_pages, v_pages,
+                      block_table, page_size, n_heads, n_kv_heads, key_dim, value_dim, write_cache=True, status=None,
+                      stream=None):
+    """Rows of [q heads | k heads | v heads] (widths key_dim, key_dim, value_dim): the first ``rot_dims`` elements of
+    every q and k head turned by ``cos_sin`` [T, rot_dims / 2, 2] (None: no rotation), then, ``eps`` given, every q and k
+    head divided by its root mean square; the values turned on neighbouring pairs by ``v_cos_sin`` [T, value_dim / 2, 2]
+    (None: as they are).  q in place, k and v into their pages; the rows' own k and v stay as projected."""
+    _check_turn(v_cos_sin, qkv.shape[0], value_dim)
+    call("fx_rotary_norm_store", _ptr(qkv), code(qkv), _rows(qkv), _ptr(positions), _ptr(token_seq), _ptr(seq_slot),
+         _ptr(cos_sin), int(rot_dims), int(pairing), float(eps) if eps is not None else -1.0, _ptr(v_cos_sin),
+         _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], page_size, qkv.shape[0], n_heads,
+         n_kv_heads, key_dim, value_dim, int(write_cache), _ptr(status), stream if stream is not None else stream_ptr())
 
 
 def latent_prep(q, dkv, positions, token_seq, seq_slot, c_weight, eps, cos_sin, rot_dims, q_plain, q_full, pages,
@@ -1061,10 +1224,10 @@ def prefill_tc_plan(entries, window, n_heads: int, sms: int = 0, run_blocks: int
 
 def prefill_attention_tc(q, k_pages, v_pages, block_table, page_size, items, seq_slot, out, n_heads, n_kv_heads,
                          head_dim, window, scale, status=None, stream=None, merges=None, part_o=None, part_ml=None,
-                         value_dim=None, chunk=None, sinks=None, gate=None):
+                         value_dim=None, chunk=None, sinks=None, gate=None, turn=None):
     """Flash attention of prompt portions on the tcgen05 tensor cores (bfloat16, keys and values of up to 128 elements
-    in steps of 8, pages of a multiple of 64 positions).  ``value_dim``, ``chunk``, ``sinks``, ``gate``: as
-    :func:`paged_attention_ex`.  ``items``, ``merges``: device copies of what :func:`prefill_tc_plan` returns;
+    in steps of 8, pages of a multiple of 64 positions).  ``value_dim``, ``chunk``, ``sinks``, ``gate``,
+    ``turn``: as :func:`paged_attention_ex`.  ``items``, ``merges``: device copies of what :func:`prefill_tc_plan` returns;
     ``part_o`` float32 [parts, n_heads, 256, :func:`prefill_value_width`] and ``part_ml`` float32 [parts, n_heads, 256, 2]: scratch for the
     tiles that were cut into runs of key blocks (a second kernel adds the runs up)."""
     global _launches
@@ -1074,7 +1237,7 @@ def prefill_attention_tc(q, k_pages, v_pages, block_table, page_size, items, seq
     call("fx_prefill_attention_tc", _ptr(q), _rows(q), q.shape[0], _ptr(k_pages), _ptr(v_pages), k_pages.shape[0],
          _ptr(block_table), block_table.shape[1], page_size, _ptr(items), items.shape[0], _ptr(seq_slot), _ptr(out),
          _rows(out), n_heads, n_kv_heads, head_dim, int(value_dim or head_dim), int(window or 0), int(chunk or 0), float(scale),
-         _ptr(sinks), _ptr(gate), _rows(gate) if gate is not None else 0, _ptr(status),
+         _ptr(sinks), _ptr(gate), _rows(gate) if gate is not None else 0, _ptr(turn), _ptr(status),
          _ptr(part_o) if n_merges else None, _ptr(part_ml) if n_merges else None, _ptr(merges) if n_merges else None,
          n_merges, stream if stream is not None else stream_ptr())
     return out
@@ -1212,22 +1375,22 @@ def decode_store_ok(qkv, k_pages, head_dim: int, page_size: int) -> bool:
 
 
 class DecodeExtras(ctypes.Structure):
-    """Options of the decode attention kernel that streams pages by TMA (csrc/api.h): ``chunk``, ``sinks``, ``gate`` as
-    :func:`paged_attention_ex`; with ``store_new`` the first ``rot`` elements of a head are rotated (0: all of it) and
+    """Options of the decode attention kernel that streams pages by TMA (csrc/api.h): ``chunk``, ``sinks``, ``gate``,
+    ``turn`` as :func:`paged_attention_ex`; with ``store_new`` the first ``rot`` elements of a head are rotated (0: all of it) and
     the stored value is (1 - lam) v + lam v_first as :func:`rotary_mix_store` says."""
 
     _fields_ = [("chunk", c_int), ("rot", c_int), ("sinks", c_void_p), ("gate", c_void_p), ("ldg", c_long),
-                ("v_first", c_void_p), ("ld_first", c_long), ("lam", c_float)]
+                ("v_first", c_void_p), ("ld_first", c_long), ("lam", c_float), ("turn", c_void_p)]
 
     @classmethod
-    def of(cls, chunk=None, sinks=None, gate=None, rot=0, v_first=None, lam=0.0):
+    def of(cls, chunk=None, sinks=None, gate=None, rot=0, v_first=None, lam=0.0, turn=None):
         if sinks is not None and sinks.dtype != torch.float32:
             raise KernelError("decode_attention: one 32-bit sink per head")
         for t in (gate, v_first):
             if t is not None and t.dtype != torch.bfloat16:
                 raise KernelError("decode_attention: the gate and the other layer's values are bfloat16 rows")
         return cls(int(chunk or 0), int(rot), _ptr(sinks), _ptr(gate), _rows(gate) if gate is not None else 0,
-                   _ptr(v_first), _rows(v_first) if v_first is not None else 0, float(lam))
+                   _ptr(v_first), _rows(v_first) if v_first is not None else 0, float(lam), _ptr(turn))
 
 
 def decode_attention(q, k_pages, v_pages, block_table, page_size, positions, token_seq, seq_slot, out, n_heads,

@@ -20,7 +20,7 @@ from ..cache.specs import CacheSpec, KvCacheSpec, PagedSpec, PagedTensorSpec, St
 from ..kernels import ops
 from ..weights.loader import TensorDecl
 from .base import Mixer, build_part, register_part
-from .specs import NoPositionSpec
+from .specs import NoPositionSpec, ScaledRotarySpec
 
 
 RANGE_COUNTERS = 16384            # (token, block of heads) pairs of a decode step whose key ranges one kernel merges
@@ -96,13 +96,28 @@ class GqaAttention(Mixer):
         self.chunk = getattr(s, "chunk", None)
         self.sink_name = getattr(s, "sink", None)
         self.mix = getattr(s, "value_mix", None)
+        self.rotated_norm_eps = getattr(s, "rotated_norm_eps", None)
+        self.turn_spec = getattr(s, "value_turn", None)
+        self.o_bias = bool(getattr(s, "o_bias", False))
         if self.chunk is not None and (self.chunk < 1 or s.window is not None):
             raise ValueError(f"chunk={self.chunk}: a positive number of positions, without a window")
         if int(getattr(s, "keep_first", 0) or 0) < 0:
             raise ValueError(f"keep_first={s.keep_first}: a number of positions")
         prepared = bool(self.qk_norm or self.temperature or self.value_norm_eps is not None)    # by qk_norm_store
         self.general = bool(prepared or self.slopes_spec or self.value_dim != s.head_dim or self.keep_first
-                            or self.gate_name or self.chunk or self.sink_name or self.mix)
+                            or self.gate_name or self.chunk or self.sink_name or self.mix
+                            or self.rotated_norm_eps is not None or self.turn_spec)
+        # queries and keys normed behind their rotation, values turned by position: a kernel of their own stands between
+        # projection and attention (rotary_norm_store)
+        self.rotates_and_norms = bool(self.rotated_norm_eps is not None or self.turn_spec)
+        self.turn = None
+        if self.turn_spec:
+            if self.value_dim % 2:
+                raise ValueError(f"value_dim={self.value_dim}: values that are turned consist of pairs")
+            if self.turn_spec[1] not in ("halves", "adjacent"):
+                raise ValueError(f"value_turn pairing {self.turn_spec[1]!r}: halves or adjacent")
+            # (the frequencies and the table of a rotary part over the value head's width)
+            self.turn = build_part(ScaledRotarySpec(rotary_dim=self.value_dim, theta=float(self.turn_spec[0])))
         # in the general form a rotary part's tables serve the kernel that also mixes the values (rotary_mix_store)
         self.rotates = self.general and s.position is not None and not isinstance(s.position, NoPositionSpec)
         if self.general:
@@ -114,6 +129,9 @@ class GqaAttention(Mixer):
         self.v_size = s.n_kv_heads * self.value_dim
         self.o_size = s.n_heads * self.value_dim
         if self.general:
+            if self.rotates_and_norms and (prepared or self.mix):
+                raise ValueError("attention that norms behind the rotation or turns its values has neither weighted norms of "
+                                 "queries and keys nor mixed values")
             if prepared and (self.rotates or self.mix):
                 raise ValueError("attention with normed queries, keys or values or a query temperature takes no rotary "
                                  "position encoding and no mixing of values")
@@ -133,7 +151,7 @@ class GqaAttention(Mixer):
         if self.softcap is not None and self.softcap < 0:
             raise ValueError(f"softcap={s.softcap}: the cap of the scores is positive")
         names = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight",
-                     q_bias="q_proj.bias", k_bias="k_proj.bias", v_bias="v_proj.bias")
+                     q_bias="q_proj.bias", k_bias="k_proj.bias", v_bias="v_proj.bias", o_bias="o_proj.bias")
         names.update(dict(s.tensor_names or ()))
         self._names = {key: s.prefix + n for key, n in names.items()}
         # tied values: the v rows of the fused product are the k rows once more, so that every kernel after it
@@ -159,6 +177,8 @@ class GqaAttention(Mixer):
                   TensorDecl(s.prefix + self.qk_norm[1], (s.head_dim,), init="ones")]
         if s.qkv_bias:
             d += [TensorDecl(n[key + "_bias"], (sizes[key],)) for key in keys]
+        if self.o_bias:
+            d.append(TensorDecl(n["o_bias"], (s.hidden,)))
         if self.gate_name:
             d.append(TensorDecl(s.prefix + self.gate_name, (self.o_size, s.hidden)))
         if self.sink_name:
@@ -167,24 +187,46 @@ class GqaAttention(Mixer):
             d.append(TensorDecl(s.prefix + self.mix.name, (), optional=self.mix.source))
         return d
 
+    def _pairs_together(self, heads: int, device):
+        """Values turned on pairs (m, m + value_dim/2): the order of a row of ``heads`` value heads in which the two
+        elements of a pair are neighbours, so that every kernel has both in one thread's hands.  The rows of Wv and of the
+        gate and the columns of Wo take this order when they are loaded; nothing behind Wo sees it.  None: as stored."""
+        if not self.turn_spec or self.turn_spec[1] == "adjacent":
+            return None
+        V = self.value_dim
+        own = torch.arange(V, device=device).reshape(2, V // 2).T.reshape(-1)
+        return (torch.arange(heads, device=device)[:, None] * V + own[None, :]).reshape(-1)
+
     def load(self, src, rt):
         super().load(src, rt)
         n = self._names
         ws = [src.get(n[key]) for key in self._qkv_keys]
+        kv_order = self._pairs_together(self.spec.n_kv_heads, rt.device)
+        q_order = self._pairs_together(self.spec.n_heads, rt.device)
+        if kv_order is not None:
+            ws[2] = ws[2][kv_order]
         if self.gate_name:
             # the output gate reads the same input as q, k and v: its rows follow theirs in the fused product
-            ws.append(src.get(self.spec.prefix + self.gate_name))
+            g = src.get(self.spec.prefix + self.gate_name)
+            ws.append(g if q_order is None else g[q_order])
         dt = _common_dtype(ws)
         self.w_qkv = torch.cat([w.to(dt) for w in ws], dim=0).contiguous()
         self.b_qkv = None
         if self.spec.qkv_bias:
             bs = [src.get(n[key + "_bias"]) for key in self._qkv_keys]
+            if kv_order is not None:
+                bs[2] = bs[2][kv_order]
             if self.gate_name:
                 bs.append(torch.zeros(self.o_size, dtype=bs[0].dtype, device=bs[0].device))    # (the gate has no bias)
             bdt = _common_dtype(bs)
             self.b_qkv = torch.cat([b.to(bdt) for b in bs]).contiguous()
         self.w_o = src.get(n["o"])
+        if q_order is not None:
+            self.w_o = self.w_o[:, q_order].contiguous()
+        self.b_o = src.get(n["o_bias"]) if self.o_bias else None
         self.position.load(src, rt)
+        if self.turn is not None:
+            self.turn.load(src, rt)
         self.q_norm_w = self.k_norm_w = self.slopes = None
         if self.qk_norm:
             ws = [src.get(self.spec.prefix + self.qk_norm[0]), src.get(self.spec.prefix + self.qk_norm[1])]
@@ -282,16 +324,16 @@ class GqaAttention(Mixer):
                 softcap=self.softcap,
             )
         # (the attention's last blocks only add up key ranges: the memory system is idle under them)
-        ops.linear(attn, self.w_o, h, accumulate=accumulate, status=batch.status, stream=batch.stream,
+        ops.linear(attn, self.w_o, h, bias=self.b_o, accumulate=accumulate, status=batch.status, stream=batch.stream,
                    after_short_kernel=True)
-
 
     def _forward_general(self, x, out, batch, cache, accumulate):
         """The form with normed queries, keys or values, a query temperature, a distance bias, kept first positions,
-        chunks, sinks, an output gate, values of their own width or mixed across layers: fused [q | k | v (| gate)]
-        product; one kernel norms q and k (and v) per head, applies the temperature and stores k and v, or rotates q
-        and k, mixes v and stores k and v; attention with the bias and the mask, whose epilogue applies the gate;
-        output product."""
+        chunks, sinks, an output gate, values of their own width, mixed across layers or turned by their position: fused
+        [q | k | v (| gate)] product; one kernel norms q and k (and v) per head, applies the temperature and stores k and
+        v, or rotates q and k, mixes v and stores k and v, or rotates and norms q and k, turns v and stores k and v;
+        attention with the bias and the mask, whose epilogue turns the result back and applies the gate; output
+        product."""
         s = self.spec
         T, D, V = x.shape[0], s.head_dim, self.value_dim
         qkv_width = self.q_size + self.kv_size + self.v_size
@@ -304,7 +346,16 @@ class GqaAttention(Mixer):
         by_tma = direct and few and ops.decode_store_ok(qkv, cache.k, D, cache.page_size)
         in_kernel = False
         first = self._values_of_first_layer(qkv, qkv_width, batch)
-        if self.rotates or self.mix:
+        turn = None
+        if self.rotates_and_norms:
+            cos_sin = self.position.table(batch) if self.rotates else None
+            turn = self.turn.table(batch) if self.turn is not None else None
+            ops.rotary_norm_store(qkv, batch.positions, batch.token_seq, batch.seq_slot, cos_sin,
+                                  self.position.rotary_dim if self.rotates else 0,
+                                  self.position.pairing if self.rotates else ops.PAIR_HALVES, self.rotated_norm_eps, turn,
+                                  cache.k, cache.v, cache.block_table, cache.page_size, s.n_heads, s.n_kv_heads, D, V,
+                                  write_cache=cache.writes, status=batch.status, stream=batch.stream)
+        elif self.rotates or self.mix:
             cos_sin = self.position.table(batch) if self.rotates else None
             rot = self.position.rotary_dim if self.rotates else 0
             pairing = self.position.pairing if self.rotates else ops.PAIR_HALVES
@@ -323,7 +374,7 @@ class GqaAttention(Mixer):
                               value_norm_eps=self.value_norm_eps)
         attn = self.rt.empty(T, self.o_size)
         if by_tma:
-            extras = ops.DecodeExtras.of(self.chunk, self.sinks, gate, *((rot, first, self.lam) if in_kernel else ()))
+            extras = ops.DecodeExtras.of(self.chunk, self.sinks, gate, *((rot, first, self.lam) if in_kernel else ()), turn=turn)
             self._decode_by_tma(qkv, attn, batch, cache, in_kernel, cos_sin if in_kernel else None, extras)
         elif (not few and not self.slopes_spec and not self.keep_first
               and ops.prefill_tc_ok(qkv, attn, cache.k, cache.page_size, D, V, self.scale)):
@@ -335,12 +386,12 @@ class GqaAttention(Mixer):
             ops.prefill_attention_tc(qkv, cache.k, cache.v, cache.block_table, cache.page_size, items, batch.seq_slot, attn,
                                      s.n_heads, s.n_kv_heads, D, s.window, self.scale, status=batch.status,
                                      stream=batch.stream, merges=merges, part_o=part_o, part_ml=part_ml, value_dim=V,
-                                     chunk=self.chunk, sinks=self.sinks, gate=gate)
+                                     chunk=self.chunk, sinks=self.sinks, gate=gate, turn=turn)
         else:
             general_attention(qkv, qkv.stride(0), D, cache.k, cache.v, D, V, attn, attn.stride(0), V, batch, cache,
                               s.n_heads, s.n_kv_heads, D, V, s.window, self.scale, self.slopes, self.rt,
-                              keep_first=self.keep_first, sinks=self.sinks, chunk=self.chunk, gate=gate)
-        ops.linear(attn, self.w_o, out, accumulate=accumulate, status=batch.status, stream=batch.stream,
+                              keep_first=self.keep_first, sinks=self.sinks, chunk=self.chunk, gate=gate, turn=turn)
+        ops.linear(attn, self.w_o, out, bias=self.b_o, accumulate=accumulate, status=batch.status, stream=batch.stream,
                    after_short_kernel=True)
 
     def _decode_by_tma(self, qkv, attn, batch, cache, store_new, cos_sin, extras):
@@ -379,11 +430,11 @@ class GqaAttention(Mixer):
 
 def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, batch, cache, n_heads, n_kv_heads,
                       key_dim, value_dim, window, scale, slopes, rt, keep_first=0, softcap=None, sinks=None,
-                      value_share=1, chunk=None, gate=None):
+                      value_share=1, chunk=None, gate=None, turn=None):
     """Attention over pages in its general form (keys and values of different widths, strided queries and outputs, an
     optional distance bias, a window that may keep the request's first positions visible, chunks, capped scores, a
-    learned number per head in the softmax's denominator, key heads that share value heads, a result multiplied by the
-    sigmoid of a gate), by the kernel that fits the step: tiles of (token, head) pairs on the tensor cores
+    learned number per head in the softmax's denominator, key heads that share value heads, a result turned back by
+    the query's position, a result multiplied by the sigmoid of a gate), by the kernel that fits the step: tiles of (token, head) pairs on the tensor cores
     in bfloat16, a warp per (token, head) on the CUDA cores in 32-bit and for widths that are no multiple of 16."""
     per_sm = ops.general_attention_ok(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, key_dim, value_dim)
     if per_sm:
@@ -413,11 +464,12 @@ def general_attention(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, out, ldo, ldoh, 
                                      batch.positions, batch.token_seq, batch.seq_slot, items, out, ldo, ldoh, n_heads,
                                      n_kv_heads, key_dim, value_dim, window, scale, slopes=slopes, stream=batch.stream,
                                      n_splits=n_splits, part_o=part_o, part_ml=part_ml, keep_first=keep_first,
-                                     softcap=softcap, sinks=sinks, value_share=value_share, chunk=chunk, gate=gate)
+                                     softcap=softcap, sinks=sinks, value_share=value_share, chunk=chunk, gate=gate,
+                                     turn=turn)
     ops.paged_attention_ex(q, ldq, ldqh, k_pages, v_pages, ldk, ldv, cache.block_table, cache.page_size, batch.positions,
                            batch.token_seq, batch.seq_slot, out, ldo, ldoh, n_heads, n_kv_heads, key_dim, value_dim,
                            window, scale, slopes=slopes, stream=batch.stream, keep_first=keep_first, softcap=softcap,
-                           sinks=sinks, value_share=value_share, chunk=chunk, gate=gate)
+                           sinks=sinks, value_share=value_share, chunk=chunk, gate=gate, turn=turn)
 
 
 class DifferentialAttention(Mixer):

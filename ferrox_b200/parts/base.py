@@ -147,6 +147,11 @@ class FeedForward(Part):
     # None if it left that norm to the caller.
     fuses_post_norm = False
 
+    # A feed-forward that can leave its result spread over the rows of the tokens' experts, for a kernel of the block's that
+    # adds them up itself, sets ``gives_rows`` and has ``expert_rows(x, batch)``: (rows in expert order, each (token,
+    # rank) pair's row, weights or None, the shared expert's rows or None, its gate's logits or None).
+    gives_rows = False
+
     def forward_add(self, x, h, batch) -> None:  # pragma: no cover - interface
         raise NotImplementedError
 

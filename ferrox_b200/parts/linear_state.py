@@ -26,6 +26,12 @@ gates' logarithms (m starts at 0),
 
 with q = Wq x head_dim^(-1/2); each head's o is RMS-normed, the concatenated heads weighted and gated by sigmoid(Wg x).
 
+``gated_linear_attention``:  per head a state S [head_dim, value_dim] with a decay per key channel,
+
+    S <- diag(alpha) S + k v^T;   o = S^T q,   alpha = sigmoid(W2 W1 x + b)^(1/tau),   q = Wq x head_dim^(-1/2)
+
+each head's o is RMS-normed, weighted by one vector that the heads share and gated by SiLU(Wg x).
+
 The states live in the cache manager's slots as 32-bit tensors; the recurrences, the gates and the norms are
 32-bit (``csrc/linear_state.cu``); the projections run in the engine's dtype.  Tokens of a request are taken in
 order whatever the step looks like, so a position's output does not depend on how the request was cut.
@@ -293,6 +299,67 @@ class Mlstm(_StateMixer):
         ops.linear(y, self.w_o, out, accumulate=accumulate, status=batch.status, stream=batch.stream)
 
 
+class GatedLinearAttention(_StateMixer):
+    """One product for everything the mixer reads from its input, rows [q | k | v | gate | low], written in 32 bits (all
+    but the gate enters the recurrence); ``ops.channel_decay_prep`` (alpha), ``ops.channel_decay_scan`` (state, read-out);
+    ``ops.gated_group_norm`` (per-head RMS, weight, SiLU gate); output product."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        s = spec
+        if s.head_dim > ops.CHANNEL_DECAY_MAX_DIM:
+            raise ValueError(f"head_dim={s.head_dim}: the recurrence kernel holds at most {ops.CHANNEL_DECAY_MAX_DIM} rows of a "
+                             "state column")
+        if not s.tau > 0 or s.decay_rank < 1:
+            raise ValueError(f"tau={s.tau}, decay_rank={s.decay_rank}: both are positive")
+        self.qk, self.vv = s.n_heads * s.head_dim, s.n_heads * s.value_dim
+
+    def cache_spec(self):
+        s = self.spec
+        return CacheSpec(state=StateSpec(parts=(("matrix", (s.n_heads, s.head_dim, s.value_dim)),)))    # S, row by row
+
+    def tensor_decls(self):
+        s, p = self.spec, self.spec.prefix
+        return [
+            TensorDecl(p + "q", (self.qk, s.hidden)), TensorDecl(p + "k", (self.qk, s.hidden)),
+            TensorDecl(p + "v", (self.vv, s.hidden)), TensorDecl(p + "g", (self.vv, s.hidden)),
+            TensorDecl(p + "o", (s.hidden, self.vv)), TensorDecl(p + "norm", (s.value_dim,), init="ones"),
+            TensorDecl(p + "a1", (s.decay_rank, s.hidden)), TensorDecl(p + "a2", (self.qk, s.decay_rank)),
+            TensorDecl(p + "a2.b", (self.qk,)),
+        ]
+
+    def load(self, src, rt):
+        super().load(src, rt)
+        s, p = self.spec, self.spec.prefix
+        ws = [src.get(p + n) for n in ("q", "k", "v", "g", "a1")]
+        rows = sum(w.shape[0] for w in ws)
+        if rows % 8:     # (rows of zeros keep the product's output rows a multiple of 32 bytes wide)
+            ws.append(torch.zeros(8 - rows % 8, s.hidden, dtype=ws[0].dtype, device=ws[0].device))
+        self.w_in = _cat_rows(ws)
+        self.w_a2, self.b_a2 = src.get(p + "a2"), src.get(p + "a2.b")
+        self.norm_w = src.get(p + "norm")
+        self.w_o = src.get(p + "o")
+
+    def forward_into(self, x, out, batch, cache, accumulate=False):
+        s, rt = self.spec, self.rt
+        T, H, D, V = x.shape[0], s.n_heads, s.head_dim, s.value_dim
+        f32 = torch.float32
+        proj = rt.empty(T, self.w_in.shape[0], dtype=f32)
+        ops.linear(x, self.w_in, proj, status=batch.status, stream=batch.stream)
+        q, k, v = proj[:, :self.qk], proj[:, self.qk:2 * self.qk], proj[:, 2 * self.qk:2 * self.qk + self.vv]
+        at = 2 * self.qk + self.vv
+        gate, low = proj[:, at:at + self.vv], proj[:, at + self.vv:at + self.vv + s.decay_rank]
+        alpha = rt.empty(T, self.qk, dtype=f32)
+        ops.channel_decay_prep(low, self.w_a2, self.b_a2, s.tau, alpha, stream=batch.stream)
+        read = rt.empty(T, self.vv, dtype=f32)
+        ops.channel_decay_scan(q, k, v, alpha, float(D) ** -0.5, cache.states["matrix"], read, batch.token_seq,
+                               batch.seq_slot, batch.n_seqs, H, D, V, stream=batch.stream)
+        y = rt.empty(T, self.vv)
+        ops.gated_group_norm(read, gate, self.norm_w, s.norm_eps, "silu", y, H, V, stream=batch.stream)
+        ops.linear(y, self.w_o, out, accumulate=accumulate, status=batch.status, stream=batch.stream)
+
+
+register_part("gated_linear_attention", GatedLinearAttention, replace=True)
 register_part("mlstm", Mlstm, replace=True)
 register_part("gated_delta_rule", GatedDeltaRule, replace=True)
 register_part("general_delta_rule", GeneralDeltaRule, replace=True)

@@ -25,6 +25,8 @@ class DecoderModel(Part):
         self.embedding_norm = build_part(spec.embedding_norm) if spec.embedding_norm is not None else None
         if self.embedding_norm is not None and not hasattr(self.embedding_norm, "forward_in_place"):
             raise ValueError("the embedding's norm must be able to norm the 32-bit stream in place")
+        if int(getattr(spec, "streams", 1)) > 1 and (self.embedding_norm is not None or spec.position_table):
+            raise ValueError("a residual of several streams starts from plain embedding rows")
         for e in spec.schedule:
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule names layer {e.layer}, the model has {len(self.layers)}")
@@ -102,11 +104,15 @@ class DecoderModel(Part):
     def forward(self, batch, caches) -> torch.Tensor:
         """``caches(entry) -> LayerCache``.  Returns [len(want_rows), vocab] float32."""
         s, rt = self.spec, self.rt
-        h = rt.empty(batch.n_tokens, s.hidden, dtype=torch.float32)
+        streams = int(getattr(s, "streams", 1))
+        h = rt.empty(batch.n_tokens, streams * s.hidden, dtype=torch.float32)    # (a token's streams side by side)
         with ops.trace_scope("embedding"):
             rms = self.embedding_norm.as_rms() if self.embedding_norm is not None else None
             fused = rms is not None and self.position_table is None and getattr(s, "embedding_scale", 1.0) == 1.0
-            if fused:
+            if streams > 1:
+                ops.embed_streams(self.embedding, batch.token_ids, h, streams, status=batch.status, stream=batch.stream,
+                                  scale=float(s.embedding_scale))
+            elif fused:
                 # rows looked up and RMS-normed in one kernel
                 ops.embed_norm(self.embedding, batch.token_ids, rms[0], rms[1], h, status=batch.status, stream=batch.stream)
             elif self.position_table is not None:

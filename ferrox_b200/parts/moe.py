@@ -58,6 +58,7 @@ class SoftmaxTopkMoe(FeedForward):
     graph_safe = True
     fuses_norm = True
     fuses_post_norm = True
+    gives_rows = True
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -222,7 +223,7 @@ class SoftmaxTopkMoe(FeedForward):
 
     def forward_add(self, x, h, batch, then_norm=None):
         st = batch.stream
-        y, inv_perm, weights, shared, gate_logit = self._expert_rows(x, batch)
+        y, inv_perm, weights, shared, gate_logit = self.expert_rows(x, batch)
         K = self.spec.top_k
         # the combination applies the norm that follows it where that is an RMSNorm over rows it can hold
         rms = then_norm.as_rms() if then_norm is not None else None
@@ -236,13 +237,13 @@ class SoftmaxTopkMoe(FeedForward):
     def forward_post(self, x, h, batch, post, then_norm=None):
         """h += post(ffn(x)): one kernel adds a token's expert rows up, norms the sum, adds it to the stream and applies
         the norm that follows to the new row."""
-        y, inv_perm, weights, shared, gate_logit = self._expert_rows(x, batch)
+        y, inv_perm, weights, shared, gate_logit = self.expert_rows(x, batch)
         (w, eps), nxt = post.as_rms(), then_norm.as_rms() if then_norm is not None else None
         then = (nxt[0], nxt[1], self.rt.empty(h.shape[0], h.shape[1])) if nxt is not None else None
         return ops.rmsnorm_residual(h, y, w, eps, then=then, expert_rows=(inv_perm, weights, shared, gate_logit),
                                     stream=batch.stream)
 
-    def _expert_rows(self, x, batch):
+    def expert_rows(self, x, batch):
         """The experts' results: (rows in expert order [T * K, H], each (token, rank) pair's row, the weights they are
         added up with (None: as they are), the shared expert's rows or None, its gate's logits or None)."""
         s, rt, st = self.spec, self.rt, batch.stream

@@ -12,16 +12,20 @@ from .base import Norm, register_part
 class RmsNorm(Norm):
     """``one_plus``: the stored weight lies around zero and the norm multiplies by 1 + w (added once, in 32 bits,
     when the weights are loaded).  ``scale_name``: the result is multiplied by one more vector; both factors are one
-    32-bit weight from the loading on."""
+    32-bit weight from the loading on.  ``scalar``: the stored weight is one number, spread over the row when it is
+    loaded, so that every kernel finds a vector."""
 
     graph_safe = True
 
     def _name(self):
         return getattr(self.spec, "name", None) or self.spec.prefix + "weight"
 
+    def _scalar(self):
+        return bool(getattr(self.spec, "scalar", False))
+
     def tensor_decls(self):
         one_plus = getattr(self.spec, "one_plus", False)
-        d = [TensorDecl(self._name(), (self.spec.size,), init="normal" if one_plus else "ones")]
+        d = [TensorDecl(self._name(), () if self._scalar() else (self.spec.size,), init="normal" if one_plus else "ones")]
         if getattr(self.spec, "scale_name", None):
             d.append(TensorDecl(self.spec.scale_name, (self.spec.size,), init="ones"))
         return d
@@ -29,6 +33,8 @@ class RmsNorm(Norm):
     def load(self, src, rt):
         super().load(src, rt)
         self.weight = src.get(self._name())
+        if self._scalar():
+            self.weight = self.weight.to(torch.float32).reshape(1).expand(self.spec.size).contiguous()
         if getattr(self.spec, "one_plus", False):
             self.weight = (1.0 + self.weight.to(torch.float32)).contiguous()
         if getattr(self.spec, "scale_name", None):

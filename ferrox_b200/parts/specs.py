@@ -29,6 +29,18 @@ class NormSpec:
     # the full name of a further [size] vector the norm's result is multiplied by, element by element (a layer scale
     # behind an output norm)
     scale_name: Optional[str] = None
+    scalar: bool = False  # the stored weight is a single number (shape []), the same for all coordinates
+
+
+@dataclass(frozen=True)
+class StreamNormSpec:
+    """What a sublayer reads of a residual of several streams: norm(sum_s in[s] x_s).  ``norm``: the spec of an RMS norm
+    over one stream's width; ``in_name``: the full name of the [streams] tensor in (None: the plain sum)."""
+
+    norm: NormSpec
+    streams: int
+    in_name: Optional[str] = None
+    kind: str = "stream_norm"
 
 
 @dataclass(frozen=True)
@@ -122,6 +134,13 @@ class AttentionSpec:
     # name (after <prefix>) of a [n_heads] vector: exp(sink_h) joins the softmax's denominator
     sink: Optional[str] = None
     value_mix: Optional["ValueMixSpec"] = None  # the values take part in the mixing of values across layers
+    # queries and keys are divided by their root mean square per head BEHIND the rotation, without a weight, with this eps
+    rotated_norm_eps: Optional[float] = None
+    # (base, pairing): the value of position j is turned by j over the whole value head, pair m at base^(-2m / value_dim),
+    # before it is cached, and a head's result at position i is turned back by i, before the gate; pairing "halves"
+    # (m, m + value_dim/2) or "adjacent" (2m, 2m + 1)
+    value_turn: Optional[Tuple[float, str]] = None
+    o_bias: bool = False  # the output projection has a bias (tensor_names key o_bias)
 
 
 @dataclass(frozen=True)
@@ -239,6 +258,39 @@ class GeneralDeltaSpec:
     norm_eps: float
     prefix: str
     kind: str = "general_delta_rule"
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """Linear attention with a decay per key channel that depends on the token: S = diag(alpha) S + k v^T, o = S^T q,
+    alpha = sigmoid(a2 a1 x + a2.b)^(1/tau), q scaled by head_dim^(-1/2); each head's o is RMS-normed with one weight
+    [value_dim] and gated by SiLU(g x).  Tensors <prefix>{q,k,v,g,o,norm}, a1 [decay_rank, hidden],
+    a2 [H*D, decay_rank], a2.b."""
+
+    hidden: int
+    n_heads: int
+    head_dim: int
+    value_dim: int
+    decay_rank: int
+    tau: float
+    norm_eps: float
+    prefix: str
+    kind: str = "gated_linear_attention"
+
+
+@dataclass(frozen=True)
+class SelectiveScanSpec:
+    """A Mamba mixer: [x | z] = in h; x = SiLU(conv x + conv.b); [dt | B | C] = x x; dt = softplus(dt dt + dt.b);
+    S[c, n] = exp(-dt_c e^(A_log[c, n])) S + dt_c x_c B_n; y_c = sum_n S C_n + D_c x_c; o (y SiLU(z)).
+    Tensors <prefix>{in,conv,conv.b,x,dt,dt.b,A_log,D,o}."""
+
+    hidden: int
+    inner: int
+    n_state: int
+    dt_rank: int
+    conv_taps: int
+    prefix: str
+    kind: str = "selective_scan"
 
 
 @dataclass(frozen=True)
@@ -379,6 +431,23 @@ class SandwichBlockSpec:
 
 
 @dataclass(frozen=True)
+class HyperBlockSpec:
+    """A layer on a residual of several streams x_1 .. x_s (hyper-connections).  For each sublayer q (1: mixer,
+    2: feed-forward): u = sum_s in[s] x_s, y = sublayer(norm(u)), x_t <- sum_s mix[s, t] x_s + out[t] y.
+    ``norm1`` and ``norm2``: StreamNormSpec; ``connections``: per sublayer the full names of its (mix [s, s], out [s])
+    tensors.  ``ffn`` None: the layer ends after the mixer."""
+
+    norm1: StreamNormSpec
+    mixer: object
+    norm2: Optional[StreamNormSpec]
+    ffn: Optional[object]
+    streams: int
+    connections: Tuple[Tuple[str, str], ...]
+    kind: str = "hyper_connections"
+    unused_tensors: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()  # (name, shape) a checkpoint may carry all the same
+
+
+@dataclass(frozen=True)
 class ScheduleEntry:
     """One call in the order of execution: run ``layer`` against cache ``cache``.
 
@@ -408,6 +477,9 @@ class ModelSpec:
     position_table: Optional[str] = None  # a learned [max_positions, hidden] table: row p is added to position p's embedding
     logit_softcap: Optional[float] = None  # c: the logits pass through c * tanh(z / c)
     embedding_scale: float = 1.0  # the embedding rows are multiplied by this
+    # residual streams: every token carries that many rows of ``hidden``, side by side, all equal to its embedding row at
+    # the start; blocks and the final norm are of the kinds that know streams
+    streams: int = 1
 
     @property
     def n_caches(self) -> int:

@@ -31,10 +31,11 @@ class WeightsError(ValueError):
 class TensorDecl:
     name: str
     shape: Tuple[int, ...]
-    init: str = "normal"  # how the random-weights mode fills it: normal | ones | zeros
+    init: str = "normal"  # how the random-weights mode fills it: normal | ones | zeros | identity (a square matrix)
     optional: bool = False  # present or absent by the file's choice (e.g. a gate vector)
     integer: bool = False  # an integer table (kept as int32)
     below: int = 0  # the integers of a row (last dimension) are distinct, from 0 on and below this (random-weights mode)
+    mean: float = 0.0  # what the random-weights mode's normal values lie around (init normal)
 
 
 def resident_dtype(stored: torch.dtype, compute: torch.dtype) -> torch.dtype:

@@ -9,7 +9,8 @@ that :func:`normal_cpu` here and ``fx_random_normal`` (csrc/random_init.cu) give
 on which other tensors exist, on the order in which they are made or on where they are drawn.  A model of any size can
 therefore be drawn on the device for the engine and handed, copied to the host, to a plain implementation.
 
-Matrices, biases and gate vectors are N(0, std); norm weights are 1 (``norm_init="ones"``), 1 + N(0, std)
+Matrices, biases and gate vectors are N(0, std), around a part's own mean where it states one (constants that only make
+sense around a value: the identity for matrices that mix residual streams); norm weights are 1 (``norm_init="ones"``), 1 + N(0, std)
 (``"around_one"``) or N(0, std) like everything else (``"normal"``).  The reference's counterpart is
 ``Decoder::new_random_small`` (crates/ferrox-models/src/decoder.rs:373-388,397-514: one xorshift64* stream from seed
 42 for every tensor, uniform +-0.05, norm weights 1, no bias, no shared gate); unlike it, this mode fills biases and
@@ -159,7 +160,12 @@ def random_tensor(decl: TensorDecl, seed: int, dtype, std: float, norm_init: str
         mean = 1.0
     elif decl.init == "ones" and norm_init != "normal":
         raise ValueError(f"norm_init={norm_init!r}: expected ones, around_one or normal")
-    return normal(tensor_key(seed, decl.name), decl.shape, dtype, mean, std, device)
+    if decl.init == "normal":
+        mean = decl.mean
+    t = normal(tensor_key(seed, decl.name), decl.shape, dtype, mean, std, device)
+    if decl.init == "identity":
+        t += torch.eye(decl.shape[0], dtype=dtype, device=t.device)
+    return t
 
 
 def random_tensors(
