@@ -6,6 +6,7 @@
     python bench.py --designs bobepel   (the Bobepel design beside the Qwen2-MoE decoder at equal sizes)
     python bench.py --designs zanezen   (the Zanezen design beside Bobepel at equal sizes)
     python bench.py --designs balelorn   (the Balelorn design beside the Qwen2-MoE decoder at equal sizes)
+    python bench.py --designs dubazen    (the Dubazen design beside the Qwen2-MoE decoder at equal sizes)
 
 Default workload: the layer sizes of the Qwen1.5-MoE-A2.7B shape (24 layers, hidden
 2048, 16 heads of 128, 60 experts top-4 of width 1408, shared expert 5632, vocab
@@ -279,6 +280,28 @@ def balelorn_shape(width, layers, vocab=32768, chunk=1024):
             "layers": [att] * layers}
 
 
+def dubazen_shape(width, layers, vocab=32768):
+    """Layer sizes that resemble a real model's: selective state spaces of twice the width with 16 states a channel and a
+    step size of inner width width / 16 (four taps); attention with heads of 128 on a quarter as many key heads, half of
+    each head rotated, beside lightning attention with as many heads of 128 x 128; linear attention with heads of 128 x
+    128 and a decay of inner width 16; in turn selective, parallel, linear, selective.  Four residual streams; experts as
+    in the Qwen2-MoE shape: 60 of which a token uses 4, a shared expert four times as wide."""
+    h = width // 128
+    ff = width * 11 // 16 // 64 * 64
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": 60, "top": 4},
+           "shared": {"ff": 4 * ff, "limit": 7.0}}
+    mamba = {"type": "mamba1", "mlp": mlp, "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                 "rot": {"dims": 64, "base": 1000000.0}},
+        "right": {"heads": h, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(3 + 8 * i / max(1, h - 1)) for i in range(h)]},
+        "left_scale": 1.0, "right_scale": 1.0}}
+    gla = {"type": "gla", "mlp": mlp, "mixer": {"heads": h, "dim": 128, "vdim": 128, "tau": 16.0}}
+    return {"architecture": "Dubazen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 4,
+            "embedding": {"scale": float(width) ** 0.5}, "max_positions": CONTEXT,
+            "layers": [(mamba, par, gla, mamba)[i % 4] for i in range(layers)]}
+
+
 def compare_designs(args) -> int:
     """Prefill and decode throughput of a design and of the closest existing decoder at a few equal sizes (random
     bfloat16 weights), with the device time of every class of kernel from a traced pass beside them."""
@@ -416,6 +439,15 @@ def compare_designs(args) -> int:
                           "batch": batch, "prompt_tokens": PREFILL_TOKENS, "decode_steps_timed": steps, "peaks": pk,
                           "data": "synthetic: random N(0,0.02) weights, uniform random token ids", "sizes": rows}))
         return 0
+    if args.designs == "dubazen":
+        for width, layers, _ in sizes:
+            a, b = dubazen_shape(width, layers), moe_like(width, layers)
+            rows.append({"width": width, "layers": layers, "expert_ff": b["moe_intermediate_size"],
+                         "dubazen": measure(a), "qwen2_moe": measure(b)})
+        print(json.dumps({"designs": "Dubazen beside the Qwen2-MoE decoder at equal size", "dtype": "bf16",
+                          "batch": batch, "prompt_tokens": PREFILL_TOKENS, "decode_steps_timed": steps, "peaks": pk,
+                          "data": "synthetic: random N(0,0.02) weights, uniform random token ids", "sizes": rows}))
+        return 0
     if args.designs == "bobepel":
         for width, layers, _ in sizes:
             a, b = bobepel_shape(width, layers), moe_like(width, layers)
@@ -448,12 +480,12 @@ def main() -> int:
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--page-size", type=int, default=64)
     ap.add_argument("--repeats", type=int, default=3, help="timed regions of --steps steps each; the median counts")
-    ap.add_argument("--designs", nargs="?", const="safepel", default=None, choices=["safepel", "bobepel", "sesuzen", "sesuzen-moe", "zanezen", "balelorn"],
+    ap.add_argument("--designs", nargs="?", const="safepel", default=None, choices=["safepel", "bobepel", "sesuzen", "sesuzen-moe", "zanezen", "balelorn", "dubazen"],
                     help="instead of the default workload: prefill and decode of a design beside the closest existing "
                          "decoder at a few equal sizes, with device time per class of kernel (safepel: beside the dense "
                          "Qwen2 decoder; bobepel: beside the Qwen2-MoE decoder; sesuzen: dense feed-forwards, beside "
                          "Safepel; sesuzen-moe: experts, beside the Qwen2-MoE decoder without its shared expert; zanezen: beside Bobepel; balelorn: beside the Qwen2-MoE decoder without its "
-                         "shared expert)")
+                         "shared expert; dubazen: beside the Qwen2-MoE decoder)")
     ap.add_argument("--widths", default="", help="--designs: only these widths (commas), e.g. 2048")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -342,8 +342,8 @@ int fx_channel_decay_scan(const float* q, long ldq, const float* k, long ldk, co
                           float q_scale, float* state, float* out, long ldo, const int* token_seq, const int* seq_slot,
                           int n_tokens, int n_entries, int H, int D, int V, void* stream);
 
-// Selective state space (selective_scan.cu): dt = softplus(dt + dt_bias), S[c, n] <- exp(dt A) S + dt x B_n,
-// out = (sum_n S C_n + D x) silu(z), A = -exp(A_log); state [slots, inner, n_state] 32-bit.
+// Selective state space (selective_scan.cu): per channel step = softplus(dt + dt_bias), the state row
+// s = e^(-step e^A_log) * s + step x B, out = (s . C + D x) silu(z); state [slots, inner, n_state] 32-bit.
 int fx_selective_scan(const float* dt, long ldt, const void* dt_bias, int db_dtype, const void* x, long ldx, const void* z,
                       long ldz, int dtype, const float* bc, long ldbc, const float* a_log, const float* d_skip,
                       float* state, void* out, long ldo, const int* token_seq, const int* seq_slot, int n_tokens,

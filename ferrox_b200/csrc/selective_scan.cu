@@ -1,7 +1,7 @@
 // The selective state space of a Mamba mixer: per request a state S [inner, n_state], 32-bit, and for every token
 //
-//   dt_c = softplus(dt_c + bias_c),    S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,    A = -exp(A_log)
-//   y_c  = sum_n S[c, n] C_n + D_c x_c,    out_c = y_c silu(z_c)
+//   a channel's row s of it:   step = softplus(dt + bias),   s = e^(-step e^A_log) * s + step x B,   y = s . C + D x
+//   out = y silu(z)                                          (B and C: one number a state, shared by the channels)
 //
 // Channels never meet: L lanes share a channel's states (NPL of them each, in runs of four, so that B and C are read
 // from shared memory sixteen bytes at a time) and keep them in registers for the whole step; the tokens of a request are

@@ -1,9 +1,9 @@
 """The selective state space of a Mamba mixer.
 
     [x | z] = Win h;   x = silu(conv(x) + b)                      (causal, per channel; its last inputs are state)
-    [dt | B | C] = Wx x;   dt = softplus(Wdt dt + bdt)            (one step size a channel)
-    S[c, n] <- exp(-dt_c e^(A_log[c, n])) S[c, n] + dt_c x_c B_n
-    y_c = sum_n S[c, n] C_n + D_c x_c;   out = Wo (y silu(z))
+    [low | B | C] = Wx x;   step = softplus(Wdt low + bdt)        (one step size a channel)
+    a channel's state row s:   s = e^(-step e^A_log) * s + step x B;   y = s . C + D x
+    out = Wo (y * silu(z))
 
 The state [inner, n_state] lives in the cache manager's slots, 32-bit, and so do the convolution's last inputs.  The
 projections run in the engine's dtype with 32-bit results where they feed the recurrence.  The inner width of dt is small

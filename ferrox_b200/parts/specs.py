@@ -29,7 +29,7 @@ class NormSpec:
     # the full name of a further [size] vector the norm's result is multiplied by, element by element (a layer scale
     # behind an output norm)
     scale_name: Optional[str] = None
-    scalar: bool = False  # the stored weight is a single number (shape []), the same for all coordinates
+    scalar: bool = False  # the stored weight has shape []: it weighs every element of the row
 
 
 @dataclass(frozen=True)
@@ -281,7 +281,7 @@ class GatedLinearAttentionSpec:
 @dataclass(frozen=True)
 class SelectiveScanSpec:
     """A Mamba mixer: [x | z] = in h; x = SiLU(conv x + conv.b); [dt | B | C] = x x; dt = softplus(dt dt + dt.b);
-    S[c, n] = exp(-dt_c e^(A_log[c, n])) S + dt_c x_c B_n; y_c = sum_n S C_n + D_c x_c; o (y SiLU(z)).
+    per channel a state row s: s = e^(-dt e^A_log) * s + dt x B, y = s . C + D x; o (y * SiLU(z)).
     Tensors <prefix>{in,conv,conv.b,x,dt,dt.b,A_log,D,o}."""
 
     hidden: int
@@ -432,8 +432,8 @@ class SandwichBlockSpec:
 
 @dataclass(frozen=True)
 class HyperBlockSpec:
-    """A layer on a residual of several streams x_1 .. x_s (hyper-connections).  For each sublayer q (1: mixer,
-    2: feed-forward): u = sum_s in[s] x_s, y = sublayer(norm(u)), x_t <- sum_s mix[s, t] x_s + out[t] y.
+    """A layer on a residual of several streams, the rows of R (hyper-connections).  Each sublayer f of the layer (the
+    mixer, then the feed-forward) makes y = f(norm(in^T R)) and leaves R <- mix^T R + out y^T.
     ``norm1`` and ``norm2``: StreamNormSpec; ``connections``: per sublayer the full names of its (mix [s, s], out [s])
     tensors.  ``ffn`` None: the layer ends after the mixer."""
 

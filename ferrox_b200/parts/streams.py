@@ -1,16 +1,17 @@
 """A residual of several streams (hyper-connections): the norm that reads it and the block that writes it.
 
-A token carries s rows x_1 .. x_s.  For each sublayer q of a layer (1: mixer, 2: feed-forward), with constants of the
-layer's own,
+A token carries a small matrix R whose rows are its streams.  The mixer (1) and the feed-forward (2) of a layer, each with
+constants of its own,
 
-    u = sum_s in_q[s] x_s;   y_q = sublayer_q(norm_q(u));   x_t <- sum_s mix_q[s, t] x_s + out_q[t] y_q
+    y_q = f_q(norm_q(in_q^T R));   R <- mix_q^T R + out_q y_q^T
 
-The constants are weights and do not depend on the token, so two updates in a row are one: with M = mix_1 mix_2,
+The constants are weights and do not depend on the token, so the layer's two updates are one,
 
-    x_t <- sum_s M[s, t] x_s + (out_1 mix_2)[t] y_1 + out_2[t] y_2
-    u_2  = sum_s (mix_1 in_2)[s] x_s + (in_2 . out_1) y_1
+    R <- (mix_1 mix_2)^T R + (mix_2^T out_1) y_1^T + out_2 y_2^T
 
-and a layer passes over the streams twice (once reading, once reading and writing) instead of reading and writing them
+and what the feed-forward reads can be had from the layer's old R: (mix_1 in_2)^T R + (in_2 . out_1) y_1^T,
+
+so that a layer passes over the streams twice (once reading, once reading and writing) instead of reading and writing them
 for every sublayer.  Both passes are one kernel (``ops.stream_step``), which also adds a token's expert rows up, applies
 the weights of a mixer made of mixers and norms what the next sublayer reads.  The products of constants are worked out
 in 64 bits when the weights are loaded and rounded once to 32.
@@ -29,7 +30,7 @@ def _floats(t: torch.Tensor) -> list:
 
 
 class StreamNorm(Norm):
-    """norm(sum_s in[s] x_s) of rows [T, streams * size]; ``in_name`` None: the plain sum."""
+    """norm(in^T R) of rows [T, streams * size]; ``in_name`` None: the plain sum."""
 
     graph_safe = True
 

@@ -36,7 +36,6 @@ def rms(x, eps):
 
 
 def scalar_rms_norm(x, g, eps):
-    """One number g for all coordinates."""
     return rms(x, eps) * g.reshape(())
 
 
@@ -147,7 +146,7 @@ def gated_linear_attention(h, W, p, m, eps):
 
 
 def selective_scan(h, W, p, m, eps):
-    """S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n; y_c = sum_n S[c, n] C_n + D_c x_c; y * silu(z)."""
+    """A channel's state row decays by e^(-step e^A_log), gains step x B and is read by C; D x beside it, a gate behind."""
     n, I, N, R = h.shape[0], m["inner"], m["state"], m["dt_rank"]
     xz = _r(h @ W[p + "in"].T)
     x, z = xz[:, :I], xz[:, I:]
