@@ -341,6 +341,11 @@ int fx_channel_decay_prep(const float* low, long ldl, const void* w2, int w2_dty
 int fx_channel_decay_scan(const float* q, long ldq, const float* k, long ldk, const float* v, long ldv, const float* alpha,
                           float q_scale, float* state, float* out, long ldo, const int* token_seq, const int* seq_slot,
                           int n_tokens, int n_entries, int H, int D, int V, void* stream);
+// The same for one fixed decay a head, state [slots, H, V, D] (as fx_state_scan's); q, k, v behind their activation.
+int fx_fixed_decay_scan(const float* q, long ldq, const float* k, long ldk, const float* v, long ldv, const float* decay,
+                        float* state, float* out, long ldo, const int* token_seq, const int* seq_slot, int n_tokens,
+                        int n_entries, int H, int D, int V, void* stream);
+int fx_silu_rows(const void* x, int dtype, long ldx, float* out, long ldo, int n_rows, int n, void* stream);   // 32-bit SiLU
 
 // Selective state space (selective_scan.cu): per channel step = softplus(dt + dt_bias), the state row
 // s = e^(-step e^A_log) * s + step x B, out = (s . C + D x) silu(z); state [slots, inner, n_state] 32-bit.

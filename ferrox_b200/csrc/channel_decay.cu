@@ -13,6 +13,9 @@
 // tokens' rows travel into shared memory CD_CH tokens at a time by cp.async, the next chunk while this one is worked on;
 // the groups' shares of the read-outs are added up once a chunk.  The order of additions does not depend on how a
 // request was cut into steps.  State [slots, H, D, V]: a row's columns lie together.
+//
+// fx_fixed_decay_scan: the same loop for one fixed decay a head, S <- d S + k v^T (the recurrence of fx_state_scan without
+// its delta rule, over a state laid out as there, column by column), for long prompts.
 #include "common.cuh"
 #include "api.h"
 
@@ -96,20 +99,22 @@ struct CdArgs {
     long ld[3];
     const float* v; long ldv;
     float q_scale;
-    float* state;          // [slots, H, D, V]
+    const float* decay;    // one fixed decay a head (no alpha rows then)
+    float* state;          // [slots, H][D, V], row i, column j of a head at i * row_stride + j * col_stride
+    long row_stride, col_stride;
     float* out; long ldo;  // [T, H * V]
     const int *token_seq, *seq_slot;
     int n_tokens, H, D, V;
     int vec;               // q, k, alpha rows may be copied 16 bytes at a time
 };
 
-// Shared memory: two buffers of [3][CD_CH][DP] rows and [CD_CH][CD_COLS] values, then [CD_CH][CD_GROUPS][CD_COLS]
+// Shared memory: two buffers of [3][CD_CH][DP] rows (FIXED: [2]) and [CD_CH][CD_COLS] values, then [CD_CH][CD_GROUPS][CD_COLS]
 // read-out shares; DP = RPL * CD_GROUPS.
-template <int RPL>
+template <int RPL, bool FIXED>
 __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const CdArgs a)
 {
-    constexpr int DP = RPL * CD_GROUPS;
-    constexpr int BUF = CD_CH * (3 * DP + CD_COLS);
+    constexpr int DP = RPL * CD_GROUPS, ROWS = FIXED ? 2 : 3;
+    constexpr int BUF = CD_CH * (ROWS * DP + CD_COLS);
     extern __shared__ __align__(16) float sm[];
     fx_pdl_wait_only();
     const int b = blockIdx.x, h = blockIdx.y, D = a.D;
@@ -120,13 +125,14 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
     float* rd_s = sm + 2 * BUF;
     const uint32_t sm_u = (uint32_t)__cvta_generic_to_shared(sm);
     const bool live = col < nc;
-    float* sp = a.state + (((long)a.seq_slot[b] * a.H + h) * D) * a.V + col0 + (live ? col : 0);
+    float* sp = a.state + ((long)a.seq_slot[b] * a.H + h) * D * a.V + (long)(col0 + (live ? col : 0)) * a.col_stride;
+    const float fixed = FIXED ? a.decay[h] : 0.f;
 
     float S[RPL];
 #pragma unroll
     for (int i = 0; i < RPL; ++i) {
         const int row = grp * RPL + i;
-        S[i] = (live && row < D) ? sp[(long)row * a.V] : 0.f;
+        S[i] = (live && row < D) ? sp[row * a.row_stride] : 0.f;
     }
     // what lies beyond the head's D rows and the live columns stays zero in both buffers
     for (int idx = threadIdx.x; idx < 2 * BUF; idx += CD_THREADS) sm[idx] = 0.f;
@@ -137,16 +143,16 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
     const int pw = a.vec ? D >> 2 : D;                   // pieces a row: 16 bytes each, or one element
     const int p_tt0 = threadIdx.x / pw, p_i0 = threadIdx.x - p_tt0 * pw;
     const int p_dq = CD_THREADS / pw, p_dr = CD_THREADS - p_dq * pw;
-    const float* srcp[3];
+    const float* srcp[ROWS];
 #pragma unroll
-    for (int arr = 0; arr < 3; ++arr) srcp[arr] = a.src[arr] + (long)h * D;
+    for (int arr = 0; arr < ROWS; ++arr) srcp[arr] = a.src[arr] + (long)h * D;
     const float* vp = a.v + (long)h * a.V + col0;
     auto issue = [&](int c0, int nt, int buf) {
         const uint32_t base = sm_u + (uint32_t)(buf * BUF) * 4u;
         for (int tt = p_tt0, i = p_i0; tt < nt;) {
             const int e = a.vec ? i * 4 : i;
 #pragma unroll
-            for (int arr = 0; arr < 3; ++arr) {
+            for (int arr = 0; arr < ROWS; ++arr) {
                 const uint32_t dst = base + (uint32_t)((arr * CD_CH + tt) * DP + e) * 4u;
                 const float* src = srcp[arr] + (long)(c0 + tt) * a.ld[arr] + e;
                 if (a.vec) cp_async16(dst, src); else cp_async4(dst, src);
@@ -155,7 +161,7 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
             if (i >= pw) { i -= pw; ++tt; }
         }
         const int tt = threadIdx.x / CD_COLS;            // (CD_CH * CD_COLS values: one a thread)
-        if (tt < nt && live) cp_async4(base + (uint32_t)(3 * CD_CH * DP + threadIdx.x) * 4u, vp + (long)(c0 + tt) * a.ldv + col);
+        if (tt < nt && live) cp_async4(base + (uint32_t)(ROWS * CD_CH * DP + threadIdx.x) * 4u, vp + (long)(c0 + tt) * a.ldv + col);
     };
 
     issue(r0, min(CD_CH, r1 - r0), 0);
@@ -174,14 +180,14 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
         const float* q_s = sm + buf * BUF + grp * RPL;
         const float* k_s = q_s + CD_CH * DP;
         const float* w_s = k_s + CD_CH * DP;
-        const float* v_s = sm + buf * BUF + 3 * CD_CH * DP + col;
+        const float* v_s = sm + buf * BUF + ROWS * CD_CH * DP + col;
 #pragma unroll 4
         for (int tt = 0; tt < nt; ++tt) {
             const float vt = v_s[tt * CD_COLS];
             float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
             for (int i = 0; i < RPL; i += 4) {
-                const float4 ww = *reinterpret_cast<const float4*>(w_s + tt * DP + i);
+                const float4 ww = FIXED ? make_float4(fixed, fixed, fixed, fixed) : *reinterpret_cast<const float4*>(w_s + tt * DP + i);
                 const float4 kk = *reinterpret_cast<const float4*>(k_s + tt * DP + i);
                 const float4 qq = *reinterpret_cast<const float4*>(q_s + tt * DP + i);
                 S[i] = fmaf(ww.x, S[i], kk.x * vt); S[i + 1] = fmaf(ww.y, S[i + 1], kk.y * vt);
@@ -208,18 +214,18 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
 #pragma unroll
         for (int i = 0; i < RPL; ++i) {
             const int row = grp * RPL + i;
-            if (row < D) sp[(long)row * a.V] = S[i];
+            if (row < D) sp[row * a.row_stride] = S[i];
         }
     }
 }
 static_assert(CD_CH == CD_GROUPS, "a chunk's read-outs are added up by one group of threads a token");
 
-template <int RPL>
+template <int RPL, bool FIXED>
 int launch_cd(const CdArgs& a, int n_entries, cudaStream_t s)
 {
     constexpr int DP = RPL * CD_GROUPS;
-    const size_t smem = ((size_t)2 * CD_CH * (3 * DP + CD_COLS) + CD_CH * CD_THREADS) * sizeof(float);
-    auto kern = channel_decay_scan_kernel<RPL>;
+    const size_t smem = ((size_t)2 * CD_CH * ((FIXED ? 2 : 3) * DP + CD_COLS) + CD_CH * CD_THREADS) * sizeof(float);
+    auto kern = channel_decay_scan_kernel<RPL, FIXED>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
@@ -228,6 +234,27 @@ int launch_cd(const CdArgs& a, int n_entries, cudaStream_t s)
     // a prompt's recurrence starts on an empty device (see fx_launch_pdl_if); a decode step's is set up early
     fx_launch_pdl_if(a.n_tokens < 8 * n_entries, kern, grid, dim3(CD_THREADS), smem, s, a);
     return fx_launch_status();
+}
+
+template <bool FIXED>
+int scan_for(const CdArgs& a, int n_entries, cudaStream_t s)
+{
+    if (a.D <= 4 * CD_GROUPS) return launch_cd<4, FIXED>(a, n_entries, s);
+    if (a.D <= 8 * CD_GROUPS) return launch_cd<8, FIXED>(a, n_entries, s);
+    if (a.D <= 12 * CD_GROUPS) return launch_cd<12, FIXED>(a, n_entries, s);
+    return launch_cd<16, FIXED>(a, n_entries, s);
+}
+
+template <typename T>
+__global__ void silu_rows_kernel(const T* __restrict__ x, long ldx, float* __restrict__ out, long ldo, int n)
+{
+    fx_pdl_wait();
+    const T* r = x + (long)blockIdx.x * ldx;
+    float* o = out + (long)blockIdx.x * ldo;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n; i += gridDim.y * blockDim.x) {
+        const float v = to_f32(r[i]);
+        o[i] = v / (1.0f + expf(-v));
+    }
 }
 
 }  // namespace
@@ -252,13 +279,38 @@ extern "C" int fx_channel_decay_scan(const float* q, long ldq, const float* k, l
     if (H <= 0 || H > 65535 || D <= 0 || V <= 0 || D > CD_MAX_D) return FX_ERR_SIZE;
     CdArgs a;
     a.src[0] = q; a.src[1] = k; a.src[2] = alpha; a.ld[0] = ldq; a.ld[1] = ldk; a.ld[2] = (long)H * D;
-    a.v = v; a.ldv = ldv; a.q_scale = q_scale; a.state = state; a.out = out; a.ldo = ldo;
+    a.v = v; a.ldv = ldv; a.q_scale = q_scale; a.decay = nullptr; a.state = state; a.row_stride = V; a.col_stride = 1;
+    a.out = out; a.ldo = ldo;
     a.token_seq = token_seq; a.seq_slot = seq_slot; a.n_tokens = n_tokens; a.H = H; a.D = D; a.V = V;
     a.vec = D % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0;
     for (int i = 0; i < 3; ++i) a.vec = a.vec && (uintptr_t)a.src[i] % 16 == 0;
+    return scan_for<false>(a, n_entries, (cudaStream_t)stream);
+}
+
+extern "C" int fx_fixed_decay_scan(const float* q, long ldq, const float* k, long ldk, const float* v, long ldv,
+                                   const float* decay, float* state, float* out, long ldo, const int* token_seq,
+                                   const int* seq_slot, int n_tokens, int n_entries, int H, int D, int V, void* stream)
+{
+    if (n_tokens <= 0 || n_entries <= 0) return FX_OK;
+    if (H <= 0 || H > 65535 || D <= 0 || V <= 0 || D > CD_MAX_D) return FX_ERR_SIZE;
+    CdArgs a;
+    a.src[0] = q; a.src[1] = k; a.src[2] = nullptr; a.ld[0] = ldq; a.ld[1] = ldk; a.ld[2] = 0;
+    a.v = v; a.ldv = ldv; a.q_scale = 1.f; a.decay = decay; a.state = state; a.row_stride = 1; a.col_stride = D;
+    a.out = out; a.ldo = ldo;
+    a.token_seq = token_seq; a.seq_slot = seq_slot; a.n_tokens = n_tokens; a.H = H; a.D = D; a.V = V;
+    a.vec = D % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0;
+    return scan_for<true>(a, n_entries, (cudaStream_t)stream);
+}
+
+extern "C" int fx_silu_rows(const void* x, int dtype, long ldx, float* out, long ldo, int n_rows, int n, void* stream)
+{
+    if (n_rows <= 0 || n <= 0) return FX_OK;
+    long by = fx_cdiv(n, 256 * 8);
+    if (by > 64) by = 64;
+    dim3 grid(n_rows, (unsigned)by);
     cudaStream_t s = (cudaStream_t)stream;
-    if (D <= 4 * CD_GROUPS) return launch_cd<4>(a, n_entries, s);
-    if (D <= 8 * CD_GROUPS) return launch_cd<8>(a, n_entries, s);
-    if (D <= 12 * CD_GROUPS) return launch_cd<12>(a, n_entries, s);
-    return launch_cd<16>(a, n_entries, s);
+    if (dtype == FX_F32) fx_launch_pdl(silu_rows_kernel<float>, grid, 256, 0, s, (const float*)x, ldx, out, ldo, n);
+    else if (dtype == FX_BF16) fx_launch_pdl(silu_rows_kernel<bf16>, grid, 256, 0, s, (const bf16*)x, ldx, out, ldo, n);
+    else return FX_ERR_DTYPE;
+    return fx_launch_status();
 }

@@ -399,6 +399,69 @@ __global__ void __launch_bounds__(128) gated_group_norm_warp_kernel(
     }
 }
 
+// The same for groups of whole 16-byte pieces: TPG threads a group (a warp, or the block), four elements each at a time,
+// the group's row in registers between the sum of its squares and the result.
+constexpr int GN_CH = 4;      // pieces a thread holds at most
+
+template <typename GT> __device__ __forceinline__ void load_gate4(const GT* p, float* g);
+template <> __device__ __forceinline__ void load_gate4<float>(const float* p, float* g) { Pack<float>::load(p, g); }
+template <> __device__ __forceinline__ void load_gate4<bf16>(const bf16* p, float* g) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    g[0] = __uint_as_float(v.x << 16); g[1] = __uint_as_float(v.x & 0xffff0000u);
+    g[2] = __uint_as_float(v.y << 16); g[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+
+template <typename GT, typename OT, int TPG>
+__global__ void __launch_bounds__(256) gated_group_norm_vec_kernel(
+    const float* __restrict__ x, const GT* __restrict__ gate, long ldg, const void* __restrict__ w, int w_dtype,
+    float eps, int act, OT* __restrict__ out, int groups, int width, long w_stride, long n_groups)
+{
+    __shared__ float scratch[33];
+    fx_pdl_wait();
+    const int own = TPG == 32 ? threadIdx.x & 31 : threadIdx.x;
+    const long at = TPG == 32 ? (long)blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;     // (token, group)
+    if (at >= n_groups) return;      // (whole warps; a block of its own group never)
+    const long t = at / groups;
+    const int grp = (int)(at - t * groups);
+    const float* xr = x + at * width;
+    const GT* gr = gate + t * ldg + (long)grp * width;
+    float v[GN_CH][4], g[GN_CH][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < GN_CH; ++c) {
+        const int i = (c * TPG + own) * 4;
+        if (i < width) { Pack<float>::load(xr + i, v[c]); load_gate4<GT>(gr + i, g[c]); }
+    }
+#pragma unroll
+    for (int c = 0; c < GN_CH; ++c)
+        if ((c * TPG + own) * 4 < width) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) ss = fmaf(v[c][e], v[c][e], ss);
+        }
+    ss = TPG == 32 ? warp_sum(ss) : block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+    OT* o = out + at * width;
+#pragma unroll
+    for (int c = 0; c < GN_CH; ++c) {
+        const int i = (c * TPG + own) * 4;
+        if (i >= width) continue;
+        float r[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float gv = g[c][e];
+            r[e] = v[c][e] * inv * load_any(w, w_dtype, (long)grp * w_stride + i + e);
+            if (sizeof(OT) == 2) r[e] *= act ? fx_sigmoid_fast(gv) : gv * fx_sigmoid_fast(gv);
+            else r[e] *= act ? sigmoid_f(gv) : silu_f(gv);
+        }
+        if (sizeof(OT) == 4) Pack<float>::store(reinterpret_cast<float*>(o) + i, r);
+        else {
+            __nv_bfloat162 p = __floats2bfloat162_rn(r[0], r[1]), q = __floats2bfloat162_rn(r[2], r[3]);
+            *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(o) + i) =
+                make_uint2(*reinterpret_cast<uint32_t*>(&p), *reinterpret_cast<uint32_t*>(&q));
+        }
+    }
+}
+
 }  // namespace
 
 extern "C" int fx_delta_prep(const void* proj, int dtype, long ldp, const void* conv_w, int cw_dtype, int taps,
@@ -484,11 +547,21 @@ extern "C" int fx_gated_group_norm(const float* x, const void* gate, int gate_dt
     if (n_tokens <= 0) return FX_OK;
     if (groups <= 0 || width <= 0) return FX_ERR_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
+    const int gb = gate_dtype == FX_F32 ? 16 : 8, ob = out_dtype == FX_F32 ? 16 : 8;     // bytes of four elements
+    const bool vec = width >= 64 && width % 4 == 0 && width <= 4 * GN_CH * 256 && ldg % 4 == 0 && (uintptr_t)x % 16 == 0 &&
+                     (uintptr_t)gate % gb == 0 && (uintptr_t)out % ob == 0;
+    const bool warp_group = width <= 4 * GN_CH * 32;
+    const long n_groups = (long)n_tokens * groups;
+    const unsigned vec_blocks = (unsigned)(warp_group ? fx_cdiv(n_groups, 8) : n_groups);
     const bool narrow = width <= 64;
     dim3 grid(n_tokens, narrow ? (unsigned)fx_cdiv(groups, 4) : groups);
 #define FX_GO(GT, OT)                                                                                                     \
     do {                                                                                                                  \
-        if (narrow) fx_launch_pdl(gated_group_norm_warp_kernel<GT, OT>, grid, 128, 0, s, x, (const GT*)gate, ldg, w, w_dtype, \
+        if (vec && warp_group) fx_launch_pdl(gated_group_norm_vec_kernel<GT, OT, 32>, vec_blocks, 256, 0, s, x, (const GT*)gate, ldg, w, \
+                                             w_dtype, eps, act, (OT*)out, groups, width, w_stride, n_groups);               \
+        else if (vec) fx_launch_pdl(gated_group_norm_vec_kernel<GT, OT, 256>, vec_blocks, 256, 0, s, x, (const GT*)gate, ldg, w,        \
+                                    w_dtype, eps, act, (OT*)out, groups, width, w_stride, n_groups);                        \
+        else if (narrow) fx_launch_pdl(gated_group_norm_warp_kernel<GT, OT>, grid, 128, 0, s, x, (const GT*)gate, ldg, w, w_dtype, \
                                   eps, act, (OT*)out, groups, width, w_stride);                                         \
         else fx_launch_pdl(gated_group_norm_kernel<GT, OT>, grid, 128, 0, s, x, (const GT*)gate, ldg, w, w_dtype, eps, act, \
                            (OT*)out, groups, width, w_stride);                                                          \

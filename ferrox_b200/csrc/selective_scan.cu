@@ -3,7 +3,7 @@
 //   a channel's row s of it:   step = softplus(dt + bias),   s = e^(-step e^A_log) * s + step x B,   y = s . C + D x
 //   out = y silu(z)                                          (B and C: one number a state, shared by the channels)
 //
-// Channels never meet: L lanes share a channel's states (NPL of them each, in runs of four, so that B and C are read
+// Channels never meet: L lanes share a channel's states (NPL of them each, in runs of up to four, so that B and C are read
 // from shared memory sixteen bytes at a time) and keep them in registers for the whole step; the tokens of a request are
 // taken in order, in the same order of operations however the request was cut into steps.  A block of 128 threads takes
 // 128 / L channels of one request; the tokens' rows come SC_CH tokens at a time, the next chunk's into registers while
@@ -18,20 +18,37 @@
 
 namespace {
 
-__device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+// log(1 + e^x) = max(x, 0) + log(1 + e) with e = e^-|x| in (0, 1]; log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3, by
+// its series 2 (s + s^3/3 + s^5/5 + ...), the first term left out below 2e-8 of the sum.
+__device__ __forceinline__ float softplus_f(float x)
+{
+    const float e = expf(-fabsf(x));
+    const float s = e / (2.0f + e), s2 = s * s;
+    float p = fmaf(s2, 1.0f / 15.0f, 1.0f / 13.0f);
+    p = fmaf(p, s2, 1.0f / 11.0f);
+    p = fmaf(p, s2, 1.0f / 9.0f);
+    p = fmaf(p, s2, 1.0f / 7.0f);
+    p = fmaf(p, s2, 1.0f / 5.0f);
+    p = fmaf(p, s2, 1.0f / 3.0f);
+    return fmaxf(x, 0.f) + 2.0f * fmaf(s * s2, p, s);
+}
+
+// z / (1 + e^-z); in 16 bits the hardware's exponential and quotient do.
+template <typename T> __device__ __forceinline__ float gate_silu(float z) {
+    return sizeof(T) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));
+}
 
 // e^a S + u for a <= 0.
 __device__ __forceinline__ float decay_add(float S, float a, float u)
 {
-    // a > -1/4: e^a - 1 = a (1 + a/2 (1 + a/3 (1 + a/4 (1 + a/5 (1 + a/6))))), the next term below 5e-8 of the sum
-    float p = fmaf(a, 1.0f / 720.0f, 1.0f / 120.0f);
-    p = fmaf(p, a, 1.0f / 24.0f);
+    // a > -1/8: e^a - 1 = a (1 + a/2 (1 + a/3 (1 + a/4 (1 + a/5)))), the next term below 5e-8 of the sum
+    float p = fmaf(a, 1.0f / 120.0f, 1.0f / 24.0f);
     p = fmaf(p, a, 1.0f / 6.0f);
     p = fmaf(p, a, 0.5f);
     p = fmaf(p, a, 1.0f) * a;
-    const float slow = fmaf(S, p, u) + S;
-    const float fast = fmaf(S, __expf(a), u);
-    return a > -0.25f ? slow : fast;
+    const float e = __expf(a);
+    const bool slow = a > -0.125f;
+    return fmaf(S, slow ? p : e, u) + (slow ? S : 0.f);
 }
 
 // first row r with token_seq[r] >= b
@@ -48,6 +65,16 @@ __device__ __forceinline__ int first_row_of(const int* __restrict__ token_seq, i
 constexpr int SC_THREADS = 128;
 constexpr int SC_CH = 16;        // tokens a chunk
 
+template <int N> __device__ __forceinline__ void load_vec(const float* p, float* o) {
+    if (N == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        o[0] = v.x; o[N > 1 ? 1 : 0] = v.y; o[N > 2 ? 2 : 0] = v.z; o[N > 3 ? 3 : 0] = v.w;
+    } else if (N == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(p);
+        o[0] = v.x; o[N > 1 ? 1 : 0] = v.y;
+    } else o[0] = *p;
+}
+
 struct ScArgs {
     const float* dt; long ldt; const void* dt_bias; int db_dtype;
     const void* x; long ldx; const void* z; long ldz;
@@ -63,6 +90,7 @@ template <typename T, int L, int NPL>
 __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs a)
 {
     constexpr int CB = SC_THREADS / L;                       // channels a block
+    constexpr int VEC = NPL < 4 ? NPL : 4;                   // states a lane holds side by side
     constexpr int NP = L * NPL;                              // states a channel, padded
     constexpr int EPT = (SC_CH * CB + SC_THREADS - 1) / SC_THREADS;     // (token, channel) pairs a thread
     constexpr int BPT = (SC_CH * NP + SC_THREADS - 1) / SC_THREADS;     // (token, state) pairs a thread
@@ -84,7 +112,7 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
     float S[NPL], A[NPL];        // the states and their rates
 #pragma unroll
     for (int i = 0; i < NPL; ++i) {
-        const int n = (i >> 2) * 4 * L + part * 4 + (i & 3);
+        const int n = (i / VEC) * VEC * L + part * VEC + i % VEC;
         const bool in = live && n < N;
         S[i] = in ? sp[n] : 0.f;
         A[i] = in ? -expf(a.a_log[(long)ch * N + n]) : 0.f;
@@ -142,15 +170,15 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
             const float d = dt_s[tt][cl], dx = dx_s[tt][cl];
             float y0 = 0.f, y1 = 0.f;
 #pragma unroll
-            for (int i = 0; i < NPL; i += 4) {
-                const float4 bb = *reinterpret_cast<const float4*>(&b_s[tt][(i >> 2) * 4 * L + part * 4]);
-                const float4 cc = *reinterpret_cast<const float4*>(&c_s[tt][(i >> 2) * 4 * L + part * 4]);
-                S[i] = decay_add(S[i], d * A[i], dx * bb.x);
-                S[i + 1] = decay_add(S[i + 1], d * A[i + 1], dx * bb.y);
-                S[i + 2] = decay_add(S[i + 2], d * A[i + 2], dx * bb.z);
-                S[i + 3] = decay_add(S[i + 3], d * A[i + 3], dx * bb.w);
-                y0 = fmaf(S[i], cc.x, y0); y1 = fmaf(S[i + 1], cc.y, y1);
-                y0 = fmaf(S[i + 2], cc.z, y0); y1 = fmaf(S[i + 3], cc.w, y1);
+            for (int i = 0; i < NPL; i += VEC) {
+                float bb[VEC], cc[VEC];
+                load_vec<VEC>(&b_s[tt][(i / VEC) * VEC * L + part * VEC], bb);
+                load_vec<VEC>(&c_s[tt][(i / VEC) * VEC * L + part * VEC], cc);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) {
+                    S[i + j] = decay_add(S[i + j], d * A[i + j], dx * bb[j]);
+                    if (j & 1) y1 = fmaf(S[i + j], cc[j], y1); else y0 = fmaf(S[i + j], cc[j], y0);
+                }
             }
             rd_s[tt][threadIdx.x] = y0 + y1;
         }
@@ -164,7 +192,7 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
                 for (int l = 0; l < L; ++l) y += rd_s[tt][pc * L + l];
                 y = fmaf(skip, x_s[tt][pc], y);
                 const float zz = z_s[tt][pc];
-                reinterpret_cast<T*>(a.out)[(long)(c0 + tt) * a.ldo + pch] = from_f32<T>(y * (zz / (1.0f + expf(-zz))));
+                reinterpret_cast<T*>(a.out)[(long)(c0 + tt) * a.ldo + pch] = from_f32<T>(y * gate_silu<T>(zz));
             }
         }
     }
@@ -172,7 +200,7 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
     if (live) {
 #pragma unroll
         for (int i = 0; i < NPL; ++i) {
-            const int n = (i >> 2) * 4 * L + part * 4 + (i & 3);
+            const int n = (i / VEC) * VEC * L + part * VEC + i % VEC;
             if (n < N) sp[n] = S[i];
         }
     }
@@ -191,6 +219,9 @@ template <typename T>
 int scan_for(const ScArgs& a, int n_entries, cudaStream_t s)
 {
     const int n = a.n_state;
+    // Few channels leave the schedulers with a warp each, which waits for its own results: two states a lane and twice
+    // the warps then.
+    if (n > 8 && n <= 16 && (long)n_entries * a.inner * 4 / 32 < 6L * fx_sm_count()) return launch_sc<T, 8, 2>(a, n_entries, s);
     if (n <= 4) return launch_sc<T, 1, 4>(a, n_entries, s);
     if (n <= 8) return launch_sc<T, 2, 4>(a, n_entries, s);
     if (n <= 16) return launch_sc<T, 4, 4>(a, n_entries, s);

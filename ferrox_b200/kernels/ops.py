@@ -86,6 +86,8 @@ _SIGNATURES = {
     "fx_embed_streams": [_P, _I, _P, _P, _I, _I, _I, _I, _F, _P, _P],
     "fx_channel_decay_prep": [_P, _L, _P, _I, _P, _I, _F, _P, _I, _I, _I, _P],
     "fx_channel_decay_scan": [_P, _L, _P, _L, _P, _L, _P, _F, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
+    "fx_fixed_decay_scan": [_P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
+    "fx_silu_rows": [_P, _I, _L, _P, _L, _I, _I, _P],
     "fx_selective_scan": [_P, _L, _P, _I, _P, _L, _P, _L, _I, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "fx_split_rows": [_P, _L, _P, _L, _I, _I, _I, _P],
     "fx_mlstm_column_blocks": [_I, _I],
@@ -646,6 +648,27 @@ def channel_decay_scan(q, k, v, alpha, q_scale, state, out, token_seq, seq_slot,
     call("fx_channel_decay_scan", _ptr(q), _rows(q), _ptr(k), _rows(k), _ptr(v), _rows(v), _ptr(alpha), float(q_scale),
          _ptr(state), _ptr(out), _rows(out), _ptr(token_seq), _ptr(seq_slot), q.shape[0], int(n_entries), int(H), int(D),
          int(V), stream if stream is not None else stream_ptr())
+    return out
+
+
+def silu_rows(x, out, stream=None):
+    """out = silu(x) in 32 bits, over row views of one shape."""
+    if out.dtype != torch.float32 or out.shape != x.shape:
+        raise KernelError("silu_rows: 32-bit rows of the input's shape")
+    call("fx_silu_rows", _ptr(x), code(x), _rows(x), _ptr(out), _rows(out), x.shape[0], x.shape[1],
+         stream if stream is not None else stream_ptr())
+    return out
+
+
+def fixed_decay_scan(q, k, v, decay, state, out, token_seq, seq_slot, n_entries, H, D, V, stream=None):
+    """:func:`state_scan` without its delta rule and with one decay a head (``decay`` [H]), for steps of many tokens:
+    S = decay S + k v^T, out = S^T q, ``state`` [slots, H, V, D]; everything 32-bit, q, k and v behind their activation."""
+    for t in (q, k, v, decay, state, out):
+        if t.dtype != torch.float32:
+            raise KernelError("fixed_decay_scan: the recurrence is 32-bit")
+    call("fx_fixed_decay_scan", _ptr(q), _rows(q), _ptr(k), _rows(k), _ptr(v), _rows(v), _ptr(decay), _ptr(state), _ptr(out),
+         _rows(out), _ptr(token_seq), _ptr(seq_slot), q.shape[0], int(n_entries), int(H), int(D), int(V),
+         stream if stream is not None else stream_ptr())
     return out
 
 

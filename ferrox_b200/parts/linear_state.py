@@ -46,6 +46,10 @@ from ..weights.loader import TensorDecl
 from .base import Mixer, register_part
 
 
+# From this many tokens an entry of the step on, the fixed-decay recurrence takes the kernel made for prompts.
+FIXED_DECAY_MIN_TOKENS = 32
+
+
 def _cat_rows(tensors):
     dt = torch.float32 if any(t.dtype == torch.float32 for t in tensors) else tensors[0].dtype
     return torch.cat([t.to(dt) for t in tensors], dim=0).contiguous()
@@ -166,14 +170,27 @@ class DecayedLinearAttention(_StateMixer):
         proj = rt.empty(T, 2 * self.qk + 2 * self.vv)
         ops.linear(x, self.w_in, proj, status=batch.status, stream=batch.stream)
         read = rt.empty(T, self.vv, dtype=torch.float32)
-        # SiLU of q, k, v where the recurrence reads them
-        ops.state_scan(proj[:, :self.qk], proj[:, self.qk:2 * self.qk], proj[:, 2 * self.qk:2 * self.qk + self.vv],
-                       self.decay, 0, None, cache.states["matrix"], read, batch.token_seq, batch.seq_slot, batch.n_seqs,
-                       H, H, D, V, silu_on_load=True, stream=batch.stream)
+        if T >= FIXED_DECAY_MIN_TOKENS * batch.n_seqs:
+            # prompts: SiLU of q, k, v once, then the recurrence without anything to work out in its way
+            act = rt.empty(T, 2 * self.qk + self.vv, dtype=torch.float32)
+            ops.silu_rows(proj[:, :2 * self.qk + self.vv], act, stream=batch.stream)
+            ops.fixed_decay_scan(act[:, :self.qk], act[:, self.qk:2 * self.qk], act[:, 2 * self.qk:], self.decay,
+                                 cache.states["matrix"], read, batch.token_seq, batch.seq_slot, batch.n_seqs, H, D, V,
+                                 stream=batch.stream)
+        else:
+            self._scan_short(proj, read, batch, cache)
         y = rt.empty(T, self.vv)
         ops.gated_group_norm(read, proj[:, 2 * self.qk + self.vv:], self.norm_w, s.norm_eps, "sigmoid", y, 1, self.vv,
                              stream=batch.stream)
         ops.linear(y, self.w_o, out, accumulate=accumulate, status=batch.status, stream=batch.stream)
+
+    def _scan_short(self, proj, read, batch, cache):
+        s = self.spec
+        H, D, V = s.n_heads, s.head_dim, s.value_dim
+        # SiLU of q, k, v where the recurrence reads them
+        ops.state_scan(proj[:, :self.qk], proj[:, self.qk:2 * self.qk], proj[:, 2 * self.qk:2 * self.qk + self.vv],
+                       self.decay, 0, None, cache.states["matrix"], read, batch.token_seq, batch.seq_slot, batch.n_seqs,
+                       H, H, D, V, silu_on_load=True, stream=batch.stream)
 
 
 class GeneralDeltaRule(_StateMixer):
