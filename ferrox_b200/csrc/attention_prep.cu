@@ -448,9 +448,8 @@ extern "C" int fx_rotary_norm_store(void* qkv, int dtype, long ld, const int* po
     const int item = dtype == FX_F32 ? 16 : 8;     // bytes of four elements
     const bool vec = key_dim % 4 == 0 && value_dim % 4 == 0 && ld % 4 == 0 && (uintptr_t)qkv % item == 0 &&
                      (uintptr_t)k_pages % item == 0 && (uintptr_t)v_pages % item == 0;
-    // few tokens (a decode step): a token's heads are shared out over blocks
     const int units = n_heads + 2 * n_kv_heads;
-    dim3 grid(n_tokens, n_tokens < 256 ? (unsigned)fx_cdiv(units, RN_WARPS) : 1u);
+    dim3 grid(n_tokens, (unsigned)fx_cdiv(units, RN_WARPS));      // (a warp a head)
 #define FX_GO(T, N)                                                                                                   \
     fx_launch_pdl(rotary_norm_store_kernel<T, N>, grid, RN_WARPS * 32, smem, s, (T*)qkv, ld, positions, token_seq,   \
                   seq_slot, cos_sin, rot, pairing, eps, v_cos_sin, (T*)k_pages, (T*)v_pages, block_table, table_width, \

@@ -32,13 +32,18 @@ __device__ __forceinline__ int first_row_of(const int* __restrict__ token_seq, i
     return lo;
 }
 
-// sigmoid(z)^p = exp(-p log(1 + e^-z)): close to 1 the exponent keeps its relative precision.  The decay is raised to the
-// power of the distance a memory travels, so that a bias in its last place grows a thousandfold over a thousand tokens:
-// the last step is taken in 64 bits and rounded once.
+// sigmoid(z)^p = e^-a with a = p log(1 + e^-z): close to 1 the exponent keeps its relative precision.  The decay is raised
+// to the power of the distance a memory travels, so that a bias in its last place grows a thousandfold over a thousand
+// tokens: where a is small, e^-a is 1 plus e^-a - 1 from its Taylor series, rounded once.
 __device__ __forceinline__ float sigmoid_power(float z, float p)
 {
-    const float s = z < -20.f ? -z : log1pf(expf(-z));
-    return (float)exp(-(double)(p * s));
+    const float a = -p * fx_softplus(-z);
+    // a > -1/8: e^a - 1 = a (1 + a/2 (1 + a/3 (1 + a/4 (1 + a/5)))), the next term below 5e-8 of the sum
+    float q = fmaf(a, 1.0f / 120.0f, 1.0f / 24.0f);
+    q = fmaf(q, a, 1.0f / 6.0f);
+    q = fmaf(q, a, 0.5f);
+    q = fmaf(q, a, 1.0f);
+    return a > -0.125f ? fmaf(q, a, 1.0f) : expf(a);
 }
 
 constexpr int CP_THREADS = 128;
@@ -135,8 +140,10 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
         S[i] = (live && row < D) ? sp[row * a.row_stride] : 0.f;
     }
     // what lies beyond the head's D rows and the live columns stays zero in both buffers
-    for (int idx = threadIdx.x; idx < 2 * BUF; idx += CD_THREADS) sm[idx] = 0.f;
-    __syncthreads();
+    if (D < DP || nc < CD_COLS) {
+        for (int idx = threadIdx.x; idx < 2 * BUF; idx += CD_THREADS) sm[idx] = 0.f;
+        __syncthreads();
+    }
 
     // Staging.  Thread t copies piece t, t + 256, ... of a chunk; a piece's (token, place in the row) moves on by the
     // same step every time, so the quotient and the remainder are taken once and carried from piece to piece.
@@ -181,8 +188,7 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
         const float* k_s = q_s + CD_CH * DP;
         const float* w_s = k_s + CD_CH * DP;
         const float* v_s = sm + buf * BUF + ROWS * CD_CH * DP + col;
-#pragma unroll 4
-        for (int tt = 0; tt < nt; ++tt) {
+        auto token = [&](int tt) {      // one token: the state moves on; this thread's share of the read-out
             const float vt = v_s[tt * CD_COLS];
             float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
@@ -195,11 +201,22 @@ __global__ void __launch_bounds__(CD_THREADS) channel_decay_scan_kernel(const Cd
                 d0 = fmaf(S[i], qq.x, d0); d1 = fmaf(S[i + 1], qq.y, d1);
                 d2 = fmaf(S[i + 2], qq.z, d2); d3 = fmaf(S[i + 3], qq.w, d3);
             }
-            rd_s[tt * CD_THREADS + threadIdx.x] = (d0 + d1) + (d2 + d3);     // [token][group][column]
+            return (d0 + d1) + (d2 + d3);
+        };
+        // Whole chunks by four tokens: the shares are stored after the four, so that the second's rows are asked for while
+        // the first is worked on (a store to shared memory between them would hold the loads back).
+        int tt = 0;
+        for (; tt + 4 <= nt; tt += 4) {
+            float rd[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) rd[u] = token(tt + u);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) rd_s[(tt + u) * CD_THREADS + threadIdx.x] = rd[u];      // [token][group][column]
         }
+        for (; tt < nt; ++tt) rd_s[tt * CD_THREADS + threadIdx.x] = token(tt);
         __syncthreads();     // (also: everyone is done with this buffer before the chunk after next is copied into it)
         {
-            const int tt = grp;      // (as many tokens a chunk as groups)
+            tt = grp;      // (as many tokens a chunk as groups)
             if (tt < nt && live) {
                 float s = 0.f;
 #pragma unroll
@@ -251,6 +268,18 @@ __global__ void silu_rows_kernel(const T* __restrict__ x, long ldx, float* __res
     fx_pdl_wait();
     const T* r = x + (long)blockIdx.x * ldx;
     float* o = out + (long)blockIdx.x * ldo;
+    constexpr int N = Pack<T>::N;
+    if (n % N == 0 && (uintptr_t)r % 16 == 0 && (uintptr_t)o % 16 == 0) {
+        for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * N; i < n; i += gridDim.y * blockDim.x * N) {
+            float v[N];
+            Pack<T>::load(r + i, v);
+#pragma unroll
+            for (int e = 0; e < N; ++e) v[e] = v[e] / (1.0f + expf(-v[e]));
+#pragma unroll
+            for (int e = 0; e < N; e += 4) Pack<float>::store(o + i + e, v + e);
+        }
+        return;
+    }
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n; i += gridDim.y * blockDim.x) {
         const float v = to_f32(r[i]);
         o[i] = v / (1.0f + expf(-v));

@@ -148,6 +148,21 @@ __device__ __forceinline__ void fx_gate_32(float* x, const uint32_t* u, int act,
     }
 }
 
+// log(1 + e^x) = max(x, 0) + log(1 + e) with e = e^-|x| in (0, 1]; log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3, by
+// its series 2 (s + s^3/3 + s^5/5 + ...), the first term left out below 2e-8 of the sum.
+__device__ __forceinline__ float fx_softplus(float x)
+{
+    const float e = expf(-fabsf(x));
+    const float s = e / (2.0f + e), s2 = s * s;
+    float p = fmaf(s2, 1.0f / 15.0f, 1.0f / 13.0f);
+    p = fmaf(p, s2, 1.0f / 11.0f);
+    p = fmaf(p, s2, 1.0f / 9.0f);
+    p = fmaf(p, s2, 1.0f / 7.0f);
+    p = fmaf(p, s2, 1.0f / 5.0f);
+    p = fmaf(p, s2, 1.0f / 3.0f);
+    return fmaxf(x, 0.f) + 2.0f * fmaf(s * s2, p, s);
+}
+
 // sigmoid(g) with the hardware's exponential and quotient, for the attention kernels' output gates.
 __device__ __forceinline__ float fx_sigmoid_fast(float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); }
 

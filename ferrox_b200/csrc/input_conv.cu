@@ -65,6 +65,17 @@ template <> __device__ __forceinline__ float2 load2<float>(const float* p) { ret
 template <> __device__ __forceinline__ float2 load2<bf16>(const bf16* p) {
     return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
 }
+template <typename T> struct T2;      // two neighbouring elements as they lie in memory
+template <> struct T2<float> {
+    float2 v;
+    __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float2*>(p); }
+    __device__ __forceinline__ float2 value() const { return v; }
+};
+template <> struct T2<bf16> {
+    __nv_bfloat162 v;
+    __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const __nv_bfloat162*>(p); }
+    __device__ __forceinline__ float2 value() const { return __bfloat1622float2(v); }
+};
 __device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void store2(bf16* p, float2 v) {
     *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y);
@@ -86,9 +97,20 @@ __global__ void __launch_bounds__(CONV_THREADS) input_conv_run_kernel(
         wt[j] = make_float2(load_any(w, w_dtype, (long)c * TAPS + j), load_any(w, w_dtype, (long)(c + 1) * TAPS + j));
     float2 b0 = make_float2(0.f, 0.f);
     if (bias) b0 = make_float2(load_any(bias, b_dtype, c), load_any(bias, b_dtype, c + 1));
+    // the run's inputs and entries, all asked for before the first is used
+    T2<T> xs[CONV_RUN];
+    int ss[CONV_RUN];
+#pragma unroll
+    for (int r = 0; r < CONV_RUN; ++r) {
+        const int t = min(t0 + r, n_tokens - 1);
+        xs[r].load(x + (long)t * ldx + c);
+        ss[r] = token_seq[t];
+    }
     int seq = -1;
-    for (int t = t0; t < t1; ++t) {
-        const int s = token_seq[t];
+#pragma unroll
+    for (int r = 0; r < CONV_RUN; ++r) {
+        const int t = t0 + r, s = ss[r];
+        if (t >= t1) break;
         if (s != seq) {       // the run's first token, or another entry's: its earlier inputs, from rows and tail
             seq = s;
             int own = 0;
@@ -103,7 +125,7 @@ __global__ void __launch_bounds__(CONV_THREADS) input_conv_run_kernel(
         }
 #pragma unroll
         for (int j = 0; j + 1 < TAPS; ++j) hist[j] = hist[j + 1];
-        const float2 xt = load2(x + (long)t * ldx + c);
+        const float2 xt = xs[r].value();
         hist[TAPS - 1] = xt;
         float2 acc = add_input ? xt : make_float2(0.f, 0.f);
         acc.x += b0.x; acc.y += b0.y;

@@ -18,21 +18,6 @@
 
 namespace {
 
-// log(1 + e^x) = max(x, 0) + log(1 + e) with e = e^-|x| in (0, 1]; log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3, by
-// its series 2 (s + s^3/3 + s^5/5 + ...), the first term left out below 2e-8 of the sum.
-__device__ __forceinline__ float softplus_f(float x)
-{
-    const float e = expf(-fabsf(x));
-    const float s = e / (2.0f + e), s2 = s * s;
-    float p = fmaf(s2, 1.0f / 15.0f, 1.0f / 13.0f);
-    p = fmaf(p, s2, 1.0f / 11.0f);
-    p = fmaf(p, s2, 1.0f / 9.0f);
-    p = fmaf(p, s2, 1.0f / 7.0f);
-    p = fmaf(p, s2, 1.0f / 5.0f);
-    p = fmaf(p, s2, 1.0f / 3.0f);
-    return fmaxf(x, 0.f) + 2.0f * fmaf(s * s2, p, s);
-}
-
 // z / (1 + e^-z); in 16 bits the hardware's exponential and quotient do.
 template <typename T> __device__ __forceinline__ float gate_silu(float z) {
     return sizeof(T) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));
@@ -123,14 +108,15 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
     const int gch = plive ? pch : I - 1;
     const float bias = load_any(a.dt_bias, a.db_dtype, gch), skip = a.d_skip[gch];
 
-    float fdt[EPT], fx[EPT], fz[EPT], fb[BPT], fc[BPT];
+    float fdt[EPT], fb[BPT], fc[BPT];
+    T fx[EPT], fz[EPT];      // (as loaded: a conversion here would wait for the load)
     auto fetch = [&](int c0, int nt) {       // every load unconditional, from places clamped into the chunk
 #pragma unroll
         for (int e = 0; e < EPT; ++e) {
             const long t = c0 + min(ptt + e * L, nt - 1);
             fdt[e] = a.dt[t * a.ldt + gch];
-            fx[e] = to_f32(xp[t * a.ldx + gch]);
-            fz[e] = to_f32(zp[t * a.ldz + gch]);
+            fx[e] = xp[t * a.ldx + gch];
+            fz[e] = zp[t * a.ldz + gch];
         }
 #pragma unroll
         for (int e = 0; e < BPT; ++e) {
@@ -149,9 +135,10 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
         for (int e = 0; e < EPT; ++e) {
             const int tt = ptt + e * L;
             if (tt < SC_CH) {
-                const float d = softplus_f(fdt[e] + bias);
-                dt_s[tt][pc] = d; dx_s[tt][pc] = d * fx[e];
-                x_s[tt][pc] = fx[e]; z_s[tt][pc] = fz[e];
+                const float d = fx_softplus(fdt[e] + bias);
+                const float xx = to_f32(fx[e]);
+                dt_s[tt][pc] = d; dx_s[tt][pc] = d * xx;
+                x_s[tt][pc] = xx; z_s[tt][pc] = to_f32(fz[e]);
             }
         }
 #pragma unroll
@@ -165,8 +152,7 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
         }
         __syncthreads();
         if (c0 + SC_CH < r1) fetch(c0 + SC_CH, min(SC_CH, r1 - c0 - SC_CH));
-#pragma unroll 4
-        for (int tt = 0; tt < nt; ++tt) {
+        auto token = [&](int tt) {      // one token: the states move on; this lane's share of the read-out
             const float d = dt_s[tt][cl], dx = dx_s[tt][cl];
             float y0 = 0.f, y1 = 0.f;
 #pragma unroll
@@ -180,8 +166,17 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
                     if (j & 1) y1 = fmaf(S[i + j], cc[j], y1); else y0 = fmaf(S[i + j], cc[j], y0);
                 }
             }
-            rd_s[tt][threadIdx.x] = y0 + y1;
+            return y0 + y1;
+        };
+        int tt0 = 0;
+        for (; tt0 + 4 <= nt; tt0 += 4) {
+            float rd[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) rd[u] = token(tt0 + u);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) rd_s[tt0 + u][threadIdx.x] = rd[u];
         }
+        for (; tt0 < nt; ++tt0) rd_s[tt0][threadIdx.x] = token(tt0);
         __syncthreads();
 #pragma unroll
         for (int e = 0; e < EPT; ++e) {

@@ -35,7 +35,11 @@ template <int N> __device__ __forceinline__ void load_row(const void* p, int dty
     o[2] = __uint_as_float(v.y << 16); o[3] = __uint_as_float(v.y & 0xffff0000u);
 }
 
-template <int S, int N>
+// EXPERTS: 0 none, 1 any, 2 bfloat16 rows of at most MAX_K experts, whose loads are all on their way together with the
+// streams'.
+constexpr int MAX_K = 8;
+
+template <int S, int N, int EXPERTS>
 __global__ void __launch_bounds__(512) stream_step_kernel(const StreamStep a)
 {
     extern __shared__ __align__(16) float u_s[];
@@ -47,14 +51,45 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamStep a)
     float sg = 1.f;
     if (a.shared && a.shared_gate) sg = 1.0f / (1.0f + expf(-a.shared_gate[t * a.gate_ld]));
     float ss = 0.f;
+    long er[MAX_K];       // where the token's experts' rows start
+    float ew[MAX_K];
+    if (EXPERTS == 2) {
+#pragma unroll
+        for (int k = 0; k < MAX_K; ++k)
+            if (k < a.top_k) {
+                er[k] = (long)a.place[t * a.top_k + k] * W;
+                ew[k] = a.weight ? a.weight[t * a.top_k + k] : 1.f;
+            }
+    }
     for (int i = threadIdx.x * N; i < W; i += blockDim.x * N) {
         float x[S][N], y[3][N], e[N];
+        uint2 raw[MAX_K + 1];
+        if (EXPERTS == 2) {
+            const bf16* rows = reinterpret_cast<const bf16*>(a.expert_rows) + i;
+#pragma unroll
+            for (int k = 0; k < MAX_K; ++k)
+                if (k < a.top_k) raw[k] = *reinterpret_cast<const uint2*>(rows + er[k]);
+            if (a.shared) raw[MAX_K] = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(a.shared) + t * W + i);
+        }
 #pragma unroll
         for (int s = 0; s < S; ++s) load32<N>(X + (long)s * W + i, x[s]);
 #pragma unroll
         for (int j = 0; j < 3; ++j)
             if (j < a.n_terms) load32<N>(a.y[j] + t * W + i, y[j]);
-        if (a.place) {
+        if (EXPERTS == 2) {
+            auto add = [&](uint2 r, float w) {      // (N is 4 here)
+                e[0] = fmaf(w, __uint_as_float(r.x << 16), e[0]);
+                e[N > 1 ? 1 : 0] = fmaf(w, __uint_as_float(r.x & 0xffff0000u), e[N > 1 ? 1 : 0]);
+                e[N > 2 ? 2 : 0] = fmaf(w, __uint_as_float(r.y << 16), e[N > 2 ? 2 : 0]);
+                e[N > 3 ? 3 : 0] = fmaf(w, __uint_as_float(r.y & 0xffff0000u), e[N > 3 ? 3 : 0]);
+            };
+#pragma unroll
+            for (int n = 0; n < N; ++n) e[n] = 0.f;
+#pragma unroll
+            for (int k = 0; k < MAX_K; ++k)
+                if (k < a.top_k) add(raw[k], ew[k]);
+            if (a.shared) add(raw[MAX_K], sg);
+        } else if (EXPERTS == 1) {
 #pragma unroll
             for (int n = 0; n < N; ++n) e[n] = 0.f;
 #pragma unroll 4
@@ -92,7 +127,7 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamStep a)
 #pragma unroll
                         for (int n = 0; n < N; ++n) z[n] = fmaf(a.coef[j][to], y[j][n], z[n]);
                     }
-                if (a.place) {
+                if (EXPERTS) {
 #pragma unroll
                     for (int n = 0; n < N; ++n) z[n] = fmaf(a.coef[3][to], e[n], z[n]);
                 }
@@ -111,7 +146,7 @@ __global__ void __launch_bounds__(512) stream_step_kernel(const StreamStep a)
 #pragma unroll
                     for (int n = 0; n < N; ++n) u[n] = fmaf(a.coef[j][0], y[j][n], u[n]);
                 }
-            if (a.place) {
+            if (EXPERTS) {
 #pragma unroll
                 for (int n = 0; n < N; ++n) u[n] = fmaf(a.coef[3][0], e[n], u[n]);
             }
@@ -149,7 +184,9 @@ int launch(const StreamStep& a, int n_rows, bool vec, cudaStream_t s)
     int nt = 64;
     while (nt < items && nt < most) nt <<= 1;
     const size_t smem = a.x_out ? (size_t)((a.hidden + 3) & ~3) * 4 : 0;
-    auto kern = vec ? stream_step_kernel<S, 4> : stream_step_kernel<S, 1>;
+    const bool ahead = vec && a.expert_dtype == FX_BF16 && a.top_k <= MAX_K;
+    auto kern = a.place ? (ahead ? stream_step_kernel<S, 4, 2> : vec ? stream_step_kernel<S, 4, 1> : stream_step_kernel<S, 1, 1>)
+                        : (vec ? stream_step_kernel<S, 4, 0> : stream_step_kernel<S, 1, 0>);
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
