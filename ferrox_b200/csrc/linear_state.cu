@@ -110,7 +110,7 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
 }
 
 // The convolution's tail after the step: the last taps - 1 inputs of every entry, from its rows of this step and,
-// where the entry brought fewer, from the old tail.  One block per entry; a thread reads all it needs of a channel
+// where the entry brought fewer, from the old tail.  Grid (entries, channels); a thread reads all it needs of a channel
 // before it writes.
 template <typename T>
 __global__ void __launch_bounds__(256) conv_tail_update_kernel(
@@ -123,7 +123,7 @@ __global__ void __launch_bounds__(256) conv_tail_update_kernel(
     const int n = r1 - r0, keep = taps - 1;
     if (n <= 0) return;
     float* tl = tail + (long)seq_slot[b] * keep * C;
-    for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
         float v[MAX_TAPS];
         for (int j = 0; j < keep; ++j) {
             const int rel = n - keep + j;     // index among the entry's rows; negative: before the step
@@ -492,9 +492,10 @@ extern "C" int fx_conv_tail_update(const void* proj, int dtype, long ldp, int ch
 {
     if (n_tokens <= 0 || n_entries <= 0 || taps <= 1) return FX_OK;
     if (taps > MAX_TAPS) return FX_ERR_SIZE;
+    dim3 grid(n_entries, (unsigned)(channels > 256 * 64 ? 64 : fx_cdiv(channels, 256)));
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == FX_F32) fx_launch_pdl(conv_tail_update_kernel<float>, n_entries, 256, 0, s, (const float*)proj, ldp, channels, taps, tail, token_seq, seq_slot, n_tokens);
-    else if (dtype == FX_BF16) fx_launch_pdl(conv_tail_update_kernel<bf16>, n_entries, 256, 0, s, (const bf16*)proj, ldp, channels, taps, tail, token_seq, seq_slot, n_tokens);
+    if (dtype == FX_F32) fx_launch_pdl(conv_tail_update_kernel<float>, grid, 256, 0, s, (const float*)proj, ldp, channels, taps, tail, token_seq, seq_slot, n_tokens);
+    else if (dtype == FX_BF16) fx_launch_pdl(conv_tail_update_kernel<bf16>, grid, 256, 0, s, (const bf16*)proj, ldp, channels, taps, tail, token_seq, seq_slot, n_tokens);
     else return FX_ERR_DTYPE;
     return fx_launch_status();
 }

@@ -356,7 +356,7 @@ def test_streams_updated_and_read(dtype, S):
     g = torch.Generator().manual_seed(S)
     R = lambda *s: torch.randn(*s, generator=g)
     tol_x = 1e-5 if dt == torch.float32 else 1e-2
-    for T, W, n_terms, K in ((1, 64, 1, 0), (5, 72, 2, 2), (300, 130, 3, 3), (3, 2048, 1, 4), (270, 4096, 2, 1), (2, 51, 0, 2), (2, 5000, 1, 0)):
+    for T, W, n_terms, K in ((1, 64, 1, 0), (5, 72, 2, 2), (300, 130, 3, 3), (3, 2048, 1, 4), (270, 4096, 2, 1), (2, 51, 0, 2), (2, 5000, 1, 0), (6, 64, 1, 9)):
         X, ys = R(S, T, W), [R(T, W) for _ in range(n_terms)]
         mix, coef, coef_e, reads = R(S, S), [R(S) for _ in ys], R(S), R(S)
         w = 1 + 0.2 * R(W)
