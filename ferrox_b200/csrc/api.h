@@ -349,7 +349,8 @@ int fx_silu_rows(const void* x, int dtype, long ldx, float* out, long ldo, int n
 
 // Selective state space (selective_scan.cu): per channel step = softplus(dt + dt_bias), the state row
 // s = e^(-step e^A_log) * s + step x B, out = (s . C + D x) silu(z); state [slots, inner, n_state] 32-bit.
-int fx_selective_scan(const float* dt, long ldt, const void* dt_bias, int db_dtype, const void* x, long ldx, const void* z,
+// w_dt (optional): dt holds low-rank rows [tokens][rank] and the step sizes are w_dt . dt; every entry brings one token.
+int fx_selective_scan(const float* dt, long ldt, const void* w_dt, int w_dtype, long ldw, int rank, const void* dt_bias, int db_dtype, const void* x, long ldx, const void* z,
                       long ldz, int dtype, const float* bc, long ldbc, const float* a_log, const float* d_skip,
                       float* state, void* out, long ldo, const int* token_seq, const int* seq_slot, int n_tokens,
                       int n_entries, int inner, int n_state, void* stream);

@@ -255,6 +255,68 @@ __global__ void __launch_bounds__(RN_WARPS * 32) rotary_norm_store_kernel(
     }
 }
 
+// The same for heads of up to 128 elements rotated on pairs (i, i + rot / 2) whose halves are whole pieces of four: a lane
+// holds its piece of the head and, where that is rotated, the partner piece, in registers; nothing passes through shared
+// memory.  (A query head is written over itself: every lane has its pieces before the sum over the warp.)
+template <typename T>
+__global__ void __launch_bounds__(RN_WARPS * 32) rotary_norm_store_128_kernel(
+    T* __restrict__ qkv, long ld, const int* __restrict__ positions, const int* __restrict__ token_seq,
+    const int* __restrict__ seq_slot, const float* __restrict__ cos_sin, int rot, float eps,
+    const float* __restrict__ v_cos_sin, T* __restrict__ k_pages, T* __restrict__ v_pages,
+    const int* __restrict__ block_table, int table_width, int page_size, int H, int G, int D, int V, int write_cache,
+    int* __restrict__ status)
+{
+    fx_pdl_wait();
+    const int t = blockIdx.x, i = (threadIdx.x & 31) * 4, warp = threadIdx.x >> 5;
+    const int u = blockIdx.y * RN_WARPS + warp;
+    if (u >= H + 2 * G) return;      // (whole warps; no barrier below)
+    const bool is_q = u < H, is_v = u >= H + G;
+    T* x = qkv + (long)t * ld + (is_v ? (long)(H + G) * D + (long)(u - H - G) * V : (long)u * D);
+    T* dst = x;
+    if (!is_q) {
+        if (!write_cache) return;
+        const int pos = positions[t], p = pos / page_size;
+        const int page = block_table[(long)seq_slot[token_seq[t]] * table_width + p];
+        if (page < 0) { if ((threadIdx.x & 31) == 0 && status) atomicExch(status, 2); return; }
+        const int g = is_v ? u - H - G : u - H;
+        dst = (is_v ? v_pages : k_pages) + (((long)page * G + g) * page_size + (pos - p * page_size)) * (is_v ? V : D);
+    }
+    const int width = is_v ? V : D, half = cos_sin ? rot >> 1 : 0;
+    const bool in = i < width;
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
+    if (in) Items<T, 4>::load(x + i, a);
+    if (is_v) {
+        if (!in) return;
+        if (v_cos_sin) {
+            const float4 f = *reinterpret_cast<const float4*>(v_cos_sin + (long)t * V + i);      // (two pairs)
+            const float b0 = a[0], b2 = a[2];
+            a[0] = b0 * f.x - a[1] * f.y; a[1] = a[1] * f.x + b0 * f.y;
+            a[2] = b2 * f.z - a[3] * f.w; a[3] = a[3] * f.z + b2 * f.w;
+        }
+        Items<T, 4>::store(dst + i, a);
+        return;
+    }
+    float b[4] = {0.f, 0.f, 0.f, 0.f};
+    const bool turned = i < 2 * half, second = i >= half;
+    if (turned) Items<T, 4>::load(x + (second ? i - half : i + half), b);
+    if (eps >= 0.f) {      // (a rotation leaves the sum of squares as it is)
+        const float ss = warp_sum(fmaf(a[0], a[0], fmaf(a[1], a[1], fmaf(a[2], a[2], a[3] * a[3]))));
+        const float r = 1.0f / sqrtf(ss / (float)D + eps);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { a[e] *= r; b[e] *= r; }
+    }
+    __syncwarp();
+    if (!in) return;
+    if (turned) {
+        const float* cs = cos_sin + ((long)t * half + (second ? i - half : i)) * 2;
+        const float4 f0 = *reinterpret_cast<const float4*>(cs), f1 = *reinterpret_cast<const float4*>(cs + 4);
+        const float sg = second ? 1.f : -1.f;
+        a[0] = a[0] * f0.x + sg * b[0] * f0.y; a[1] = a[1] * f0.z + sg * b[1] * f0.w;
+        a[2] = a[2] * f1.x + sg * b[2] * f1.y; a[3] = a[3] * f1.z + sg * b[3] * f1.w;
+    }
+    Items<T, 4>::store(dst + i, a);
+}
+
 // ---------------------------------------------------------------------------------------------------------------
 // The latent form.  Per token: `dkv` = [C latent | R rotated key part] as projected, `q` = H heads of [D | R].
 //   c <- dkv[:C] / sqrt(mean(dkv[:C]^2) + eps) * wc            -> pages[position][0:C]
@@ -454,6 +516,18 @@ extern "C" int fx_rotary_norm_store(void* qkv, int dtype, long ld, const int* po
     fx_launch_pdl(rotary_norm_store_kernel<T, N>, grid, RN_WARPS * 32, smem, s, (T*)qkv, ld, positions, token_seq,   \
                   seq_slot, cos_sin, rot, pairing, eps, v_cos_sin, (T*)k_pages, (T*)v_pages, block_table, table_width, \
                   page_size, n_heads, n_kv_heads, key_dim, value_dim, write_cache, status)
+    if (vec && pairing == 0 && rot % 8 == 0 && key_dim <= 128 && value_dim <= 128 && (uintptr_t)cos_sin % 16 == 0 &&
+        (uintptr_t)v_cos_sin % 16 == 0) {
+#define FX_GO128(T)                                                                                                   \
+    fx_launch_pdl(rotary_norm_store_128_kernel<T>, grid, RN_WARPS * 32, 0, s, (T*)qkv, ld, positions, token_seq,     \
+                  seq_slot, cos_sin, rot, eps, v_cos_sin, (T*)k_pages, (T*)v_pages, block_table, table_width, page_size, \
+                  n_heads, n_kv_heads, key_dim, value_dim, write_cache, status)
+        if (dtype == FX_F32) FX_GO128(float);
+        else if (dtype == FX_BF16) FX_GO128(bf16);
+        else return FX_ERR_DTYPE;
+#undef FX_GO128
+        return fx_launch_status();
+    }
     if (dtype == FX_F32) { if (vec) FX_GO(float, 4); else FX_GO(float, 1); }
     else if (dtype == FX_BF16) { if (vec) FX_GO(bf16, 4); else FX_GO(bf16, 1); }
     else return FX_ERR_DTYPE;

@@ -69,6 +69,8 @@ template <int N> __device__ __forceinline__ void load_vec(const float* p, float*
 
 struct ScArgs {
     const float* dt; long ldt; const void* dt_bias; int db_dtype;
+    // (instead of dt, every entry bringing one token) rows [rank] of the small matrix, and the tokens' low-rank rows
+    const void* w_dt; long ldw; int w_bf16, rank; const float* low; long ldlow;
     const void* x; long ldx; const void* z; long ldz;
     const float* bc; long ldbc;              // [tokens][B (n_state) | C (n_state)]
     const float* a_log; const float* d_skip; // [inner][n_state], [inner]
@@ -78,7 +80,8 @@ struct ScArgs {
     int n_tokens, inner, n_state;
 };
 
-template <typename T, int L, int NPL>
+// STEPS: the kernel works out the step sizes itself (a.w_dt).
+template <typename T, int L, int NPL, bool STEPS>
 __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs a)
 {
     constexpr int CB = SC_THREADS / L;                       // channels a block
@@ -92,24 +95,19 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
     __shared__ float x_s[SC_CH][CB], z_s[SC_CH][CB];
     __shared__ __align__(16) float b_s[SC_CH][NP], c_s[SC_CH][NP];
     __shared__ float rd_s[SC_CH][SC_THREADS];
-    fx_pdl_wait_only();
-    const int b = blockIdx.x;
-    const int r0 = first_row_of(a.token_seq, a.n_tokens, b), r1 = first_row_of(a.token_seq, a.n_tokens, b + 1);
-    if (r1 <= r0) return;
     const int ch0 = blockIdx.y * CB, I = a.inner, N = a.n_state;
     const int cl = threadIdx.x / L, part = threadIdx.x % L, ch = ch0 + cl;
     const bool live = ch < I;
-    float* sp = a.state + ((long)a.seq_slot[b] * I + (live ? ch : 0)) * N;
     const T* xp = reinterpret_cast<const T*>(a.x);
     const T* zp = reinterpret_cast<const T*>(a.z);
 
+    // Weights first: they are nobody's work.  (Nothing that any kernel or copy writes is read before the wait, however long
+    // ago it was written: the SM's own cache may still hold what stood there before.)
     float S[NPL], A[NPL];        // the states and their rates
 #pragma unroll
     for (int i = 0; i < NPL; ++i) {
         const int n = (i / VEC) * VEC * L + part * VEC + i % VEC;
-        const bool in = live && n < N;
-        S[i] = in ? sp[n] : 0.f;
-        A[i] = in ? -expf(a.a_log[(long)ch * N + n]) * (sizeof(T) == 2 ? 1.4426950408889634f : 1.f) : 0.f;
+        A[i] = live && n < N ? -expf(a.a_log[(long)ch * N + n]) * (sizeof(T) == 2 ? 1.4426950408889634f : 1.f) : 0.f;
     }
     // the channel of this thread's (token, channel) pairs is the same in every chunk: CB divides the block
     const int pc = threadIdx.x % CB, ptt = threadIdx.x / CB, pch = ch0 + pc;
@@ -117,13 +115,60 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScArgs
     const int gch = plive ? pch : I - 1;
     const float bias = load_any(a.dt_bias, a.db_dtype, gch), skip = a.d_skip[gch];
 
+    // A decode step's step sizes: the low-rank row of the entry's one token times the block's rows of the small matrix,
+    // which the lanes of a channel share out.
+    const int row_pieces = a.rank / 8;
+    uint4 wp[2];
+    const bool pieces = STEPS && a.w_bf16 && a.rank % 8 == 0 && row_pieces <= 2 * L;
+    if (pieces && live) {
+        const uint4* wr = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.w_dt) + (long)ch * a.ldw);
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            if (part + k * L < row_pieces) wp[k] = wr[part + k * L];
+    }
+    fx_pdl_wait_only();
+    const int b = blockIdx.x;
+    const int r0 = first_row_of(a.token_seq, a.n_tokens, b), r1 = first_row_of(a.token_seq, a.n_tokens, b + 1);
+    if (r1 <= r0) return;
+    float* sp = a.state + ((long)a.seq_slot[b] * I + (live ? ch : 0)) * N;
+#pragma unroll
+    for (int i = 0; i < NPL; ++i) {
+        const int n = (i / VEC) * VEC * L + part * VEC + i % VEC;
+        S[i] = live && n < N ? sp[n] : 0.f;
+    }
+    if (STEPS) {
+        float acc = 0.f;
+        const float* lr = a.low + (long)r0 * a.ldlow;
+        if (live) {
+            if (pieces) {
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+                    if (part + k * L < row_pieces) {
+                        const float* l = lr + (part + k * L) * 8;
+                        const uint32_t w4[4] = {wp[k].x, wp[k].y, wp[k].z, wp[k].w};
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            acc = fmaf(__uint_as_float(w4[e] << 16), l[2 * e], acc);
+                            acc = fmaf(__uint_as_float(w4[e] & 0xffff0000u), l[2 * e + 1], acc);
+                        }
+                    }
+            } else {
+                for (int r = part; r < a.rank; r += L) acc = fmaf(load_any(a.w_dt, a.w_bf16 ? FX_BF16 : FX_F32, (long)ch * a.ldw + r), lr[r], acc);
+            }
+        }
+#pragma unroll
+        for (int o = L >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (part == 0) dt_s[0][cl] = acc;
+        __syncthreads();
+    }
+
     float fdt[EPT], fb[BPT], fc[BPT];
     T fx[EPT], fz[EPT];      // (as loaded: a conversion here would wait for the load)
     auto fetch = [&](int c0, int nt) {       // every load unconditional, from places clamped into the chunk
 #pragma unroll
         for (int e = 0; e < EPT; ++e) {
             const long t = c0 + min(ptt + e * L, nt - 1);
-            fdt[e] = a.dt[t * a.ldt + gch];
+            fdt[e] = STEPS ? dt_s[0][pc] : a.dt[t * a.ldt + gch];      // (STEPS: one token, one chunk)
             fx[e] = xp[t * a.ldx + gch];
             fz[e] = zp[t * a.ldz + gch];
         }
@@ -215,7 +260,8 @@ int launch_sc(const ScArgs& a, int n_entries, cudaStream_t s)
 {
     dim3 grid(n_entries, (unsigned)fx_cdiv(a.inner, SC_THREADS / L));
     // a prompt's recurrence starts on an empty device (see fx_launch_pdl_if); a decode step's is set up early
-    fx_launch_pdl_if(a.n_tokens < 8 * n_entries, selective_scan_kernel<T, L, NPL>, grid, dim3(SC_THREADS), 0, s, a);
+    if (a.w_dt) fx_launch_pdl(selective_scan_kernel<T, L, NPL, true>, grid, dim3(SC_THREADS), 0, s, a);
+    else fx_launch_pdl_if(a.n_tokens < 8 * n_entries, selective_scan_kernel<T, L, NPL, false>, grid, dim3(SC_THREADS), 0, s, a);
     return fx_launch_status();
 }
 
@@ -252,14 +298,21 @@ __global__ void split_rows_kernel(const float* __restrict__ x, long ldx, bf16* _
 
 }  // namespace
 
-extern "C" int fx_selective_scan(const float* dt, long ldt, const void* dt_bias, int db_dtype, const void* x, long ldx,
+// w_dt (optional, [inner][ldw], its first `rank` columns): dt is then w_dt . low, worked out here, `dt` being the rows low
+// [tokens][rank]; only when every entry of the step brings exactly one token.
+extern "C" int fx_selective_scan(const float* dt, long ldt, const void* w_dt, int w_dtype, long ldw, int rank,
+                                 const void* dt_bias, int db_dtype, const void* x, long ldx,
                                  const void* z, long ldz, int dtype, const float* bc, long ldbc, const float* a_log,
                                  const float* d_skip, float* state, void* out, long ldo, const int* token_seq,
                                  const int* seq_slot, int n_tokens, int n_entries, int inner, int n_state, void* stream)
 {
     if (n_tokens <= 0 || n_entries <= 0) return FX_OK;
     if (inner <= 0 || n_state <= 0 || n_state > 256 || fx_cdiv(inner, 4) > 65535) return FX_ERR_SIZE;
+    if (w_dt && (n_tokens != n_entries || rank <= 0 || ldw < rank || (w_dtype == FX_BF16 && rank % 8 == 0 && (ldw % 8 || (uintptr_t)w_dt % 16))))
+        return FX_ERR_SIZE;
+    if (w_dt && w_dtype != FX_BF16 && w_dtype != FX_F32) return FX_ERR_DTYPE;
     ScArgs a;
+    a.w_dt = w_dt; a.ldw = ldw; a.w_bf16 = w_dtype == FX_BF16; a.rank = w_dt ? rank : 0; a.low = dt; a.ldlow = ldt;
     a.dt = dt; a.ldt = ldt; a.dt_bias = dt_bias; a.db_dtype = db_dtype; a.x = x; a.ldx = ldx; a.z = z; a.ldz = ldz;
     a.bc = bc; a.ldbc = ldbc; a.a_log = a_log; a.d_skip = d_skip; a.state = state; a.out = out; a.ldo = ldo;
     a.token_seq = token_seq; a.seq_slot = seq_slot; a.n_tokens = n_tokens; a.inner = inner; a.n_state = n_state;

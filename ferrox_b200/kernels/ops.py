@@ -88,7 +88,7 @@ _SIGNATURES = {
     "fx_channel_decay_scan": [_P, _L, _P, _L, _P, _L, _P, _F, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
     "fx_fixed_decay_scan": [_P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
     "fx_silu_rows": [_P, _I, _L, _P, _L, _I, _I, _P],
-    "fx_selective_scan": [_P, _L, _P, _I, _P, _L, _P, _L, _I, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P],
+    "fx_selective_scan": [_P, _L, _P, _I, _L, _I, _P, _I, _P, _L, _P, _L, _I, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "fx_split_rows": [_P, _L, _P, _L, _I, _I, _I, _P],
     "fx_mlstm_column_blocks": [_I, _I],
     "fx_mlstm_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _I, _F, _F, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I,
@@ -675,11 +675,14 @@ def fixed_decay_scan(q, k, v, decay, state, out, token_seq, seq_slot, n_entries,
 SELECTIVE_SCAN_MAX_STATE = 256
 
 
-def selective_scan(dt, dt_bias, x, z, bc, a_log, d_skip, state, out, token_seq, seq_slot, n_entries, stream=None):
+def selective_scan(dt, dt_bias, x, z, bc, a_log, d_skip, state, out, token_seq, seq_slot, n_entries, stream=None, w_dt=None):
     """The selective state space over every entry's tokens in order (csrc/selective_scan.cu): ``dt`` [T, inner] 32-bit
     before bias and softplus, ``x`` and ``z`` row views [T, inner] of the engine's element type, ``bc`` 32-bit row views
     [T, B | C], ``a_log`` [inner, n_state] and ``d_skip`` [inner] 32-bit, ``state`` [slots, inner, n_state] 32-bit;
-    ``out`` [T, inner] = (S C + D x) silu(z)."""
+    ``out`` [T, inner] = (S C + D x) silu(z).  ``w_dt`` (row views [inner, rank], every entry of the step bringing exactly
+    one token): ``dt`` holds low-rank rows [T, rank] and the step sizes are w_dt . dt, worked out in the kernel."""
+    if w_dt is not None and (w_dt.shape[1] != dt.shape[1] or x.shape[0] != n_entries):
+        raise KernelError("selective_scan: low-rank step sizes in rows of the small matrix's width, one token an entry")
     for t in (dt, bc, a_log, d_skip, state):
         if t.dtype != torch.float32:
             raise KernelError("selective_scan: the recurrence is 32-bit")
@@ -688,7 +691,8 @@ def selective_scan(dt, dt_bias, x, z, bc, a_log, d_skip, state, out, token_seq, 
     inner, n_state = a_log.shape
     if not (a_log.is_contiguous() and d_skip.is_contiguous() and bc.shape[1] == 2 * n_state):
         raise KernelError("selective_scan: contiguous constants, rows of [B | C]")
-    call("fx_selective_scan", _ptr(dt), _rows(dt), _ptr(dt_bias), code(dt_bias), _ptr(x), _rows(x), _ptr(z), _rows(z), code(x),
+    call("fx_selective_scan", _ptr(dt), _rows(dt), _ptr(w_dt), code(w_dt) if w_dt is not None else 0,
+         _rows(w_dt) if w_dt is not None else 0, w_dt.shape[1] if w_dt is not None else 0, _ptr(dt_bias), code(dt_bias), _ptr(x), _rows(x), _ptr(z), _rows(z), code(x),
          _ptr(bc), _rows(bc), _ptr(a_log), _ptr(d_skip), _ptr(state), _ptr(out), _rows(out), _ptr(token_seq),
          _ptr(seq_slot), x.shape[0], int(n_entries), int(inner), int(n_state), stream if stream is not None else stream_ptr())
     return out

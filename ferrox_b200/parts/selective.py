@@ -20,6 +20,10 @@ from ..weights.loader import TensorDecl
 from .base import Mixer, register_part
 
 
+# A decode step of up to this many requests leaves the step sizes' small product to the recurrence's kernel.
+STEP_IN_SCAN_MAX_TOKENS = 16
+
+
 def _pad_rows(w: torch.Tensor, multiple: int) -> torch.Tensor:
     """Rows of zeros that bring a matrix's height to a multiple."""
     extra = -w.shape[0] % multiple
@@ -97,14 +101,17 @@ class SelectiveScan(Mixer):
             ops.conv_tail_update(xz, I, s.conv_taps, tail, batch.token_seq, batch.seq_slot, batch.n_seqs, stream=st)
         low = rt.empty(T, self.w_x.shape[0], dtype=f32)              # [dt | B | C]
         ops.linear(xc, self.w_x, low, status=batch.status, stream=st)
-        dt = rt.empty(T, I, dtype=f32)
-        dt_low = low[:, :R]
-        if self.dt_pad:
-            dt_low = ops.split_rows(dt_low, rt.empty(T, 2 * self.dt_pad, dtype=torch.bfloat16), stream=st)
-        ops.linear(dt_low, self.w_dt, dt, status=batch.status, stream=st)
+        dt, dt_low, w_dt = None, low[:, :R], None
+        if single and T <= STEP_IN_SCAN_MAX_TOKENS:
+            dt, w_dt = dt_low, self.w_dt[:, :R]      # the recurrence's kernel works out its channels' step sizes itself
+        else:
+            dt = rt.empty(T, I, dtype=f32)
+            if self.dt_pad:
+                dt_low = ops.split_rows(dt_low, rt.empty(T, 2 * self.dt_pad, dtype=torch.bfloat16), stream=st)
+            ops.linear(dt_low, self.w_dt, dt, status=batch.status, stream=st)
         y = rt.empty(T, I)
         ops.selective_scan(dt, self.dt_b, xc, xz[:, I:], low[:, R:R + 2 * s.n_state], self.a_log, self.d_skip, state, y,
-                           batch.token_seq, batch.seq_slot, batch.n_seqs, stream=st)
+                           batch.token_seq, batch.seq_slot, batch.n_seqs, stream=st, w_dt=w_dt)
         ops.linear(y, self.w_o, out, accumulate=accumulate, status=batch.status, stream=st)
 
 
