@@ -68,7 +68,7 @@ __global__ void __launch_bounds__(NTHREADS) decode_mma_kernel(
     const int h0 = kvh * group_size + (blockIdx.x % chunks) * MAXQ;   // first query head of this block
     const int nq = min(MAXQ, kvh * group_size + group_size - h0);
     const int tkn = blockIdx.y, split = blockIdx.z;
-    const int pos = positions[tkn];
+    const int pos = fx_ld_old(positions + tkn);
     const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     int k_begin, k_end;
     fx_split_range(pos, lo, split, n_splits, split_len, k_begin, k_end);
@@ -84,7 +84,7 @@ __global__ void __launch_bounds__(NTHREADS) decode_mma_kernel(
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t4 = lane & 3;
     const int chunks_row = head_dim / 8;                   // 16-byte chunks per row
-    const int* table = block_table + (long)seq_slot[token_seq[tkn]] * table_width;
+    const int* table = block_table + (long)fx_ld_old(seq_slot + fx_ld_old(token_seq + tkn)) * table_width;
     const long head_stride = (long)page_size * head_dim;
     const int n_tiles = (k_end - k_begin + TK - 1) / TK;
 

@@ -125,8 +125,8 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
     const int h0 = kvh * group_size + (blockIdx.x % chunks) * MAXQ;   // first query head of this block
     const int nq = min(MAXQ, kvh * group_size + group_size - h0);
     const int tkn = blockIdx.y, split = blockIdx.z;
-    const int pos = a.positions[tkn];
-    const int seq = a.token_seq[tkn];                 // (asked for beside the position: the table row hangs on it)
+    const int pos = fx_ld_old(a.positions + tkn);
+    const int seq = fx_ld_old(a.token_seq + tkn);                 // (asked for beside the position: the table row hangs on it)
     const int lo = fx_first_key(pos, a.window, a.x.chunk);
     int k_begin, k_end;
     fx_split_range(pos, lo, split, a.n_splits, a.split_len, k_begin, k_end);
@@ -164,7 +164,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
     if (warp == 4) {
         // ---------------- producer: one thread asks for every tile ----------------
         if (lane == 0) {
-            const int* table = a.block_table + (long)a.seq_slot[seq] * a.table_width;
+            const int* table = a.block_table + (long)fx_ld_old(a.seq_slot + seq) * a.table_width;
             bool waited = false;
             // table entries are read one tile ahead, so that a stage that comes free is asked for at once
             int page_next = table[first_tile * TK / a.page_size];
@@ -204,7 +204,7 @@ __global__ void __launch_bounds__(NTHREADS, DMAX <= 128 ? 2 : 1) decode_tma_kern
         const bool owns_new = a.store_new && pos >= k_begin && pos < k_end && warp == ((pos % TK) >> 4);
         const bool writes_page = owns_new && a.write_pages && blockIdx.x % chunks == 0;
         // (the table is not the work of the kernel before this one: the page is looked up before the wait for it)
-        const int new_page = writes_page ? a.block_table[(long)a.seq_slot[seq] * a.table_width + pos / a.page_size] : -1;
+        const int new_page = writes_page ? fx_ld_old(a.block_table + (long)fx_ld_old(a.seq_slot + seq) * a.table_width + pos / a.page_size) : -1;
         fx_pdl_wait();
         // query rows of this block (zero beyond the group): on their way while the new key is prepared
         for (int c = threadIdx.x; c < 16 * chunks_row; c += NCONSUMERS) {

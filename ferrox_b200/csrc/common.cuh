@@ -214,6 +214,11 @@ __device__ __forceinline__ void fx_pdl_wait() {
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
 }
 
+// What may be read before the wait: constants, and with fx_ld_old what an earlier kernel or copy than the one before this
+// one has written.  (A plain load may find a line in the SM's own cache that was read before it was written, when no kernel
+// has come to its wait on this SM since: fx_ld_old asks the L2.)
+__device__ __forceinline__ int fx_ld_old(const int* p) { return __ldcg(p); }
+
 // The two halves apart, for a kernel that runs long on few warps (a recurrence over a prompt's tokens): it waits first
 // thing and lets its dependents be set up when its long loop is over, so that their waiting blocks do not sit on its
 // SMs meanwhile.

@@ -91,8 +91,8 @@ __device__ __forceinline__ Tile tile_of(int id, const SwArgs& a, int t_tiles, in
         int lo = 0, hi = a.n_groups;            // largest e with cum[e] <= ti
         while (hi - lo > 1) { const int mid = (lo + hi) >> 1; if (cum[mid] <= ti) lo = mid; else hi = mid; }
         t.group = lo;
-        t.r0 = a.group_offsets[lo] + (ti - cum[lo]) * TNB;
-        t.row_end = a.group_offsets[lo + 1];
+        t.r0 = fx_ld_old(a.group_offsets + lo) + (ti - cum[lo]) * TNB;
+        t.row_end = fx_ld_old(a.group_offsets + lo + 1);
     }
     return t;
 }
@@ -152,7 +152,7 @@ __global__ void __launch_bounds__(NTHREADS, (TNB <= 32 ? 2 : 1)) gemm_tc_swap_ke
     int t_tiles = (a.M + TNB - 1) / TNB;
     if (a.group_offsets) {
         for (int e = threadIdx.x; e < a.n_groups; e += NTHREADS)
-            cum_s[e + 1] = (a.group_offsets[e + 1] - a.group_offsets[e] + TNB - 1) / TNB;
+            cum_s[e + 1] = (fx_ld_old(a.group_offsets + e + 1) - fx_ld_old(a.group_offsets + e) + TNB - 1) / TNB;
         __syncthreads();
         if (threadIdx.x == 0) {
             int run = 0;
